@@ -13,6 +13,9 @@ LIB_PATH = os.path.join(HERE, "libcutb.so")
 OK, ERR_INVALID, ERR_UNSUPPORTED, ERR_CUDA, ERR_WORKSPACE, ERR_TIMEOUT, ERR_RANGE = range(7)
 Q8_0, Q4_0, Q4_K, Q5_K, Q6_K, BF16, Q4_1, Q5_0 = 0, 1, 2, 3, 4, 5, 6, 7  # from Q5_K on: cutb_dequant only
 F32, F16 = 0, 1
+UNARY_RELU_SQUARE, NO_TOKEN = 200, 0xFFFFFFFF
+DENSE_AUTO, DENSE_MATVEC, DENSE_TC, DENSE_SIMT = -1, 0, 1, 2
+ROT_HALVES, ROT_NEIGHBOURS = 0, 1
 LAYOUT_GGUF_BLOCKS, LAYOUT_KN_PLANES = 0, 1
 FUSION_NONE, FUSION_UNARY, FUSION_BINARY = 0, 1, 2
 VARIANT_AUTO, VARIANT_GENERIC, VARIANT_GEMV_MMA, VARIANT_GEMM_TC, VARIANT_GEMV_PLANES = -1, 0, 1, 2, 3
@@ -33,6 +36,8 @@ EXPORTS = [
     "cutb_dequant", "cutb_separate_blocks", "cutb_transpose_2d", "cutb_requant_q4k_affine", "cutb_quantize_rows_q8_0", "cutb_requant_q8_0_blocks",
     "cutb_transpose_q4", "cutb_version", "cutb_status_string", "cutb_last_error", "cutb_device_sm_count",
     "cutb_variant_name",
+    "cutb_dense_select_variant", "cutb_dense_workspace_bytes", "cutb_dense_matmul", "cutb_residual_norm", "cutb_embedding_bigram",
+    "cutb_mingru_scan", "cutb_sequence_advance", "cutb_window_kv_write", "cutb_window_attention", "cutb_window_attention_decode",
 ]
 
 
@@ -50,6 +55,62 @@ class QMatmulDesc(C.Structure):
         ("status", C.c_void_p),
         ("flags", C.c_uint32),
         ("a_norm_weight", C.c_void_p), ("a_norm_eps", C.c_float),
+    ]
+
+
+class DenseDesc(C.Structure):
+    _fields_ = [
+        ("a_dtype", C.c_int32), ("c_dtype", C.c_int32),
+        ("M", C.c_uint32), ("K", C.c_uint32), ("N", C.c_uint32),
+        ("A", C.c_void_p), ("lda", C.c_uint32),
+        ("W", C.c_void_p), ("ldw", C.c_uint32),
+        ("bias", C.c_void_p), ("unary_op", C.c_int32),
+        ("C", C.c_void_p), ("ldc", C.c_uint32),
+        ("variant", C.c_int32), ("flags", C.c_uint32),
+        ("workspace", C.c_void_p), ("workspace_bytes", C.c_uint64),
+        ("status", C.c_void_p),
+        ("res_x", C.c_void_p), ("res_y", C.c_void_p), ("res_norm_w", C.c_void_p), ("norm_w", C.c_void_p),
+        ("res_out", C.c_void_p),
+        ("norm_groups", C.c_uint32), ("norm_eps", C.c_float),
+        ("gru_state", C.c_void_p),
+    ]
+
+
+class ResidualNormDesc(C.Structure):
+    _fields_ = [
+        ("x", C.c_void_p), ("y", C.c_void_p), ("post_w", C.c_void_p), ("pre_w", C.c_void_p),
+        ("x_out", C.c_void_p), ("h", C.c_void_p), ("row_index", C.c_void_p),
+        ("ldx", C.c_uint64), ("ldy", C.c_uint64), ("ldh", C.c_uint64),
+        ("rows", C.c_uint32), ("dim", C.c_uint32), ("groups", C.c_uint32),
+        ("eps", C.c_float), ("h_dtype", C.c_int32),
+    ]
+
+
+class EmbedDesc(C.Structure):
+    _fields_ = [
+        ("tokens", C.c_void_p), ("prev", C.c_void_p), ("embed", C.c_void_p), ("bigram", C.c_void_p), ("out", C.c_void_p),
+        ("ld_embed", C.c_uint64), ("ld_bigram", C.c_uint64), ("ldo", C.c_uint64),
+        ("n", C.c_uint32), ("dim", C.c_uint32), ("vocab", C.c_uint32), ("buckets", C.c_uint32),
+        ("mul_prev", C.c_uint32), ("mul_cur", C.c_uint32),
+        ("status", C.c_void_p),
+    ]
+
+
+class WindowAttnDesc(C.Structure):
+    _fields_ = [
+        ("kv_dtype", C.c_int32), ("out_dtype", C.c_int32),
+        ("n_heads", C.c_uint32), ("n_kv_heads", C.c_uint32), ("dim", C.c_uint32), ("vdim", C.c_uint32),
+        ("k_head", C.c_uint32), ("v_head", C.c_uint32),
+        ("ring_rows", C.c_uint32), ("window", C.c_uint32), ("rot_dims", C.c_uint32), ("max_pos", C.c_uint32),
+        ("rot_pairing", C.c_int32), ("sink", C.c_int32),
+        ("scale", C.c_float), ("v_mix", C.c_float),
+        ("cos_table", C.c_void_p), ("sin_table", C.c_void_p),
+        ("q", C.c_void_p), ("k", C.c_void_p), ("v", C.c_void_p), ("ldqkv", C.c_uint64),
+        ("k_cache", C.c_void_p), ("v_cache", C.c_void_p),
+        ("v_first", C.c_void_p), ("v_first_out", C.c_void_p), ("ld_first", C.c_uint64),
+        ("pos_ptr", C.c_void_p), ("pos", C.c_uint32), ("n_tokens", C.c_uint32),
+        ("out", C.c_void_p), ("ldo", C.c_uint64),
+        ("status", C.c_void_p),
     ]
 
 
@@ -72,91 +133,119 @@ class CutbError(RuntimeError):
 _lib = None
 
 
-def lib() -> C.CDLL:
+def _bind_layers(l: C.CDLL) -> None:
+    l.cutb_copy_batch.restype = C.c_int
+    l.cutb_copy_batch.argtypes = [C.c_void_p, C.c_uint32, C.c_uint64, C.c_void_p]
+    l.cutb_rmsnorm.restype = C.c_int
+    l.cutb_rmsnorm.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64, C.c_float, C.c_void_p]
+    l.cutb_embedding.restype = C.c_int
+    l.cutb_embedding.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint64, C.c_uint32, C.c_uint32, C.c_void_p, C.c_void_p]
+    l.cutb_embedding_col.restype = C.c_int
+    l.cutb_embedding_col.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32,
+                                     C.c_uint32, C.c_uint32, C.c_uint32, C.c_void_p, C.c_void_p]
+    l.cutb_argreduce.restype = C.c_int
+    l.cutb_argreduce.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_uint32, C.c_void_p]
+    l.cutb_glu_pairs.restype = C.c_int
+    l.cutb_glu_pairs.argtypes = [C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint64, C.c_int, C.c_void_p]
+    l.cutb_version.restype = C.c_int
+    l.cutb_status_string.restype = C.c_char_p
+    l.cutb_status_string.argtypes = [C.c_int]
+    l.cutb_last_error.restype = C.c_char_p
+    l.cutb_device_sm_count.restype = C.c_int
+    for name, desc in (("cutb_dense_matmul", DenseDesc), ("cutb_residual_norm", ResidualNormDesc), ("cutb_embedding_bigram", EmbedDesc),
+                       ("cutb_window_kv_write", WindowAttnDesc), ("cutb_window_attention", WindowAttnDesc),
+                       ("cutb_window_attention_decode", WindowAttnDesc)):
+        getattr(l, name).restype = C.c_int
+        getattr(l, name).argtypes = [C.POINTER(desc), C.c_void_p]
+    l.cutb_dense_select_variant.restype = C.c_int
+    l.cutb_dense_select_variant.argtypes = [C.POINTER(DenseDesc)]
+    l.cutb_dense_workspace_bytes.restype = C.c_uint64
+    l.cutb_dense_workspace_bytes.argtypes = [C.POINTER(DenseDesc)]
+    l.cutb_mingru_scan.restype = C.c_int
+    l.cutb_mingru_scan.argtypes = [C.c_void_p, C.c_uint64, C.c_uint32, C.c_void_p, C.c_void_p, C.c_int, C.c_uint64, C.c_uint32, C.c_void_p]
+    l.cutb_sequence_advance.restype = C.c_int
+    l.cutb_sequence_advance.argtypes = [C.c_void_p, C.c_void_p, C.c_uint32, C.c_void_p, C.c_void_p]
+
+
+def _bind_quantized(l: C.CDLL) -> None:
+    l.cutb_qmatmul_workspace_bytes.restype = C.c_uint64
+    l.cutb_qmatmul_workspace_bytes.argtypes = [C.POINTER(QMatmulDesc)]
+    l.cutb_qmatmul_select_variant.restype = C.c_int
+    l.cutb_qmatmul_select_variant.argtypes = [C.POINTER(QMatmulDesc)]
+    l.cutb_qmatmul.restype = C.c_int
+    l.cutb_qmatmul.argtypes = [C.POINTER(QMatmulDesc), C.c_void_p]
+    l.cutb_qmatmul_decode_noalloc.restype = C.c_int
+    l.cutb_qmatmul_decode_noalloc.argtypes = [C.POINTER(QMatmulDesc), C.c_void_p]
+    l.cutb_qmatmul_scatter.restype = C.c_int
+    l.cutb_qmatmul_scatter.argtypes = [C.POINTER(QMatmulDesc), C.POINTER(PeerScatter), C.c_void_p]
+    l.cutb_peer_exchange.restype = C.c_int
+    l.cutb_peer_exchange.argtypes = [C.POINTER(PeerScatter), C.c_void_p, C.c_void_p, C.c_void_p]
+    l.cutb_peer_buffer_alloc.restype = C.c_int
+    l.cutb_peer_buffer_alloc.argtypes = [C.c_uint64, C.POINTER(C.c_void_p), C.c_char_p]
+    l.cutb_peer_buffer_open.restype = C.c_int
+    l.cutb_peer_buffer_open.argtypes = [C.c_char_p, C.POINTER(C.c_void_p)]
+    l.cutb_peer_buffer_close.restype = C.c_int
+    l.cutb_peer_buffer_close.argtypes = [C.c_void_p]
+    l.cutb_peer_buffer_free.restype = C.c_int
+    l.cutb_peer_buffer_free.argtypes = [C.c_void_p]
+    l.cutb_dequant.restype = C.c_int
+    l.cutb_dequant.argtypes = [C.c_int, C.c_void_p, C.c_uint64, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32,
+                               C.c_void_p]
+    l.cutb_embedding_blocks.restype = C.c_int
+    l.cutb_embedding_blocks.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32,
+                                        C.c_void_p, C.c_void_p]
+    l.cutb_requant_q8_0_blocks.restype = C.c_int
+    l.cutb_requant_q8_0_blocks.argtypes = [C.c_int, C.c_void_p, C.c_uint64, C.c_void_p, C.c_uint64, C.c_uint32, C.c_void_p]
+    l.cutb_rope_kv_write.restype = C.c_int
+    l.cutb_rope_kv_write.argtypes = [C.c_int] + [C.c_void_p] * 9 + [C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32,
+                                                                    C.c_void_p, C.c_void_p]
+    l.cutb_attention_workspace_bytes.restype = C.c_uint64
+    l.cutb_attention_workspace_bytes.argtypes = [C.c_uint32] * 4
+    l.cutb_attention_decode.restype = C.c_int
+    l.cutb_attention_decode.argtypes = [C.c_int] + [C.c_void_p] * 5 + [C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32,
+                                                                       C.c_float, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p]
+    l.cutb_rope_attention_decode.restype = C.c_int
+    l.cutb_rope_attention_decode.argtypes = [C.c_int] + [C.c_void_p] * 9 + [C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32,
+                                                                            C.c_float, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p]
+    l.cutb_batched_kv_write.restype = C.c_int
+    l.cutb_batched_kv_write.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32] + [C.c_void_p] * 5 + [
+        C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32, C.c_void_p, C.c_void_p]
+    l.cutb_batched_attention.restype = C.c_int
+    l.cutb_batched_attention.argtypes = [C.c_int, C.c_void_p, C.c_uint32] + [C.c_void_p] * 6 + [
+        C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32, C.c_float, C.c_void_p, C.c_void_p]
+    l.cutb_separate_blocks.restype = C.c_int
+    l.cutb_separate_blocks.argtypes = [C.c_int, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p, C.c_uint64, C.c_uint64, C.c_void_p]
+    l.cutb_transpose_2d.restype = C.c_int
+    l.cutb_transpose_2d.argtypes = [C.c_uint32, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint64, C.c_void_p]
+    l.cutb_requant_q4k_affine.restype = C.c_int
+    l.cutb_requant_q4k_affine.argtypes = [C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64,
+                                          C.c_uint64, C.c_void_p]
+    l.cutb_quantize_rows_q8_0.restype = C.c_int
+    l.cutb_quantize_rows_q8_0.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint64, C.c_void_p]
+    l.cutb_transpose_q4.restype = C.c_int
+    l.cutb_transpose_q4.argtypes = [C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32,
+                                    C.c_void_p]
+    l.cutb_variant_name.restype = C.c_char_p
+    l.cutb_variant_name.argtypes = [C.c_int]
+
+
+def load(path: str) -> C.CDLL:
+    """Loads libcutb.so, or the smaller libcutb_layers.so (no quantized matmul), as the library of this process."""
     global _lib
+    l = C.CDLL(path)
+    _bind_layers(l)
+    if os.path.basename(path) == os.path.basename(LIB_PATH):
+        _bind_quantized(l)
+    _lib = l
+    return l
+
+
+def lib() -> C.CDLL:
     if _lib is None:
         if not os.path.exists(LIB_PATH):
             raise RuntimeError(
                 f"{LIB_PATH} is missing: build it with `python -m cut_b200.build` (there is no CPU fallback)")
-        l = C.CDLL(LIB_PATH)
-        l.cutb_qmatmul_workspace_bytes.restype = C.c_uint64
-        l.cutb_qmatmul_workspace_bytes.argtypes = [C.POINTER(QMatmulDesc)]
-        l.cutb_qmatmul_select_variant.restype = C.c_int
-        l.cutb_qmatmul_select_variant.argtypes = [C.POINTER(QMatmulDesc)]
-        l.cutb_qmatmul.restype = C.c_int
-        l.cutb_qmatmul.argtypes = [C.POINTER(QMatmulDesc), C.c_void_p]
-        l.cutb_qmatmul_decode_noalloc.restype = C.c_int
-        l.cutb_qmatmul_decode_noalloc.argtypes = [C.POINTER(QMatmulDesc), C.c_void_p]
-        l.cutb_qmatmul_scatter.restype = C.c_int
-        l.cutb_qmatmul_scatter.argtypes = [C.POINTER(QMatmulDesc), C.POINTER(PeerScatter), C.c_void_p]
-        l.cutb_copy_batch.restype = C.c_int
-        l.cutb_copy_batch.argtypes = [C.c_void_p, C.c_uint32, C.c_uint64, C.c_void_p]
-        l.cutb_peer_exchange.restype = C.c_int
-        l.cutb_peer_exchange.argtypes = [C.POINTER(PeerScatter), C.c_void_p, C.c_void_p, C.c_void_p]
-        l.cutb_peer_buffer_alloc.restype = C.c_int
-        l.cutb_peer_buffer_alloc.argtypes = [C.c_uint64, C.POINTER(C.c_void_p), C.c_char_p]
-        l.cutb_peer_buffer_open.restype = C.c_int
-        l.cutb_peer_buffer_open.argtypes = [C.c_char_p, C.POINTER(C.c_void_p)]
-        l.cutb_peer_buffer_close.restype = C.c_int
-        l.cutb_peer_buffer_close.argtypes = [C.c_void_p]
-        l.cutb_peer_buffer_free.restype = C.c_int
-        l.cutb_peer_buffer_free.argtypes = [C.c_void_p]
-        l.cutb_dequant.restype = C.c_int
-        l.cutb_dequant.argtypes = [C.c_int, C.c_void_p, C.c_uint64, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32,
-                                   C.c_void_p]
-        l.cutb_rmsnorm.restype = C.c_int
-        l.cutb_rmsnorm.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64, C.c_float, C.c_void_p]
-        l.cutb_embedding.restype = C.c_int
-        l.cutb_embedding.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint64, C.c_uint32, C.c_uint32, C.c_void_p, C.c_void_p]
-        l.cutb_embedding_col.restype = C.c_int
-        l.cutb_embedding_col.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32,
-                                         C.c_uint32, C.c_uint32, C.c_uint32, C.c_void_p, C.c_void_p]
-        l.cutb_embedding_blocks.restype = C.c_int
-        l.cutb_embedding_blocks.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32,
-                                            C.c_void_p, C.c_void_p]
-        l.cutb_requant_q8_0_blocks.restype = C.c_int
-        l.cutb_requant_q8_0_blocks.argtypes = [C.c_int, C.c_void_p, C.c_uint64, C.c_void_p, C.c_uint64, C.c_uint32, C.c_void_p]
-        l.cutb_argreduce.restype = C.c_int
-        l.cutb_argreduce.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_uint32, C.c_void_p]
-        l.cutb_rope_kv_write.restype = C.c_int
-        l.cutb_rope_kv_write.argtypes = [C.c_int] + [C.c_void_p] * 9 + [C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32,
-                                                                        C.c_void_p, C.c_void_p]
-        l.cutb_attention_workspace_bytes.restype = C.c_uint64
-        l.cutb_attention_workspace_bytes.argtypes = [C.c_uint32] * 4
-        l.cutb_attention_decode.restype = C.c_int
-        l.cutb_attention_decode.argtypes = [C.c_int] + [C.c_void_p] * 5 + [C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32,
-                                                                           C.c_float, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p]
-        l.cutb_rope_attention_decode.restype = C.c_int
-        l.cutb_rope_attention_decode.argtypes = [C.c_int] + [C.c_void_p] * 9 + [C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32,
-                                                                                C.c_float, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p]
-        l.cutb_batched_kv_write.restype = C.c_int
-        l.cutb_batched_kv_write.argtypes = [C.c_int, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32] + [C.c_void_p] * 5 + [
-            C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32, C.c_void_p, C.c_void_p]
-        l.cutb_batched_attention.restype = C.c_int
-        l.cutb_batched_attention.argtypes = [C.c_int, C.c_void_p, C.c_uint32] + [C.c_void_p] * 6 + [
-            C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint32, C.c_float, C.c_void_p, C.c_void_p]
-        l.cutb_glu_pairs.restype = C.c_int
-        l.cutb_glu_pairs.argtypes = [C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint64, C.c_int, C.c_void_p]
-        l.cutb_separate_blocks.restype = C.c_int
-        l.cutb_separate_blocks.argtypes = [C.c_int, C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p, C.c_uint64, C.c_uint64, C.c_void_p]
-        l.cutb_transpose_2d.restype = C.c_int
-        l.cutb_transpose_2d.argtypes = [C.c_uint32, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64, C.c_uint64, C.c_void_p]
-        l.cutb_requant_q4k_affine.restype = C.c_int
-        l.cutb_requant_q4k_affine.argtypes = [C.c_void_p, C.c_uint64, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint64,
-                                              C.c_uint64, C.c_void_p]
-        l.cutb_quantize_rows_q8_0.restype = C.c_int
-        l.cutb_quantize_rows_q8_0.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint64, C.c_void_p]
-        l.cutb_transpose_q4.restype = C.c_int
-        l.cutb_transpose_q4.argtypes = [C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32,
-                                        C.c_void_p]
-        l.cutb_version.restype = C.c_int
-        l.cutb_status_string.restype = C.c_char_p
-        l.cutb_status_string.argtypes = [C.c_int]
-        l.cutb_last_error.restype = C.c_char_p
-        l.cutb_device_sm_count.restype = C.c_int
-        l.cutb_variant_name.restype = C.c_char_p
-        l.cutb_variant_name.argtypes = [C.c_int]
-        _lib = l
+        load(LIB_PATH)
     return _lib
 
 

@@ -13,9 +13,14 @@ import subprocess
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libcutb.so")
-SOURCES = ["cabi.cu", "common.cu", "qgemv_blocks.cu", "qmatmul_generic.cu", "dequant.cu", "transpose_q4.cu",
-           "qgemm_tc.cu", "qgemm_skinny.cu", "repack.cu", "layer_ops.cu", "attention.cu", "attention_prefill.cu", "qgemv_planes.cu"]
-HEADERS = ["common.cuh", "kernels.h", "qgemm_tc_common.cuh", os.path.join("..", "..", "include", "cutb.h")]
+# layer operators and the layer-list models over dense bf16 weights: what a model without quantized weights needs
+LAYER_SOURCES = ["cabi_layers.cu", "common.cu", "layer_ops.cu", "mixer_ops.cu", "dense_matvec.cu", "dense_gemm.cu", "window_attention.cu"]
+QUANT_SOURCES = ["cabi.cu", "qgemv_blocks.cu", "qmatmul_generic.cu", "dequant.cu", "transpose_q4.cu",
+                 "qgemm_tc.cu", "qgemm_skinny.cu", "repack.cu", "attention.cu", "attention_prefill.cu", "qgemv_planes.cu"]
+SOURCES = QUANT_SOURCES + LAYER_SOURCES
+LAYERS_LIB = os.path.join(HERE, "libcutb_layers.so")
+HEADERS = ["common.cuh", "kernels.h", "tcgen05.cuh", "qgemm_tc_common.cuh", "dense_common.cuh", "norm_stage.cuh",
+           os.path.join("..", "..", "include", "cutb.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC,-fvisibility=hidden"]
 
@@ -34,31 +39,54 @@ def _stale(target: str, deps: list[str]) -> bool:
     return any(os.path.getmtime(d) > t for d in deps)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
-    """Compile every .cu into an object (only the stale ones) and link libcutb.so."""
+def _build(lib: str, sources: list[str], force: bool, verbose: bool) -> str:
+    """Compile the stale objects of `sources` side by side and link `lib`.  Objects and library appear under their names only
+    when complete, so two builds of one tree do not read each other's halves."""
     objdir = os.path.join(HERE, "build")
     os.makedirs(objdir, exist_ok=True)
     hdrs = [os.path.join(CSRC, h) for h in HEADERS]
     objs, procs = [], []
-    for src in SOURCES:
+    for src in sources:
         s = os.path.join(CSRC, src)
         o = os.path.join(objdir, src.replace(".cu", ".o"))
         objs.append(o)
         if force or _stale(o, [s] + hdrs):
-            cmd = [_nvcc(), *NVCC_FLAGS, "-c", s, "-o", o] + (["-Xptxas", "-v"] if verbose else [])
-            procs.append((src, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
-    for src, p in procs:
+            tmp = f"{o}.{os.getpid()}"
+            cmd = [_nvcc(), *NVCC_FLAGS, "-c", s, "-o", tmp] + (["-Xptxas", "-v"] if verbose else [])
+            procs.append((src, o, tmp, subprocess.Popen(cmd, stdout=subprocess.PIPE, stderr=subprocess.STDOUT, text=True)))
+    failed = []
+    for src, o, tmp, p in procs:
         out, _ = p.communicate()
         if p.returncode != 0:
-            raise RuntimeError(f"nvcc failed on {src}:\n{out}")
+            failed.append(f"nvcc failed on {src}:\n{out}")
+            continue
+        os.replace(tmp, o)
         if verbose:
             print(out)
-    if force or procs or _stale(LIB, objs):
-        cmd = [_nvcc(), "-shared", "-o", LIB, *objs, "-Xcompiler", "-fPIC"]
+    if failed:
+        raise RuntimeError("\n".join(failed))
+    if force or procs or _stale(lib, objs):
+        tmp = f"{lib}.{os.getpid()}"
+        cmd = [_nvcc(), "-shared", "-o", tmp, *objs, "-Xcompiler", "-fPIC"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}{r.stderr}")
-    return LIB
+        os.replace(tmp, lib)
+    return lib
+
+
+def build(force: bool = False, verbose: bool = False) -> str:
+    """Compile every .cu into an object (only the stale ones) and link libcutb.so."""
+    return _build(LIB, SOURCES, force, verbose)
+
+
+def build_layers(force: bool = False, verbose: bool = False) -> str:
+    """The library a model without quantized weights runs on: libcutb.so if it is there and current, else libcutb_layers.so
+    from the same objects without the quantized-matmul kernels (a fraction of the compile time)."""
+    every = [os.path.join(CSRC, f) for f in SOURCES + HEADERS]
+    if not force and not _stale(LIB, every):
+        return LIB
+    return _build(LAYERS_LIB, LAYER_SOURCES, force, verbose)
 
 
 HOST_LIB = os.path.join(HERE, "libcut_host.so")

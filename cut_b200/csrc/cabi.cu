@@ -135,23 +135,6 @@ using namespace cutb;
 
 extern "C" {
 
-int cutb_version(void) { return CUTB_VERSION; }
-
-const char *cutb_status_string(int status) {
-  switch (status) {
-    case CUTB_OK: return "ok";
-    case CUTB_ERR_INVALID: return "invalid argument";
-    case CUTB_ERR_UNSUPPORTED: return "unsupported request";
-    case CUTB_ERR_CUDA: return "CUDA error";
-    case CUTB_ERR_WORKSPACE: return "workspace missing or too small";
-    case CUTB_ERR_TIMEOUT: return "device-side wait timed out";
-    case CUTB_ERR_RANGE: return "activation outside the fp16 operand range";
-    default: return "unknown status";
-  }
-}
-
-const char *cutb_last_error(void) { return cutb::last_error(); }
-
 const char *cutb_variant_name(int variant) {
   switch (variant) {
     case CUTB_VARIANT_GENERIC: return "QMatMulGeneric";
@@ -160,12 +143,6 @@ const char *cutb_variant_name(int variant) {
     case CUTB_VARIANT_GEMV_PLANES: return "QGemvPlanes";
     default: return "Unknown";
   }
-}
-
-int cutb_device_sm_count(void) {
-  DeviceInfo di;
-  if (get_device_info(&di) != CUTB_OK) return -1;
-  return di.sm_count;
 }
 
 int cutb_qmatmul_select_variant(const cutb_qmatmul_desc *desc) {
@@ -392,51 +369,6 @@ int cutb_requant_q8_0_blocks(int format, const void *raw, uint64_t raw_bytes, vo
   return requant_q8_0_blocks_launch(format, raw, out, rows, cols, reinterpret_cast<cudaStream_t>(stream));
 }
 
-int cutb_rmsnorm(int dtype, const void *x, const void *weight, void *y, uint32_t rows, uint32_t dim, uint64_t ldx, float eps,
-                 void *stream) {
-  if (dtype != CUTB_F32 && dtype != CUTB_F16) {
-    set_last_error("rmsnorm: dtype must be fp32 or fp16");
-    return CUTB_ERR_INVALID;
-  }
-  if (rows == 0 || dim == 0) return CUTB_OK;
-  if (!x || !weight || !y || ldx < dim) {
-    set_last_error("rmsnorm: null pointer or row stride shorter than the row");
-    return CUTB_ERR_INVALID;
-  }
-  return rmsnorm_launch(dtype, x, weight, y, rows, dim, ldx, eps, reinterpret_cast<cudaStream_t>(stream));
-}
-
-int cutb_embedding(const uint32_t *indices, const float *table, float *out, uint64_t n, uint32_t dim, uint32_t vocab, int *status,
-                   void *stream) {
-  if (n == 0 || dim == 0) return CUTB_OK;
-  if (!indices || !table || !out || reinterpret_cast<uintptr_t>(table) % 16 || reinterpret_cast<uintptr_t>(out) % 16) {
-    set_last_error("embedding: null pointer, or table / output not 16-byte aligned");
-    return CUTB_ERR_INVALID;
-  }
-  return embedding_launch(indices, table, out, n, dim, vocab, status, reinterpret_cast<cudaStream_t>(stream));
-}
-
-int cutb_embedding_col(int format, const uint32_t *indices, const void *matrix, const void *scales, float *out, uint32_t n,
-                       uint32_t dim, uint32_t vocab, uint32_t vocab_stride, uint32_t scale_stride, uint32_t out_stride, int *status,
-                       void *stream) {
-  if (n == 0 || dim == 0) return CUTB_OK;
-  if (format != 0 && format != 1) {
-    set_last_error("embedding_col: format must be 0 (fp16 matrix) or 1 (int8 values + fp16 scales)");
-    return CUTB_ERR_INVALID;
-  }
-  if (!indices || !matrix || !out || (format == 1 && !scales)) {
-    set_last_error("embedding_col: null pointer");
-    return CUTB_ERR_INVALID;
-  }
-  if (vocab_stride < vocab || out_stride < dim || (format == 1 && scale_stride < vocab) ||
-      (format == 0 && reinterpret_cast<uintptr_t>(matrix) % 2) || (format == 1 && reinterpret_cast<uintptr_t>(scales) % 2)) {
-    set_last_error("embedding_col: a stride is shorter than its row, or an fp16 pointer is misaligned");
-    return CUTB_ERR_INVALID;
-  }
-  return embedding_col_launch(format, indices, matrix, scales, out, n, dim, vocab, vocab_stride, scale_stride, out_stride, status,
-                              reinterpret_cast<cudaStream_t>(stream));
-}
-
 int cutb_embedding_blocks(int format, const uint32_t *indices, const void *raw, float *out, uint32_t n, uint32_t rows, uint32_t cols,
                           uint32_t ldo, int *status, void *stream) {
   if (n == 0 || cols == 0) return CUTB_OK;
@@ -449,14 +381,6 @@ int cutb_embedding_blocks(int format, const uint32_t *indices, const void *raw, 
     return CUTB_ERR_INVALID;
   }
   return dequant_gather_launch(format, indices, raw, out, n, rows, cols, ldo, status, reinterpret_cast<cudaStream_t>(stream));
-}
-
-int cutb_argreduce(int is_max, const float *values, float *out, uint32_t n, void *stream) {
-  if (!out || (n && !values)) {
-    set_last_error("argreduce: null pointer");
-    return CUTB_ERR_INVALID;
-  }
-  return argreduce_launch(is_max, values, out, n, reinterpret_cast<cudaStream_t>(stream));
 }
 
 int cutb_rope_kv_write(int kv_dtype, const float *q, const float *k, const float *v, const uint32_t *params, const float *cos_table,
@@ -614,28 +538,6 @@ int cutb_batched_attention(int kv_dtype, const float *q_in, uint32_t q_stride, c
   }
   return batched_attention_launch(kv_dtype, q_in, q_stride, k_cache, v_cache, positions, cos_table, sin_table, out, out_stride, n_tokens,
                                   n_heads, n_kv_heads, head_dim, ld, max_seq, scale, status, reinterpret_cast<cudaStream_t>(stream));
-}
-
-int cutb_copy_batch(const cutb_copy_range *table, uint32_t n, uint64_t max_bytes, void *stream) {
-  if (n == 0) return CUTB_OK;
-  if (!table || n > 65535) {
-    set_last_error("copy_batch: null table or more than 65535 ranges");
-    return CUTB_ERR_INVALID;
-  }
-  // (the ranges themselves are read on the device: their alignment is the caller's contract)
-  uint64_t blocks = (max_bytes / 16 + 2047) / 2048;  // about eight vectors per thread
-  if (blocks < 1) blocks = 1;
-  if (blocks > 64) blocks = 64;
-  return copy_batch_launch(table, n, (uint32_t)blocks, reinterpret_cast<cudaStream_t>(stream));
-}
-
-int cutb_glu_pairs(const float *in, float *out, uint32_t rows, uint32_t cols_out, uint64_t ldi, uint64_t ldo, int unary_op, void *stream) {
-  if (rows == 0 || cols_out == 0) return CUTB_OK;
-  if (!in || !out || ldi % 2 || ldi < 2ull * cols_out || ldo < cols_out || reinterpret_cast<uintptr_t>(in) % 8) {
-    set_last_error("glu_pairs: null pointer, odd or short ldi, short ldo, or input not 8-byte aligned");
-    return CUTB_ERR_INVALID;
-  }
-  return glu_pairs_launch(in, out, rows, cols_out, ldi, ldo, unary_op, reinterpret_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

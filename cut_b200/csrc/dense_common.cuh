@@ -1,0 +1,47 @@
+// Elementwise pieces shared by the kernels of the layer-list models (dense bf16 weights).
+#pragma once
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace cutb {
+namespace {
+
+__device__ __forceinline__ float bf16_lo(uint32_t x) { return __uint_as_float(x << 16); }
+__device__ __forceinline__ float bf16_hi(uint32_t x) { return __uint_as_float(x & 0xffff0000u); }
+__device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
+  const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t *>(&h);
+}
+// 16 bytes that are read once: keep them out of L1
+__device__ __forceinline__ uint4 ld_stream(const uint4 *p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+__device__ __forceinline__ void store_out(void *C, int bf16, size_t i, float v) {
+  if (bf16) reinterpret_cast<__nv_bfloat16 *>(C)[i] = __float2bfloat16_rn(v);
+  else reinterpret_cast<float *>(C)[i] = v;
+}
+__device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+
+// Elementwise epilogue: 0 none, CUTB_UNARY_RELU_SQUARE, or one of the unary codes of the quantized matmul.
+__device__ __forceinline__ float dense_unary(float x, int op) {
+  if (op == 0) return x;
+  if (op == CUTB_UNARY_RELU_SQUARE) {
+    const float r = fmaxf(x, 0.f);
+    return r * r;
+  }
+  return apply_epilogue(x, CUTB_FUSION_UNARY, op, 0.f);
+}
+
+// The gated recurrence of one channel: gate z and candidate c from this token's pre-activations.
+__device__ __forceinline__ float mingru_candidate(float u) { return u >= 0.f ? u + 0.5f : sigmoid(u); }
+__device__ __forceinline__ float mingru_update(float s, float z_pre, float u) {
+  const float z = sigmoid(z_pre);
+  return fmaf(1.0f - z, s, z * mingru_candidate(u));
+}
+
+}  // namespace
+}  // namespace cutb

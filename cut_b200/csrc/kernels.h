@@ -82,6 +82,22 @@ int attention_decode_launch(int kv_dtype, const float *q, const void *kC, const 
                             uint32_t nHeads, uint32_t nKvHeads, uint32_t headDim, uint64_t ld, uint32_t max_seq, float scale,
                             void *workspace, int *status, cudaStream_t stream);
 
+// Layer-list models over dense bf16 weights (dense_matvec.cu, dense_gemm.cu, mixer_ops.cu, window_attention.cu).
+bool dense_matvec_supported(const cutb_dense_desc &d);
+int dense_matvec_launch(const cutb_dense_desc &d, cudaStream_t stream);
+bool dense_gemm_tc_supported(const cutb_dense_desc &d);
+uint64_t dense_gemm_tc_workspace(const cutb_dense_desc &d);
+int dense_gemm_tc_launch(const cutb_dense_desc &d, cudaStream_t stream);
+int dense_gemm_simt_launch(const cutb_dense_desc &d, cudaStream_t stream);
+int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream);
+int embedding_bigram_launch(const cutb_embed_desc &d, cudaStream_t stream);
+int mingru_scan_launch(const float *zxg, uint64_t ld, uint32_t width, float *state, void *out, int out_dtype, uint64_t ldo, uint32_t T,
+                       cudaStream_t stream);
+int sequence_advance_launch(cutb_sequence_state *s, const uint32_t *tokens, uint32_t n, const float *next, cudaStream_t stream);
+int window_kv_write_launch(const cutb_window_attn_desc &d, cudaStream_t stream);
+int window_attention_launch(const cutb_window_attn_desc &d, cudaStream_t stream);
+int window_attention_decode_launch(const cutb_window_attn_desc &d, cudaStream_t stream);
+
 // Load-time repacks (repack.cu), bit-exact with the reference's CPU loader / runner code.
 int separate_launch(int format, const void *raw, void *values, void *scales, uint64_t rows, uint64_t cols, cudaStream_t stream);
 int transpose_launch(uint32_t elem_bytes, const void *in, void *out, uint32_t R, uint32_t C, uint64_t ldi, uint64_t ldo,

@@ -1,0 +1,150 @@
+// Bandwidth-bound operators of the layer-list models: embedding with a hashed bigram table, the norm / residual step between
+// two sublayers for a batch of tokens, the minGRU scan, and the hand-over of a sequence's {token, previous token, position}.
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+#include "dense_common.cuh"
+#include "kernels.h"
+#include "norm_stage.cuh"
+
+namespace cutb {
+namespace {
+
+// out[i, :] = embed[token_i] + bigram[(prev_i * mul_prev + token_i * mul_cur) mod buckets]; a sequence's first token has no
+// previous one and takes row `buckets`.  One block per token.
+__global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_desc d) {
+  pdl_enter();
+  const uint32_t i = blockIdx.x;
+  uint32_t tok = __ldg(d.tokens + i);
+  uint32_t prev = i ? __ldg(d.tokens + i - 1) : (d.prev ? *d.prev : CUTB_NO_TOKEN);
+  const bool bad = tok >= d.vocab || (prev != CUTB_NO_TOKEN && prev >= d.vocab);
+  float *out = d.out + (size_t)i * d.ldo;
+  if (bad) {  // never read outside the tables
+    if (d.status && threadIdx.x == 0) atomicExch(d.status, (int)CUTB_ERR_INVALID);
+    for (uint32_t c = threadIdx.x; c < d.dim; c += 256) out[c] = 0.f;
+    return;
+  }
+  const __nv_bfloat16 *e = reinterpret_cast<const __nv_bfloat16 *>(d.embed) + (size_t)tok * d.ld_embed;
+  const __nv_bfloat16 *b = nullptr;
+  if (d.bigram) {
+    const uint64_t row = prev == CUTB_NO_TOKEN ? d.buckets : ((uint64_t)prev * d.mul_prev + (uint64_t)tok * d.mul_cur) % d.buckets;
+    b = reinterpret_cast<const __nv_bfloat16 *>(d.bigram) + row * d.ld_bigram;
+  }
+  for (uint32_t c = threadIdx.x; c < d.dim; c += 256) out[c] = __bfloat162float(e[c]) + (b ? __bfloat162float(b[c]) : 0.f);
+}
+
+// One block per row: x' = x + N(y), h = N(x') (norm_stage.cuh), h in bf16 or fp32.
+__global__ void __launch_bounds__(256) residual_norm_kernel(NormStage n, uint64_t ldx, uint64_t ldy, const uint32_t *row_index, void *h,
+                                                            uint64_t ldh, int h_bf16) {
+  extern __shared__ __align__(16) float rn_smem[];
+  pdl_enter();
+  const uint32_t row = blockIdx.x, src = row_index ? __ldg(row_index + row) : row;
+  n.x += src * ldx;
+  if (n.y) n.y += src * ldy;
+  if (n.x_out) n.x_out += src * ldx;
+  const size_t base = (size_t)row * ldh;
+  auto put4 = [&](uint32_t i, float4 v) {
+    if (h_bf16) *reinterpret_cast<uint2 *>(reinterpret_cast<__nv_bfloat16 *>(h) + base + i) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+    else *reinterpret_cast<float4 *>(reinterpret_cast<float *>(h) + base + i) = v;
+  };
+  auto put1 = [&](uint32_t i, float v) { store_out(h, h_bf16, base + i, v); };
+  stage_norm(n, rn_smem, n.x_out != nullptr, put4, put1);
+}
+
+// The recurrence over T tokens.  A block owns SC_CH channels; SC_SEG groups of threads take consecutive segments of SC_L
+// tokens each, so a turn covers SC_SEG * SC_L tokens.  A segment is first reduced to the affine map s -> A s + B it applies,
+// the maps meet in shared memory, and every segment is then run from its true start state.  All in fp32.
+constexpr int SC_CH = 16, SC_SEG = 32, SC_L = 8, SC_THREADS = SC_CH * SC_SEG;
+
+__global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float *__restrict__ zxg, uint64_t ld, uint32_t width, float *state,
+                                                                    void *out, uint64_t ldo, int out_bf16, uint32_t T) {
+  __shared__ float As[2][SC_SEG][SC_CH], Bs[2][SC_SEG][SC_CH];
+  pdl_enter();
+  const uint32_t c = threadIdx.x % SC_CH, seg = threadIdx.x / SC_CH, ch = blockIdx.x * SC_CH + c;
+  const bool live = ch < width;
+  float carry = live ? state[ch] : 0.f;
+  uint32_t buf = 0;
+  for (uint32_t t0 = 0; t0 < T; t0 += SC_SEG * SC_L, buf ^= 1) {
+    float a[SC_L], b[SC_L], g[SC_L];
+#pragma unroll
+    for (int i = 0; i < SC_L; ++i) {
+      const uint32_t t = t0 + seg * SC_L + i;
+      const bool in = live && t < T;
+      const float *row = zxg + (size_t)t * ld + ch;
+      a[i] = in ? __ldg(row) : 0.f;
+      b[i] = in ? __ldg(row + width) : 0.f;
+      g[i] = in ? __ldg(row + 2 * (size_t)width) : 0.f;
+    }
+    float A = 1.f, B = 0.f;
+#pragma unroll
+    for (int i = 0; i < SC_L; ++i) {
+      const bool in = t0 + seg * SC_L + i < T;
+      const float z = in ? sigmoid(a[i]) : 0.f;
+      b[i] = z * mingru_candidate(b[i]);
+      a[i] = 1.0f - z;
+      A *= a[i];
+      B = fmaf(a[i], B, b[i]);
+    }
+    As[buf][seg][c] = A, Bs[buf][seg][c] = B;
+    __syncthreads();
+    float s = carry, mine = carry;
+#pragma unroll 8
+    for (uint32_t k = 0; k < SC_SEG; ++k) {
+      if (k == seg) mine = s;
+      s = fmaf(As[buf][k][c], s, Bs[buf][k][c]);
+    }
+    carry = s;
+#pragma unroll
+    for (int i = 0; i < SC_L; ++i) {
+      const uint32_t t = t0 + seg * SC_L + i;
+      mine = fmaf(a[i], mine, b[i]);
+      if (live && t < T) store_out(out, out_bf16, (size_t)t * ldo + ch, mine * silu(g[i]));
+    }
+  }
+  if (live && seg == 0) state[ch] = carry;
+}
+
+__global__ void sequence_advance_kernel(cutb_sequence_state *s, const uint32_t *tokens, uint32_t n, const float *next) {
+  pdl_enter();
+  s->prev = tokens ? tokens[n - 1] : s->token;
+  if (next) s->token = (uint32_t)*next;
+  s->pos += tokens ? n : 1;
+}
+
+}  // namespace
+
+int embedding_bigram_launch(const cutb_embed_desc &d, cudaStream_t stream) {
+  CUTB_CUDA_TRY(launch_pdl(embedding_bigram_kernel, dim3(d.n), dim3(256), 0, stream, d));
+  return CUTB_OK;
+}
+
+int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) {
+  const NormStage n{d.x, d.y, d.post_w, d.pre_w, d.y ? d.x_out : nullptr, d.dim, d.groups, d.eps};
+  const uint32_t smem = 4 * norm_stage_floats(d.dim, d.groups);
+  if (smem > 48 * 1024) {
+    DeviceInfo di;
+    if (int rc = get_device_info(&di)) return rc;
+    if (smem > di.smem_optin) {
+      set_last_error("residual_norm: rows of %u elements do not fit in shared memory", d.dim);
+      return CUTB_ERR_UNSUPPORTED;
+    }
+    CUTB_CUDA_TRY(cudaFuncSetAttribute(residual_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  }
+  CUTB_CUDA_TRY(launch_pdl(residual_norm_kernel, dim3(d.rows), dim3(256), smem, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh,
+                           (int)(d.h_dtype == CUTB_BF16)));
+  return CUTB_OK;
+}
+
+int mingru_scan_launch(const float *zxg, uint64_t ld, uint32_t width, float *state, void *out, int out_dtype, uint64_t ldo, uint32_t T,
+                       cudaStream_t stream) {
+  CUTB_CUDA_TRY(launch_pdl(mingru_scan_kernel, dim3((width + SC_CH - 1) / SC_CH), dim3(SC_THREADS), 0, stream, zxg, ld, width, state, out,
+                           ldo, (int)(out_dtype == CUTB_BF16), T));
+  return CUTB_OK;
+}
+
+int sequence_advance_launch(cutb_sequence_state *s, const uint32_t *tokens, uint32_t n, const float *next, cudaStream_t stream) {
+  CUTB_CUDA_TRY(launch_pdl(sequence_advance_kernel, dim3(1), dim3(1), 0, stream, s, tokens, n, next));
+  return CUTB_OK;
+}
+
+}  // namespace cutb

@@ -427,6 +427,136 @@ CUTB_API int cutb_attention_decode(int kv_dtype, const float *q, const void *k_c
                                    uint32_t max_seq, float scale, void *workspace, uint64_t workspace_bytes, int *status,
                                    void *stream);
 
+/*
+ * Layer-list models over dense bf16 weights (a model whose configuration lists its layers, each with a mixer -- windowed
+ * attention or a gated recurrence -- and an optional feed-forward, with norms before and after each).  These entry points
+ * have no counterpart in the reference, whose runner covers llama-style GGUF models.  Element types: CUTB_F32 or CUTB_BF16
+ * wherever a *_dtype field says so; weights are always bf16, everything the recurrences, norms and softmaxes read is fp32.
+ */
+enum { CUTB_UNARY_RELU_SQUARE = 200 }; /* max(x, 0)^2, beside the unary codes of the quantized matmul */
+enum { CUTB_NO_TOKEN = 0xFFFFFFFFu };  /* `prev` of a sequence that has not started */
+enum { CUTB_DENSE_AUTO = -1, CUTB_DENSE_MATVEC = 0, CUTB_DENSE_TC = 1, CUTB_DENSE_SIMT = 2 };
+
+/*
+ * C[M, N] = unary(A[M, K] W[N, K]^T + bias), W bf16 with rows of ldw elements (a multiple of 8, zero past K, 16-byte
+ * aligned), fp32 accumulation.
+ *   CUTB_DENSE_MATVEC  one row; A fp32 or bf16, used as it is (no rounding).  Fused input: with norm_w set, A is ignored and
+ *     the row is N(x'; norm_w) of x' = res_x + N(res_y; res_norm_w) (res_y may be null: x' = res_x), N = RMS norm in
+ *     norm_groups equal parts; x' is stored to res_out when that is not null (res_out != res_x).  Fused output: with
+ *     gru_state set, W stacks three matrices (z, x, g; N / 3 rows each) and the call is one token of the recurrence
+ *     s = (1 - z) s + z c,  C[j] = s silu(g), over the fp32 states gru_state[N / 3]; C then has N / 3 elements.
+ *   CUTB_DENSE_TC      tcgen05 tensor cores, A bf16 (rows 16-byte aligned, lda % 8 == 0): prefill.
+ *   CUTB_DENSE_SIMT    fp32 fused multiply-adds, A fp32 or bf16: the true 32-bit path of a prefill.
+ * CUTB_DENSE_AUTO: one row -> mat-vec, more bf16 rows -> tensor cores, fp32 rows -> SIMT.
+ */
+typedef struct cutb_dense_desc {
+  int32_t a_dtype, c_dtype;
+  uint32_t M, K, N;
+  const void *A;
+  uint32_t lda;
+  const void *W;
+  uint32_t ldw;
+  const float *bias;
+  int32_t unary_op; /* 0 none, CUTB_UNARY_RELU_SQUARE, or a unary code of the quantized matmul */
+  void *C;
+  uint32_t ldc;
+  int32_t variant;
+  uint32_t flags; /* CUTB_FLAG_NO_OVERLAP */
+  void *workspace;
+  uint64_t workspace_bytes;
+  int *status;
+  const float *res_x, *res_y, *res_norm_w, *norm_w;
+  float *res_out;
+  uint32_t norm_groups;
+  float norm_eps;
+  float *gru_state;
+} cutb_dense_desc;
+CUTB_API int cutb_dense_select_variant(const cutb_dense_desc *desc);
+CUTB_API uint64_t cutb_dense_workspace_bytes(const cutb_dense_desc *desc);
+CUTB_API int cutb_dense_matmul(const cutb_dense_desc *desc, void *stream);
+
+/* The step between two sublayers for `rows` rows: x' = x + N(y; post_w) (y null: x' = x), h = N(x'; pre_w); x' goes to x_out
+ * (may be x; null: not kept).  row_index (device, optional): row r of h comes from row row_index[r] of x and y. */
+typedef struct cutb_residual_norm_desc {
+  const float *x, *y, *post_w, *pre_w;
+  float *x_out;
+  void *h;
+  const uint32_t *row_index;
+  uint64_t ldx, ldy, ldh;
+  uint32_t rows, dim, groups;
+  float eps;
+  int32_t h_dtype;
+} cutb_residual_norm_desc;
+CUTB_API int cutb_residual_norm(const cutb_residual_norm_desc *desc, void *stream);
+
+/* out[i, :] = embed[tokens[i]] + bigram[(previous token * mul_prev + tokens[i] * mul_cur) mod buckets]; the token before
+ * tokens[0] is *prev (device; null or CUTB_NO_TOKEN: none, which takes table row `buckets`).  bigram null: embed only.  A
+ * token past the vocabulary writes zeros and sets *status to CUTB_ERR_INVALID. */
+typedef struct cutb_embed_desc {
+  const uint32_t *tokens, *prev;
+  const void *embed, *bigram; /* bf16 tables [vocab][ld_embed], [buckets + 1][ld_bigram] */
+  float *out;
+  uint64_t ld_embed, ld_bigram, ldo;
+  uint32_t n, dim, vocab, buckets, mul_prev, mul_cur;
+  int *status;
+} cutb_embed_desc;
+CUTB_API int cutb_embedding_bigram(const cutb_embed_desc *desc, void *stream);
+
+/* The gated recurrence over T tokens: zxg [T][ld] holds the pre-activations z | x | g (width each); the fp32 states are
+ * continued and left as the last token leaves them; out [T][ldo] = s silu(g). */
+CUTB_API int cutb_mingru_scan(const float *zxg, uint64_t ld, uint32_t width, float *state, void *out, int out_dtype, uint64_t ldo,
+                              uint32_t T, void *stream);
+
+/* What a sequence carries besides caches and recurrence states, in device memory. */
+typedef struct cutb_sequence_state {
+  uint32_t token; /* the next input */
+  uint32_t prev;  /* the input before it, CUTB_NO_TOKEN at the start */
+  uint32_t pos;   /* position of `token` */
+  uint32_t reserved;
+} cutb_sequence_state;
+/* After a step: prev = the last input (tokens[n - 1], or `token` when tokens is null), pos moves on by n (1), token = the
+ * index at *next (what cutb_argreduce wrote) when next is not null. */
+CUTB_API int cutb_sequence_advance(cutb_sequence_state *state, const uint32_t *tokens, uint32_t n, const float *next, void *stream);
+
+/*
+ * Windowed attention over ring caches.  Position p lives in ring row p % ring_rows; a query at position i sees the keys
+ * j with 0 <= i - j < window, so ring_rows >= window + n_tokens - 1 keeps everything a call reads.  ring_rows is a multiple
+ * of 64.  A cache row holds n_kv_heads heads of k_head (v_head) elements, dim (vdim) of them used, k_head and v_head
+ * multiples of 8; the unused ones must be zero.  Query head h reads KV head h / (n_heads / n_kv_heads).
+ * Rotation of q and k: the first rot_dims elements of a head, tables [max_pos][rot_dims / 2]; rot_pairing 0 pairs element i
+ * with i + rot_dims / 2, 1 pairs neighbours (2 i, 2 i + 1).
+ * Values: v' = (1 - v_mix) v + v_mix v_first when v_first is given (rows of ld_first elements, one per token of this call);
+ * the mixed value is cached.  v_first_out (optional) receives this layer's own unmixed values for the layers behind it.
+ * sink: the softmax denominator has an extra 1 (a key of score 0 without a value).
+ * The first token's position is *pos_ptr (device), or pos when pos_ptr is null; positions past max_pos set *status.
+ *   cutb_window_kv_write     n_tokens roped keys and mixed values into the ring
+ *   cutb_window_attention    prefill, after the write: out [n_tokens][ldo].  bf16 caches with dim, vdim <= 128 run on the
+ *                            tensor cores (queries rounded to bf16; the weights enter the value product as two bf16 terms)
+ *   cutb_window_attention_decode  one token, both steps in one launch; n_heads / n_kv_heads and the window are not limited
+ */
+typedef struct cutb_window_attn_desc {
+  int32_t kv_dtype, out_dtype;
+  uint32_t n_heads, n_kv_heads, dim, vdim, k_head, v_head;
+  uint32_t ring_rows, window, rot_dims, max_pos;
+  int32_t rot_pairing, sink;
+  float scale, v_mix;
+  const float *cos_table, *sin_table;
+  const float *q, *k, *v; /* rows of one token are ldqkv elements apart */
+  uint64_t ldqkv;
+  void *k_cache, *v_cache;
+  const float *v_first;
+  float *v_first_out;
+  uint64_t ld_first;
+  const uint32_t *pos_ptr;
+  uint32_t pos, n_tokens;
+  void *out;
+  uint64_t ldo;
+  int *status;
+} cutb_window_attn_desc;
+CUTB_API int cutb_window_kv_write(const cutb_window_attn_desc *desc, void *stream);
+CUTB_API int cutb_window_attention(const cutb_window_attn_desc *desc, void *stream);
+CUTB_API int cutb_window_attention_decode(const cutb_window_attn_desc *desc, void *stream);
+
 CUTB_API int cutb_version(void);
 CUTB_API const char *cutb_status_string(int status);
 CUTB_API const char *cutb_last_error(void);
