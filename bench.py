@@ -1249,7 +1249,31 @@ def main() -> None:
                     help="with --decode-only: skip the prompt, fill cache rows 0..511 with synthetic values (profiling aid)")
     ap.add_argument("--exchange", choices=["fused", "nccl"], default="fused",
                     help="N > 1: slices meet through the mat-vec's own peer-store epilogue, or through an NCCL all-gather")
+    ap.add_argument("--layer-list", action="store_true",
+                    help="measure the layer-list models (kernels against their rooflines and the llama path's like kernels, prefill "
+                         "and decode throughput at equal size) on one GPU and print that (not the contract line)")
+    ap.add_argument("--layer-list-sizes", default="2048,4096", help="with --layer-list: widths of the whole-model measurement")
     args = ap.parse_args()
+    if args.layer_list:
+        import torch
+
+        if not torch.cuda.is_available():
+            raise SystemExit("bench: --layer-list needs a CUDA device (there is no CPU path)")
+        torch.cuda.set_device(0)
+        from cut_b200 import layer_bench
+
+        hbm, source = measured_peak_gbs()
+        tflops = 1590.0
+        path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+        if os.path.exists(path):
+            with open(path) as f:
+                tflops = float(json.load(f).get("bf16_tflops", tflops))
+        clocks = ClockSampler(0)
+        clocks.start()
+        res = layer_bench.measure(hbm, tflops, source, models=[x for x in args.layer_list_sizes.split(",") if x])
+        res["clocks"] = clocks.stop()
+        print(json.dumps({"layer_list": res}), flush=True)
+        return
     if args.decode_only:
         import torch
 

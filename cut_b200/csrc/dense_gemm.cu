@@ -84,73 +84,71 @@ __global__ void __launch_bounds__(DG_THREADS, 1) dense_gemm_tc_kernel(const __gr
     nk = min(p.nk_per, p.nk - k0);  // (the launcher leaves no share empty)
   };
 
+  // The copy and MMA warps run converged, with one elected lane issuing: loop variables stay warp-uniform.  A wait that runs
+  // out marks the warp dead; it then runs through its remaining steps without waiting, so that every loop ends.
   if (warp == 0) {
-    if (lane == 0) {
-      uint32_t s = 0, ph = 0, issued = 0, m0, n0, k0, nk, z;
-      const uint32_t bytes = p.a_box_rows * DG_BK * 2 + BN * DG_BK * 2;
-      bool dead = false;
-      for (uint32_t j = blockIdx.x; j < jobs && !dead; j += gridDim.x) {
-        job_of(j, m0, n0, k0, nk, z);
-        for (uint32_t ks = 0; ks < nk; ++ks) {
-          if (issued >= S && !mbar_spin_bounded(empty_u + s * 8, ph ^ 1u)) {
-            give_up();
-            dead = true;
-            break;
-          }
-          if (aborted()) {
-            dead = true;
-            break;
-          }
-          const uint32_t bar = full_u + s * 8, dst = ring_u + s * STAGE, x = (k0 + ks) * DG_BK;
+    const bool leader = elect_one();
+    uint32_t s = 0, ph = 1, m0, n0, k0, nk, z;  // (a fresh barrier lets a wait on the phase before its first pass)
+    const uint32_t bytes = p.a_box_rows * DG_BK * 2 + BN * DG_BK * 2;
+    bool dead = false;
+    for (uint32_t j = blockIdx.x; j < jobs; j += gridDim.x) {
+      job_of(j, m0, n0, k0, nk, z);
+      for (uint32_t ks = 0; ks < nk; ++ks) {
+        if (!dead && !mbar_spin_bounded(empty_u + s * 8, ph)) {
+          give_up();
+          dead = true;
+        }
+        const uint32_t bar = full_u + s * 8, dst = ring_u + s * STAGE, x = (k0 + ks) * DG_BK;
+        if (leader && !dead) {
           mbar_arrive_expect_tx(bar, bytes);
           tma_load_2d(dst, &map_a, x, m0, bar);
           tma_load_2d(dst + DG_A_BYTES, &map_w, x, n0, bar);
-          ++issued;
-          if (++s == S) s = 0, ph ^= 1u;
         }
+        if (++s == S) s = 0, ph ^= 1u;
       }
-      if (aborted()) {  // do not retire with copies still landing in shared memory
-        const uint32_t pending = issued < S ? issued : S;
-        for (uint32_t i = 0; i < pending; ++i) {
-          if (s == 0) s = S, ph ^= 1u;
-          --s;
-          mbar_wait_bounded(full_u + s * 8, ph, 1u << 10);
-        }
+    }
+    // do not retire with copies still landing in shared memory: every stage's last fill (bounded; a stage that was never
+    // filled, or whose fill the MMA warp has consumed, answers at once or runs into the small limit of an aborted launch)
+    if (aborted()) {
+      for (uint32_t i = 0; i < S; ++i) {
+        if (s == 0) s = S, ph ^= 1u;
+        --s;
+        mbar_wait_bounded(full_u + s * 8, ph ^ 1u, 1u << 8);
       }
     }
     __syncwarp();
   } else if (warp == 1) {
-    if (lane == 0) {
-      const uint64_t proto = umma_desc_sw128(0);
-      const uint32_t desc_hi = (uint32_t)(proto >> 32), lo0 = (uint32_t)proto;
-      const uint32_t idesc = umma_idesc_bf16(DG_BM, BN);
-      uint32_t s = 0, ph = 0, turn = 0, m0, n0, k0, nk, z;
-      bool dead = false;
-      for (uint32_t j = blockIdx.x; j < jobs && !dead; j += gridDim.x, ++turn) {
-        job_of(j, m0, n0, k0, nk, z);
-        const uint32_t a = turn & 1, d = tmem + a * BN;
-        if (turn >= 2 && !mbar_spin_bounded(aempty_u + a * 8, ((turn >> 1) - 1) & 1u)) {
+    const bool leader = elect_one();
+    const uint64_t proto = umma_desc_sw128(0);
+    const uint32_t desc_hi = (uint32_t)(proto >> 32), base = (uint32_t)proto + ((ring_u & 0x3FFFFu) >> 4);
+    const uint32_t idesc = umma_idesc_bf16(DG_BM, BN);
+    uint32_t s = 0, ph = 0, turn = 0, m0, n0, k0, nk, z;
+    bool dead = false;
+    for (uint32_t j = blockIdx.x; j < jobs; j += gridDim.x, ++turn) {
+      job_of(j, m0, n0, k0, nk, z);
+      const uint32_t a = turn & 1, d = tmem + a * BN;
+      if (turn >= 2 && !dead && !mbar_spin_bounded(aempty_u + a * 8, ((turn >> 1) - 1) & 1u)) {
+        give_up();
+        dead = true;
+      }
+      tc_fence_after();
+      for (uint32_t ks = 0; ks < nk; ++ks) {
+        if (!dead && !mbar_spin_bounded(full_u + s * 8, ph)) {
           give_up();
-          break;
+          dead = true;
         }
         tc_fence_after();
-        for (uint32_t ks = 0; ks < nk; ++ks) {
-          if (aborted() || !mbar_spin_bounded(full_u + s * 8, ph)) {
-            give_up();
-            dead = true;
-            break;
-          }
-          tc_fence_after();
-          const uint32_t at = lo0 + (((ring_u + s * STAGE) & 0x3FFFFu) >> 4), wt = at + (DG_A_BYTES >> 4);
+        const uint32_t at = base + s * (STAGE >> 4), wt = at + (DG_A_BYTES >> 4);
+        if (leader) {
           umma_f16(d, at, wt, desc_hi, idesc, ks != 0);
           umma_f16(d, at + 2, wt + 2, desc_hi, idesc, 1);
           umma_f16(d, at + 4, wt + 4, desc_hi, idesc, 1);
           umma_f16(d, at + 6, wt + 6, desc_hi, idesc, 1);
           umma_commit(empty_u + s * 8);
-          if (++s == S) s = 0, ph ^= 1u;
         }
-        if (!dead) umma_commit(afull_u + a * 8);
+        if (++s == S) s = 0, ph ^= 1u;
       }
+      if (leader) umma_commit(afull_u + a * 8);
     }
     __syncwarp();
   } else {
@@ -283,19 +281,21 @@ struct DgPlan {
   int bn;
   uint32_t tiles_m, tiles_n, ksplit, nk, nk_per;
 };
-// Tile width by the time of its waves (a tile's time is about proportional to its width); K split when even narrow tiles
-// leave most SMs idle.
+// Tile width by the time of its waves; K split when even narrow tiles leave most SMs idle.
 DgPlan dg_plan(const cutb_dense_desc &d, uint32_t sms) {
   DgPlan b{};
   uint64_t best = ~0ull;
   const uint32_t tm = (d.M + DG_BM - 1) / DG_BM;
-  for (int bn : {256, 128, 64}) {
+  // measured time of a wave of tiles, relative: a 64-k stage costs at least what its operands take to arrive
+  const struct { int bn; uint32_t cost; } kinds[] = {{256, 100}, {128, 66}, {64, 62}};
+  for (const auto &kind : kinds) {
+    const int bn = kind.bn;
     const uint32_t tn = (d.N + bn - 1) / bn;
-    const uint64_t cost = (uint64_t)((tm * tn + sms - 1) / sms) * (bn + 24);
+    const uint64_t cost = (uint64_t)((tm * tn + sms - 1) / sms) * kind.cost;
     if (cost < best) best = cost, b.bn = bn, b.tiles_m = tm, b.tiles_n = tn;
   }
   b.nk = (d.K + DG_BK - 1) / DG_BK;
-  if (b.tiles_m * b.tiles_n * 2 <= sms && b.nk >= 16) {  // (then the narrowest tile was chosen: widen it, K covers the SMs)
+  if (tm * ((d.N + 127) / 128) * 2 <= sms && b.nk >= 16) {
     b.bn = 128;
     b.tiles_n = (d.N + 127) / 128;
     uint32_t want = sms / (b.tiles_m * b.tiles_n);

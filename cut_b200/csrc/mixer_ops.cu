@@ -12,7 +12,7 @@ namespace {
 
 // out[i, :] = embed[token_i] + bigram[(prev_i * mul_prev + token_i * mul_cur) mod buckets]; a sequence's first token has no
 // previous one and takes row `buckets`.  One block per token.
-__global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_desc d) {
+__global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_desc d, int vec) {
   pdl_enter();
   const uint32_t i = blockIdx.x;
   uint32_t tok = __ldg(d.tokens + i);
@@ -30,10 +30,20 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_
     const uint64_t row = prev == CUTB_NO_TOKEN ? d.buckets : ((uint64_t)prev * d.mul_prev + (uint64_t)tok * d.mul_cur) % d.buckets;
     b = reinterpret_cast<const __nv_bfloat16 *>(d.bigram) + row * d.ld_bigram;
   }
+  if (vec) {  // eight elements at a time
+    for (uint32_t c = threadIdx.x; c < d.dim / 8; c += 256) {
+      const uint4 x = __ldg(reinterpret_cast<const uint4 *>(e) + c), y = b ? __ldg(reinterpret_cast<const uint4 *>(b) + c) : make_uint4(0, 0, 0, 0);
+      float4 *o = reinterpret_cast<float4 *>(out) + 2 * c;
+      o[0] = make_float4(bf16_lo(x.x) + bf16_lo(y.x), bf16_hi(x.x) + bf16_hi(y.x), bf16_lo(x.y) + bf16_lo(y.y), bf16_hi(x.y) + bf16_hi(y.y));
+      o[1] = make_float4(bf16_lo(x.z) + bf16_lo(y.z), bf16_hi(x.z) + bf16_hi(y.z), bf16_lo(x.w) + bf16_lo(y.w), bf16_hi(x.w) + bf16_hi(y.w));
+    }
+    return;
+  }
   for (uint32_t c = threadIdx.x; c < d.dim; c += 256) out[c] = __bfloat162float(e[c]) + (b ? __bfloat162float(b[c]) : 0.f);
 }
 
 // One block per row: x' = x + N(y), h = N(x') (norm_stage.cuh), h in bf16 or fp32.
+template <int IT>  // 16-byte pieces per thread of the register path; 0: any row
 __global__ void __launch_bounds__(256) residual_norm_kernel(NormStage n, uint64_t ldx, uint64_t ldy, const uint32_t *row_index, void *h,
                                                             uint64_t ldh, int h_bf16) {
   extern __shared__ __align__(16) float rn_smem[];
@@ -48,13 +58,14 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(NormStage n, uint64_
     else *reinterpret_cast<float4 *>(reinterpret_cast<float *>(h) + base + i) = v;
   };
   auto put1 = [&](uint32_t i, float v) { store_out(h, h_bf16, base + i, v); };
-  stage_norm(n, rn_smem, n.x_out != nullptr, put4, put1);
+  if constexpr (IT > 0) stage_norm_regs<IT>(n, rn_smem, nullptr, n.x_out != nullptr, put4);
+  else stage_norm(n, rn_smem, n.x_out != nullptr, put4, put1);
 }
 
 // The recurrence over T tokens.  A block owns SC_CH channels; SC_SEG groups of threads take consecutive segments of SC_L
 // tokens each, so a turn covers SC_SEG * SC_L tokens.  A segment is first reduced to the affine map s -> A s + B it applies,
 // the maps meet in shared memory, and every segment is then run from its true start state.  All in fp32.
-constexpr int SC_CH = 16, SC_SEG = 32, SC_L = 8, SC_THREADS = SC_CH * SC_SEG;
+constexpr int SC_CH = 16, SC_SEG = 32, SC_L = 4, SC_THREADS = SC_CH * SC_SEG;
 
 __global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float *__restrict__ zxg, uint64_t ld, uint32_t width, float *state,
                                                                     void *out, uint64_t ldo, int out_bf16, uint32_t T) {
@@ -64,18 +75,25 @@ __global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float 
   const bool live = ch < width;
   float carry = live ? state[ch] : 0.f;
   uint32_t buf = 0;
-  for (uint32_t t0 = 0; t0 < T; t0 += SC_SEG * SC_L, buf ^= 1) {
-    float a[SC_L], b[SC_L], g[SC_L];
+  float z1[SC_L], u1[SC_L], g1[SC_L];  // the next turn's pre-activations, in flight
+  auto load = [&](uint32_t t0) {
 #pragma unroll
     for (int i = 0; i < SC_L; ++i) {
       const uint32_t t = t0 + seg * SC_L + i;
       const bool in = live && t < T;
       const float *row = zxg + (size_t)t * ld + ch;
-      a[i] = in ? __ldg(row) : 0.f;
-      b[i] = in ? __ldg(row + width) : 0.f;
-      g[i] = in ? __ldg(row + 2 * (size_t)width) : 0.f;
+      z1[i] = in ? __ldg(row) : 0.f;
+      u1[i] = in ? __ldg(row + width) : 0.f;
+      g1[i] = in ? __ldg(row + 2 * (size_t)width) : 0.f;
     }
+  };
+  load(0);
+  for (uint32_t t0 = 0; t0 < T; t0 += SC_SEG * SC_L, buf ^= 1) {
+    float a[SC_L], b[SC_L], g[SC_L];
     float A = 1.f, B = 0.f;
+#pragma unroll
+    for (int i = 0; i < SC_L; ++i) a[i] = z1[i], b[i] = u1[i], g[i] = g1[i];
+    load(t0 + SC_SEG * SC_L);
 #pragma unroll
     for (int i = 0; i < SC_L; ++i) {
       const bool in = t0 + seg * SC_L + i < T;
@@ -114,12 +132,25 @@ __global__ void sequence_advance_kernel(cutb_sequence_state *s, const uint32_t *
 }  // namespace
 
 int embedding_bigram_launch(const cutb_embed_desc &d, cudaStream_t stream) {
-  CUTB_CUDA_TRY(launch_pdl(embedding_bigram_kernel, dim3(d.n), dim3(256), 0, stream, d));
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(d.embed) | reinterpret_cast<uintptr_t>(d.bigram) | reinterpret_cast<uintptr_t>(d.out);
+  const int vec = (d.dim | d.ld_embed | d.ld_bigram | d.ldo) % 8 == 0 && bases % 16 == 0;
+  CUTB_CUDA_TRY(launch_pdl(embedding_bigram_kernel, dim3(d.n), dim3(256), 0, stream, d, vec));
   return CUTB_OK;
 }
 
 int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) {
   const NormStage n{d.x, d.y, d.post_w, d.pre_w, d.y ? d.x_out : nullptr, d.dim, d.groups, d.eps};
+  const int bf16 = d.h_dtype == CUTB_BF16;
+  if (norm_stage_fits(d.dim, d.groups, 256, 8)) {  // the row stays in registers
+    const uint32_t small = 4 * (d.dim / 64);
+    auto go = [&](auto kernel) -> cudaError_t {
+      return launch_pdl(kernel, dim3(d.rows), dim3(256), small, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16);
+    };
+    if (d.dim <= 2048) CUTB_CUDA_TRY(go(residual_norm_kernel<2>));
+    else if (d.dim <= 4096) CUTB_CUDA_TRY(go(residual_norm_kernel<4>));
+    else CUTB_CUDA_TRY(go(residual_norm_kernel<8>));
+    return CUTB_OK;
+  }
   const uint32_t smem = 4 * norm_stage_floats(d.dim, d.groups);
   if (smem > 48 * 1024) {
     DeviceInfo di;
@@ -128,10 +159,9 @@ int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) 
       set_last_error("residual_norm: rows of %u elements do not fit in shared memory", d.dim);
       return CUTB_ERR_UNSUPPORTED;
     }
-    CUTB_CUDA_TRY(cudaFuncSetAttribute(residual_norm_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CUTB_CUDA_TRY(cudaFuncSetAttribute(residual_norm_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   }
-  CUTB_CUDA_TRY(launch_pdl(residual_norm_kernel, dim3(d.rows), dim3(256), smem, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh,
-                           (int)(d.h_dtype == CUTB_BF16)));
+  CUTB_CUDA_TRY(launch_pdl(residual_norm_kernel<0>, dim3(d.rows), dim3(256), smem, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16));
   return CUTB_OK;
 }
 

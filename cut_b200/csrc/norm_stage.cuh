@@ -18,8 +18,8 @@ struct NormStage {
   float eps;
 };
 
-// floats of shared memory stage_norm needs: two rows, a partial sum per warp, a factor per group
-__host__ __device__ inline uint32_t norm_stage_floats(uint32_t dim, uint32_t groups) { return 2 * ((dim + 3) / 4 * 4) + 32 + groups; }
+// floats of shared memory a stage may need: two rows, a partial sum per warp, a factor per group, two sums per 128 elements
+__host__ __device__ inline uint32_t norm_stage_floats(uint32_t dim, uint32_t groups) { return 2 * ((dim + 3) / 4 * 4) + 32 + (groups + 3) / 4 * 4 + dim / 64; }
 
 // inv[g] = 1 / sqrt(mean of row[part g]^2 + eps); part = 32 floats of scratch.  Fixed summation order.
 __device__ __forceinline__ void group_factors(const float *row, uint32_t dim, uint32_t groups, float eps, float *part, float *inv) {
@@ -51,6 +51,73 @@ __device__ __forceinline__ void group_factors(const float *row, uint32_t dim, ui
     }
   }
   __syncthreads();
+}
+
+// Fast path for rows whose groups are whole multiples of 128 elements and which the block holds in registers (IT 16-byte pieces
+// per thread): a warp's piece of 128 elements lies in one group, its sum of squares is one entry of `part`, and every warp adds
+// up its own group's entries.  Two barriers in all.  `norms` (optional): post_w then pre_w in shared
+// memory, copied there by this block's own cp.async.
+template <int IT, class Store4>
+__device__ __forceinline__ void stage_norm_regs(const NormStage &n, float *part, const float *norms, bool write_x, Store4 store4) {
+  const uint32_t tid = threadIdx.x, lane = tid & 31, nt = blockDim.x, d4 = n.dim / 4, chunks = n.dim / 128, per = chunks / n.groups;
+  const float inv_gs = 1.0f / (float)(n.dim / n.groups);
+  float4 x[IT], y[IT];
+#pragma unroll
+  for (int it = 0; it < IT; ++it) {
+    const uint32_t i = tid + it * nt;
+    x[it] = i < d4 ? reinterpret_cast<const float4 *>(n.x)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    y[it] = n.y && i < d4 ? reinterpret_cast<const float4 *>(n.y)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  if (norms) asm volatile("cp.async.wait_all;" ::: "memory");  // (this thread's pieces; a barrier lies before their use)
+  auto factors = [&](const float4 (&v)[IT], float *buf, float (&f)[IT]) {
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      float s = fmaf(v[it].x, v[it].x, fmaf(v[it].y, v[it].y, fmaf(v[it].z, v[it].z, v[it].w * v[it].w)));
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      const uint32_t c = (tid + it * nt) / 32;
+      if (lane == 0 && c < chunks) buf[c] = s;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      const uint32_t c = (tid + it * nt) / 32, g0 = c / per * per;
+      float s = 0.f;
+      if (c < chunks)
+        for (uint32_t k = lane; k < per; k += 32) s += buf[g0 + k];
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      f[it] = 1.0f / sqrtf(s * inv_gs + n.eps);
+    }
+  };
+  float f[IT];
+  if (n.y) {
+    factors(y, part, f);
+    const float4 *w4 = reinterpret_cast<const float4 *>(norms ? norms : n.post_w);
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      const uint32_t i = tid + it * nt;
+      if (i < d4) {
+        const float4 w = w4[i];
+        x[it].x = fmaf(y[it].x * f[it], w.x, x[it].x), x[it].y = fmaf(y[it].y * f[it], w.y, x[it].y);
+        x[it].z = fmaf(y[it].z * f[it], w.z, x[it].z), x[it].w = fmaf(y[it].w * f[it], w.w, x[it].w);
+        if (write_x) reinterpret_cast<float4 *>(n.x_out)[i] = x[it];
+      }
+    }
+  }
+  factors(x, part + chunks, f);
+  const float4 *w4 = reinterpret_cast<const float4 *>(norms ? norms + n.dim : n.pre_w);
+#pragma unroll
+  for (int it = 0; it < IT; ++it) {
+    const uint32_t i = tid + it * nt;
+    if (i < d4) {
+      const float4 w = w4[i];
+      store4(4 * i, make_float4(x[it].x * f[it] * w.x, x[it].y * f[it] * w.y, x[it].z * f[it] * w.z, x[it].w * f[it] * w.w));
+    }
+  }
+}
+__host__ __device__ inline bool norm_stage_fits(uint32_t dim, uint32_t groups, uint32_t threads, int it) {
+  return dim % groups == 0 && dim / groups % 128 == 0 && dim <= threads * 4 * (uint32_t)it;
 }
 
 // Runs on all threads of the block; `smem` holds norm_stage_floats() floats.  store4(i, h[i .. i+3]) is called for every i

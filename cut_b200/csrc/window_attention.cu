@@ -63,6 +63,21 @@ __device__ __forceinline__ float rotated(const float *x, uint32_t e, uint32_t po
   return second ? v * c + o * s : v * c - o * s;
 }
 
+// Elements of a head two at a time: pair i < rot_dims / 2 is rotated, the others are (2 i, 2 i + 1) as they are.
+struct Pair {
+  uint32_t e0, e1;
+  float x0, x1, c, s;
+};
+__device__ __forceinline__ Pair load_pair(const float *x, uint32_t i, uint32_t pos, const cutb_window_attn_desc &d) {
+  Pair r;
+  const uint32_t half = d.rot_dims / 2;
+  const bool rot = i < half;
+  r.e0 = d.rot_pairing || !rot ? 2 * i : i, r.e1 = d.rot_pairing || !rot ? 2 * i + 1 : i + half;
+  r.x0 = r.e0 < d.dim ? __ldg(x + r.e0) : 0.f, r.x1 = r.e1 < d.dim ? __ldg(x + r.e1) : 0.f;
+  r.c = rot ? __ldg(d.cos_table + (size_t)pos * half + i) : 1.f, r.s = rot ? __ldg(d.sin_table + (size_t)pos * half + i) : 0.f;
+  return r;
+}
+
 __device__ __forceinline__ float mixed_value(const cutb_window_attn_desc &d, uint32_t tok, uint32_t i) {
   const float v = d.v[tok * d.ldqkv + i];
   if (d.v_first_out) d.v_first_out[tok * d.ld_first + i] = v;
@@ -79,9 +94,13 @@ template <typename KV> __global__ void __launch_bounds__(256) window_kv_write_ke
   const size_t row = pos % d.ring_rows;
   KV *kc = reinterpret_cast<KV *>(d.k_cache) + row * d.n_kv_heads * d.k_head;
   KV *vc = reinterpret_cast<KV *>(d.v_cache) + row * d.n_kv_heads * d.v_head;
-  for (uint32_t i = threadIdx.x; i < d.n_kv_heads * d.dim; i += 256) {
-    const uint32_t g = i / d.dim, e = i % d.dim;
-    kv_put(kc + g * d.k_head + e, rotated(d.k + tok * d.ldqkv + g * d.dim, e, pos, d));
+  const uint32_t pairs = d.k_head / 2;
+  for (uint32_t i = threadIdx.x; i < d.n_kv_heads * pairs; i += 256) {
+    const uint32_t g = i / pairs;
+    const Pair x = load_pair(d.k + tok * d.ldqkv + g * d.dim, i - g * pairs, pos, d);  // (zeros past the head's elements)
+    KV *dst = kc + g * d.k_head;
+    kv_put(dst + x.e0, x.x0 * x.c - x.x1 * x.s);
+    kv_put(dst + x.e1, x.x1 * x.c + x.x0 * x.s);
   }
   for (uint32_t i = threadIdx.x; i < d.n_kv_heads * d.vdim; i += 256) kv_put(vc + i / d.vdim * d.v_head + i % d.vdim, mixed_value(d, tok, i));
 }
@@ -103,7 +122,8 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t &r0, uint3
                : "r"(addr));
 }
 __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+  // (not volatile: a pure function of its registers, free to move between the loads of the next fragments)
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -137,20 +157,30 @@ template <int DK, int DV> __global__ void __launch_bounds__(WT_THREADS) window_a
   const size_t kld = (size_t)G * d.k_head, vld = (size_t)G * d.v_head;
   // Keys nobody in the block sees are zero (a weight of zero times a stray NaN would not be); columns past the head's
   // elements are zeroed once and never written again.
+  constexpr uint32_t KC = DK / 8, VC = DV / 8, KR = WT_THREADS / KC, VR = WT_THREADS / VC;  // 16-byte pieces per row, rows per pass
+  const uint32_t kr0 = tid / KC, kc = tid % KC, vr0 = tid / VC, vc = tid % VC;
+  const bool k_live = kc * 8 < d.k_head, v_live = vc * 8 < d.v_head;
   auto load_tile = [&](uint32_t t, uint32_t buf) {
     const uint32_t ring0 = (t * WT_BN) % d.ring_rows;
-    for (uint32_t i = tid; i < WT_BN * (DK / 8); i += WT_THREADS) {
-      const uint32_t r = i / (DK / 8), c = i % (DK / 8), key = t * WT_BN + r, off = (r * LK + c * 8) * 2;
-      if (c * 8 < d.k_head) {
-        if (key >= key_lo && key <= p_last) cp_async16(k_u + buf * KT + off, kbase + (ring0 + r) * kld + c * 8);
-        else *reinterpret_cast<uint4 *>(wt_smem + (k_u - qs_u) + buf * KT + off) = make_uint4(0, 0, 0, 0);
+    const bool whole = t * WT_BN >= key_lo && t * WT_BN + WT_BN - 1 <= p_last;
+    if (k_live) {
+      const __nv_bfloat16 *src = kbase + (ring0 + kr0) * kld + kc * 8;
+      const uint32_t off = buf * KT + (kr0 * LK + kc * 8) * 2;
+#pragma unroll
+      for (uint32_t j = 0; j < WT_BN / KR; ++j, src += KR * kld) {
+        const uint32_t key = t * WT_BN + kr0 + j * KR;
+        if (whole || (key >= key_lo && key <= p_last)) cp_async16(k_u + off + j * KR * LK * 2, src);
+        else *reinterpret_cast<uint4 *>(wt_smem + (k_u - qs_u) + off + j * KR * LK * 2) = make_uint4(0, 0, 0, 0);
       }
     }
-    for (uint32_t i = tid; i < WT_BN * (DV / 8); i += WT_THREADS) {
-      const uint32_t r = i / (DV / 8), c = i % (DV / 8), key = t * WT_BN + r, off = (r * LV + c * 8) * 2;
-      if (c * 8 < d.v_head) {
-        if (key >= key_lo && key <= p_last) cp_async16(v_u + buf * VT + off, vbase + (ring0 + r) * vld + c * 8);
-        else *reinterpret_cast<uint4 *>(wt_smem + (v_u - qs_u) + buf * VT + off) = make_uint4(0, 0, 0, 0);
+    if (v_live) {
+      const __nv_bfloat16 *src = vbase + (ring0 + vr0) * vld + vc * 8;
+      const uint32_t off = buf * VT + (vr0 * LV + vc * 8) * 2;
+#pragma unroll
+      for (uint32_t j = 0; j < WT_BN / VR; ++j, src += VR * vld) {
+        const uint32_t key = t * WT_BN + vr0 + j * VR;
+        if (whole || (key >= key_lo && key <= p_last)) cp_async16(v_u + off + j * VR * LV * 2, src);
+        else *reinterpret_cast<uint4 *>(wt_smem + (v_u - qs_u) + off + j * VR * LV * 2) = make_uint4(0, 0, 0, 0);
       }
     }
     cp_async_commit();
@@ -165,10 +195,26 @@ template <int DK, int DV> __global__ void __launch_bounds__(WT_THREADS) window_a
         *reinterpret_cast<uint4 *>(wt_smem + (v_u - qs_u) + (i / (DV / 8) * LV + i % (DV / 8) * 8) * 2) = make_uint4(0, 0, 0, 0);
   load_tile(t_first, 0);
 
-  for (uint32_t i = tid; i < WT_BM * DK; i += WT_THREADS) {
-    const uint32_t r = i / DK, e = i % DK;
-    const float v = r < ntok && e < d.dim ? rotated(d.q + (size_t)(tok0 + r) * d.ldqkv + (size_t)h * d.dim, e, p0 + r, d) : 0.f;
-    Qs[r * LK + e] = __float2bfloat16_rn(v);
+  // queries: rotated at their own positions, rounded to bf16; eight pairs in flight per thread
+  {
+    constexpr uint32_t PP = DK / 2, QU = 8;  // pairs per row
+    const uint32_t pi = tid % PP, rr = tid / PP;
+    const float *q0 = d.q + (size_t)tok0 * d.ldqkv + (size_t)h * d.dim;
+    for (uint32_t r0 = rr; r0 < WT_BM; r0 += QU * (WT_THREADS / PP)) {
+      Pair pr[QU];
+#pragma unroll
+      for (uint32_t u = 0; u < QU; ++u) {
+        const uint32_t r = r0 + u * (WT_THREADS / PP), rc = min(r, ntok - 1);  // (rows past the last token repeat it)
+        pr[u] = load_pair(q0 + rc * d.ldqkv, pi, p0 + rc, d);
+      }
+#pragma unroll
+      for (uint32_t u = 0; u < QU; ++u) {
+        const uint32_t r = r0 + u * (WT_THREADS / PP);
+        const Pair &x = pr[u];
+        Qs[r * LK + x.e0] = __float2bfloat16_rn(x.x0 * x.c - x.x1 * x.s);
+        Qs[r * LK + x.e1] = __float2bfloat16_rn(x.x1 * x.c + x.x0 * x.s);
+      }
+    }
   }
   __syncthreads();
 
@@ -379,6 +425,7 @@ template <typename KV, int RG> __global__ void __launch_bounds__(WD_THREADS) win
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, split = blockIdx.y, S = gridDim.y, G = d.n_kv_heads;
   const uint32_t rep = d.n_heads / G, ngrp = (rep + RG - 1) / RG, kvh = blockIdx.x / ngrp, grp = blockIdx.x % ngrp;
   const uint32_t h0 = kvh * rep + grp * RG, nr = min((uint32_t)RG, rep - grp * RG);
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");  // (a mat-vec behind this starts its weight stream)
   pdl_enter();
   const uint32_t pos = d.pos_ptr ? *d.pos_ptr : d.pos;
   if (pos >= d.max_pos) {  // (the same in every block of the cluster)
@@ -388,10 +435,60 @@ template <typename KV, int RG> __global__ void __launch_bounds__(WD_THREADS) win
   const KV *kb = reinterpret_cast<const KV *>(d.k_cache) + (size_t)kvh * d.k_head;
   const KV *vb = reinterpret_cast<const KV *>(d.v_cache) + (size_t)kvh * d.v_head;
   const size_t kld = (size_t)G * d.k_head, vld = (size_t)G * d.v_head;
+  // lanes per cache row: eight elements each
+  uint32_t lpk = 1, lpv = 1;
+  while (lpk * 8 < d.k_head) lpk *= 2;
+  while (lpv * 8 < d.v_head) lpv *= 2;
+  const uint32_t ke = lane % lpk * 8, ksub = lane / lpk, kpw = 32 / lpk;  // element, key within a pass, keys per warp and pass
+  const uint32_t ve = lane % lpv * 8, vsub = lane / lpv, vpw = 32 / lpv;
+  // keys before this token, dealt to the slices
+  const uint32_t n_old = min(d.window - 1, pos), per = (n_old + S - 1) / S;
+  const uint32_t s0 = min(split * per, n_old), s1 = min(s0 + per, n_old), row0 = (pos - n_old) % d.ring_rows;
+  constexpr int U = 4;  // passes in flight
+  auto load_k = [&](Raw (&raw)[U], uint32_t c0, uint32_t i0, uint32_t cnt) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t i = i0 + u * WD_WARPS * kpw + ksub;
+      uint32_t row = row0 + c0 + i;
+      if (row >= d.ring_rows) row -= d.ring_rows;
+      if (i < cnt && ke < d.k_head) raw[u] = kv_raw8(kb + (size_t)row * kld + ke);
+      else kv_zero8(raw[u]);
+    }
+  };
+  auto load_v = [&](Raw (&raw)[U], uint32_t c0, uint32_t i0, uint32_t cnt) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const uint32_t i = i0 + u * WD_WARPS * vpw + vsub;
+      uint32_t row = row0 + c0 + i;
+      if (row >= d.ring_rows) row -= d.ring_rows;
+      if (i < cnt && ve < d.v_head) raw[u] = kv_raw8(vb + (size_t)row * vld + ve);
+      else kv_zero8(raw[u]);
+    }
+  };
+  // the first keys and values are on their way while the queries are rotated
+  Raw kr0[U], vr0[U];
+  const uint32_t cnt0 = min((uint32_t)WD_CHUNK, s1 - s0);
+  load_k(kr0, s0, warp * kpw, cnt0);
+  load_v(vr0, s0, warp * vpw, cnt0);
 
-  for (uint32_t i = tid; i < RG * d.k_head; i += WD_THREADS) {
-    const uint32_t r = i / d.k_head, e = i % d.k_head;
-    qs[r][e] = r < nr && e < d.dim ? rotated(d.q + (size_t)(h0 + r) * d.dim, e, pos, d) * d.scale : 0.f;
+  {  // pairs of the query heads, 32 lanes along a head
+    const uint32_t pairs = d.k_head / 2;
+#pragma unroll
+    for (uint32_t r = 0; r < RG; ++r)
+      if (r % WD_WARPS == warp || RG < WD_WARPS) {
+        // fewer heads than warps: the warps of a head share its pairs
+        constexpr uint32_t SH = RG < WD_WARPS ? WD_WARPS / RG : 1;
+        if (RG < WD_WARPS && warp / SH != r) continue;
+        for (uint32_t i = (RG < WD_WARPS ? warp % SH : 0) * 32 + lane; i < pairs; i += 32 * SH) {
+          if (r < nr) {
+            const Pair x = load_pair(d.q + (size_t)(h0 + r) * d.dim, i, pos, d);
+            qs[r][x.e0] = (x.x0 * x.c - x.x1 * x.s) * d.scale;
+            qs[r][x.e1] = (x.x1 * x.c + x.x0 * x.s) * d.scale;
+          } else {
+            qs[r][2 * i] = qs[r][2 * i + 1] = 0.f;
+          }
+        }
+      }
   }
   if (split == 0) {  // this token's key and value, rounded as the cache holds them
     const bool store = grp == 0;
@@ -408,51 +505,29 @@ template <typename KV, int RG> __global__ void __launch_bounds__(WD_THREADS) win
       if (store && e < d.vdim) kv_put(vw + e, v);
     }
   }
+  if (tid < RG) head_m[tid] = WA_NEG, head_l[tid] = 0.f, p_new[tid] = 0.f;
   __syncthreads();
-  for (uint32_t r = warp; r < RG; r += WD_WARPS) {
-    float m = WA_NEG, l = 0.f, p = 0.f;
-    if (split == 0) {
-      float s = 0.f;
-      for (uint32_t e = lane; e < d.k_head; e += 32) s = fmaf(qs[r][e], kn[e], s);
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-      m = d.sink ? fmaxf(s, 0.f) : s;
-      p = expf(s - m);
-      l = p + (d.sink ? expf(-m) : 0.f);
-    }
-    if (lane == 0) head_m[r] = m, head_l[r] = l, p_new[r] = p;
-  }
-  // lanes per cache row: eight elements each
-  uint32_t lpk = 1, lpv = 1;
-  while (lpk * 8 < d.k_head) lpk *= 2;
-  while (lpv * 8 < d.v_head) lpv *= 2;
-  const uint32_t ke = lane % lpk * 8, ksub = lane / lpk, kpw = 32 / lpk;  // element, key within a pass, keys per warp and pass
-  const uint32_t ve = lane % lpv * 8, vsub = lane / lpv, vpw = 32 / lpv;
   float qr[RG][8];
 #pragma unroll
   for (int r = 0; r < RG; ++r)
 #pragma unroll
     for (int j = 0; j < 8; ++j) qr[r][j] = ke < d.k_head ? qs[r][ke + j] : 0.f;
-  __syncthreads();
   float acc[RG][8];
 #pragma unroll
   for (int r = 0; r < RG; ++r)
 #pragma unroll
-    for (int j = 0; j < 8; ++j) acc[r][j] = split == 0 && warp == 0 && vsub == 0 && ve < d.v_head ? p_new[r] * vn[ve + j] : 0.f;
+    for (int j = 0; j < 8; ++j) acc[r][j] = 0.f;
 
-  // keys before this token, dealt to the slices
-  const uint32_t n_old = min(d.window - 1, pos), per = (n_old + S - 1) / S;
-  const uint32_t s0 = min(split * per, n_old), s1 = min(s0 + per, n_old), first = pos - n_old;
-  for (uint32_t c0 = s0; c0 < s1; c0 += WD_CHUNK) {
-    const uint32_t cnt = min((uint32_t)WD_CHUNK, s1 - c0), base = first + c0;
-    constexpr int U = 4;
+  // (the first slice has the new key to add even when there are no others)
+  for (uint32_t c0 = s0; c0 < s1 || (c0 == s0 && split == 0); c0 += WD_CHUNK) {
+    const uint32_t cnt = min((uint32_t)WD_CHUNK, s1 - c0);
     for (uint32_t i0 = warp * kpw; i0 < cnt; i0 += WD_WARPS * kpw * U) {
       Raw raw[U];
+      if (c0 == s0 && i0 == warp * kpw) {
 #pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const uint32_t i = i0 + u * WD_WARPS * kpw + ksub;
-        if (i < cnt && ke < d.k_head) raw[u] = kv_raw8(kb + (size_t)((base + i) % d.ring_rows) * kld + ke);
-        else kv_zero8(raw[u]);
+        for (int u = 0; u < U; ++u) raw[u] = kr0[u];
+      } else {
+        load_k(raw, c0, i0, cnt);
       }
 #pragma unroll
       for (int u = 0; u < U; ++u) {
@@ -464,22 +539,27 @@ template <typename KV, int RG> __global__ void __launch_bounds__(WD_THREADS) win
           dot[r] = 0.f;
 #pragma unroll
           for (int j = 0; j < 8; ++j) dot[r] = fmaf(qr[r][j], kv[j], dot[r]);
-          for (uint32_t o = lpk >> 1; o > 0; o >>= 1) dot[r] += __shfl_xor_sync(0xffffffffu, dot[r], o);
-          if (i < cnt && ke == 0) sc[r][i] = dot[r];
+        }
+        for (uint32_t o = lpk >> 1; o > 0; o >>= 1)
+#pragma unroll
+          for (int r = 0; r < RG; ++r) dot[r] += __shfl_xor_sync(0xffffffffu, dot[r], o);
+        if (i < cnt && ke == 0) {
+#pragma unroll
+          for (int r = 0; r < RG; ++r) sc[r][i] = dot[r];
         }
       }
     }
-    // the values of the first passes are on their way while the softmax runs
-    Raw vr0[U];
-#pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const uint32_t i = warp * vpw + u * WD_WARPS * vpw + vsub;
-      if (i < cnt && ve < d.v_head) vr0[u] = kv_raw8(vb + (size_t)((base + i) % d.ring_rows) * vld + ve);
-      else kv_zero8(vr0[u]);
-    }
+    if (c0 != s0) load_v(vr0, c0, warp * vpw, cnt);  // on their way while the softmax runs
     __syncthreads();
     for (uint32_t r = warp; r < RG; r += WD_WARPS) {
-      float m = head_m[r];
+      const bool fresh = c0 == s0 && split == 0;  // the new token's key, and the sink as a key of score 0
+      float m = head_m[r], s_new = 0.f;
+      if (fresh) {
+        for (uint32_t e = lane; e < d.k_head; e += 32) s_new = fmaf(qs[r][e], kn[e], s_new);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) s_new += __shfl_xor_sync(0xffffffffu, s_new, o);
+        m = d.sink ? fmaxf(s_new, 0.f) : s_new;
+      }
       for (uint32_t i = lane; i < cnt; i += 32) m = fmaxf(m, sc[r][i]);
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
@@ -493,21 +573,34 @@ template <typename KV, int RG> __global__ void __launch_bounds__(WD_THREADS) win
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
       __syncwarp();
-      if (lane == 0) head_l[r] = fmaf(head_l[r], f, l), head_m[r] = m, fac[r] = f;
+      if (lane == 0) {
+        if (fresh) {
+          const float p = expf(s_new - m);
+          p_new[r] = p;
+          l += p + (d.sink ? expf(-m) : 0.f);
+        }
+        head_l[r] = fmaf(head_l[r], f, l), head_m[r] = m, fac[r] = f;
+      }
     }
     __syncthreads();
+    if (c0 != s0) {
 #pragma unroll
-    for (int r = 0; r < RG; ++r)
+      for (int r = 0; r < RG; ++r)
 #pragma unroll
-      for (int j = 0; j < 8; ++j) acc[r][j] *= fac[r];
+        for (int j = 0; j < 8; ++j) acc[r][j] *= fac[r];
+    } else if (split == 0 && warp == 0 && vsub == 0 && ve < d.v_head) {
+#pragma unroll
+      for (int r = 0; r < RG; ++r)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[r][j] = p_new[r] * vn[ve + j];
+    }
     for (uint32_t i0 = warp * vpw; i0 < cnt; i0 += WD_WARPS * vpw * U) {
       Raw raw[U];
+      if (i0 == warp * vpw) {
 #pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const uint32_t i = i0 + u * WD_WARPS * vpw + vsub;
-        if (i0 == warp * vpw) raw[u] = vr0[u];
-        else if (i < cnt && ve < d.v_head) raw[u] = kv_raw8(vb + (size_t)((base + i) % d.ring_rows) * vld + ve);
-        else kv_zero8(raw[u]);
+        for (int u = 0; u < U; ++u) raw[u] = vr0[u];
+      } else {
+        load_v(raw, c0, i0, cnt);
       }
 #pragma unroll
       for (int u = 0; u < U; ++u) {
@@ -545,14 +638,24 @@ template <typename KV, int RG> __global__ void __launch_bounds__(WD_THREADS) win
   cluster.sync();
   for (uint32_t i = split * WD_THREADS + tid; i < nr * d.vdim; i += S * WD_THREADS) {
     const uint32_t r = i / d.vdim, e = i % d.vdim;
-    float m = WA_NEG;
-    for (uint32_t k = 0; k < S; ++k) m = fmaxf(m, *cluster.map_shared_rank(&head_m[r], k));
-    float l = 0.f, s = 0.f;
-    for (uint32_t k = 0; k < S; ++k) {
-      const float w = expf(*cluster.map_shared_rank(&head_m[r], k) - m);
-      l = fmaf(w, *cluster.map_shared_rank(&head_l[r], k), l);
-      s = fmaf(w, *cluster.map_shared_rank(&pacc[r][e], k), s);
+    float mk[WD_MAX_SPLITS], lk[WD_MAX_SPLITS], ak[WD_MAX_SPLITS], m = WA_NEG, l = 0.f, s = 0.f;
+#pragma unroll
+    for (uint32_t k = 0; k < WD_MAX_SPLITS; ++k) {  // every remote read in flight at once
+      const uint32_t from = k < S ? k : 0;
+      mk[k] = *cluster.map_shared_rank(&head_m[r], from);
+      lk[k] = *cluster.map_shared_rank(&head_l[r], from);
+      ak[k] = *cluster.map_shared_rank(&pacc[r][e], from);
     }
+#pragma unroll
+    for (uint32_t k = 0; k < WD_MAX_SPLITS; ++k)
+      if (k < S) m = fmaxf(m, mk[k]);
+#pragma unroll
+    for (uint32_t k = 0; k < WD_MAX_SPLITS; ++k)
+      if (k < S) {
+        const float w = expf(mk[k] - m);
+        l = fmaf(w, lk[k], l);
+        s = fmaf(w, ak[k], s);
+      }
     store_out(d.out, d.out_dtype == CUTB_BF16, (size_t)(h0 + r) * d.vdim + e, s / l);
   }
   cluster.sync();  // nobody leaves while its shared memory may still be read
@@ -589,12 +692,13 @@ template <typename KV, int RG> int wd_launch(const cutb_window_attn_desc &d, cud
   CUTB_CUDA_TRY(cudaLaunchKernelEx(&cfg, window_attention_decode_kernel<KV, RG>, d));
   return CUTB_OK;
 }
+// Query heads per block: one as long as the blocks fit the GPU twice over (keys and values then come from L2 once per head;
+// the kernel is bound by latency, not by bytes), more for models with many heads.
 template <typename KV> int wd_dispatch(const cutb_window_attn_desc &d, cudaStream_t stream) {
   const uint32_t rep = d.n_heads / d.n_kv_heads;
-  if (rep == 1) return wd_launch<KV, 1>(d, stream);
-  if (rep == 2) return wd_launch<KV, 2>(d, stream);
-  if (rep <= 4) return wd_launch<KV, 4>(d, stream);
-  return wd_launch<KV, 8>(d, stream);
+  if (rep == 1 || d.n_heads <= 48) return wd_launch<KV, 1>(d, stream);
+  if (rep == 2 || d.n_heads <= 96) return wd_launch<KV, 2>(d, stream);
+  return wd_launch<KV, 4>(d, stream);
 }
 
 }  // namespace

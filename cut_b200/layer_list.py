@@ -22,6 +22,7 @@ import numpy as np
 import torch
 
 from . import _lib as L
+from . import ops
 from .decoding import RecordedStep
 
 
@@ -191,7 +192,7 @@ class LayerListDecoder:
         L.lib()
         self.cfg, self.dev = cfg, torch.device(device)
         self.half = dtype == "bfloat16"
-        self.act_t, self.act_code = (torch.bfloat16, L.BF16) if self.half else (torch.float32, L.F32)
+        self.act_t = torch.bfloat16 if self.half else torch.float32
         self.max_seq = max(1, int(max_seq))
         self.max_portion = max(1, min(int(max_portion), self.max_seq))
         self.ldx = pad(cfg.width, 8)
@@ -293,21 +294,12 @@ class LayerListDecoder:
         self.launches += 1
         L.check(getattr(L.lib(), name)(C.byref(d), self._stream()))
 
-    def _dense_desc(self, lin: Linear, M: int, a, c, a_code: int, c_code: int, unary: int = 0):
-        d = L.DenseDesc()
-        d.a_dtype, d.c_dtype, d.M, d.K, d.N = a_code, c_code, M, lin.K, lin.N
-        if a is not None:
-            d.A, d.lda = a.data_ptr(), a.stride(0)
-        d.W, d.ldw = lin.w.data_ptr(), lin.ldw
-        d.bias = lin.bias.data_ptr() if lin.bias is not None else None
-        d.unary_op, d.C, d.ldc = unary, c.data_ptr(), c.stride(0)
-        d.variant, d.status = L.DENSE_AUTO, self.status.data_ptr()
-        return d
+    def _dense_desc(self, lin: Linear, M: int, a, c, unary: int = 0):
+        return ops.dense_desc(a, lin.w, lin.K, c, bias=lin.bias, unary=unary, status=self.status, M=M)
 
     def _dense(self, lin: Linear, M: int, a, c, unary: int = 0, matvec: bool = False) -> None:
         """c[:M] = unary(a[:M] W^T + bias) on the batch kernels (a single row on the mat-vec if `matvec`)."""
-        code = lambda t: L.BF16 if t.dtype == torch.bfloat16 else L.F32
-        d = self._dense_desc(lin, M, a, c, code(a), code(c), unary)
+        d = self._dense_desc(lin, M, a, c, unary)
         if not (matvec and M == 1):
             d.variant = L.DENSE_TC if self.half else L.DENSE_SIMT
         need = int(L.lib().cutb_dense_workspace_bytes(C.byref(d)))
@@ -328,35 +320,21 @@ class LayerListDecoder:
         return d
 
     def _norm(self, rows: int, x, y, post, pre, h, keep: bool, row_index=None) -> None:
-        d = L.ResidualNormDesc()
-        d.x, d.ldx, d.pre_w = x.data_ptr(), x.stride(0), pre.data_ptr()
-        if y is not None:
-            d.y, d.ldy, d.post_w = y.data_ptr(), y.stride(0), post.data_ptr()
-            d.x_out = x.data_ptr() if keep else None
-        d.h, d.ldh, d.h_dtype = h.data_ptr(), h.stride(0), self.act_code if h.dtype == self.act_t else L.F32
-        d.row_index = row_index.data_ptr() if row_index is not None else None
-        d.rows, d.dim, d.groups, d.eps = rows, self.cfg.width, self.cfg.norm_groups, self.cfg.norm_eps
-        self._call("cutb_residual_norm", d)
+        self.launches += 1
+        ops.residual_norm(x[:rows] if row_index is None else x, pre, self.cfg.norm_groups, self.cfg.norm_eps, dim=self.cfg.width, y=y,
+                          post_w=post, x_out=x if keep else None, out=h, row_index=row_index)
 
     def _attn_desc(self, i: int, seq: Sequence, n: int, qkv, out, v_first):
-        m, (kc, vc), d = self.cfg.layers[i].mixer, seq.kv[i], L.WindowAttnDesc()
-        d.kv_dtype, d.out_dtype = self.act_code, L.BF16 if out.dtype == torch.bfloat16 else L.F32
-        d.n_heads, d.n_kv_heads, d.dim, d.vdim, d.k_head, d.v_head = m.heads, m.kv_heads, m.dim, m.vdim, pad(m.dim, 8), pad(m.vdim, 8)
-        d.ring_rows, d.window, d.rot_dims, d.max_pos = kc.shape[0], m.window, m.rot.dims, self.max_seq
-        d.rot_pairing, d.sink, d.scale = m.rot.pairing, int(m.sink), m.scale
-        d.cos_table, d.sin_table = (t.data_ptr() for t in self._tables[m.rot])
-        p = qkv.data_ptr()
-        d.q, d.k, d.v, d.ldqkv = p, p + 4 * m.q_rows, p + 4 * (m.q_rows + m.k_rows), qkv.stride(0)
-        d.k_cache, d.v_cache = kc.data_ptr(), vc.data_ptr()
-        if m.v_mix and v_first is not None:
-            if i == self.cfg.first_mixing:
-                d.v_first_out = v_first.data_ptr()
-            else:
-                d.v_first, d.v_mix = v_first.data_ptr(), self.layers[i]["vmix"]
-            d.ld_first = v_first.stride(0)
-        d.pos_ptr, d.pos, d.n_tokens = seq.state.data_ptr() + 8, seq.pos, n
-        d.out, d.ldo, d.status = out.data_ptr(), out.stride(0), self.status.data_ptr()
-        return d
+        m, (kc, vc) = self.cfg.layers[i].mixer, seq.kv[i]
+        cos_t, sin_t = self._tables[m.rot]
+        mix = {}
+        if m.v_mix and i == self.cfg.first_mixing:
+            mix = {"v_first_out": v_first}
+        elif m.v_mix:
+            mix = {"v_first": v_first, "v_mix": self.layers[i]["vmix"]}
+        return ops.window_desc(qkv[:n], m.heads, m.kv_heads, m.dim, m.vdim, kc, vc, window=m.window, scale=m.scale, out=out, cos_t=cos_t,
+                               sin_t=sin_t, rot_dims=m.rot.dims, pairing=m.rot.pairing, max_pos=self.max_seq, sink=m.sink, pos=seq.pos,
+                               pos_ptr=seq.state.data_ptr() + 8, status=self.status, **mix)
 
     # -- a portion of a prompt ----------------------------------------------------------------------------------------
     def _sizes(self):
@@ -396,8 +374,7 @@ class LayerListDecoder:
                 self._call("cutb_window_attention", a)
             else:
                 self.launches += 1
-                L.check(L.lib().cutb_mingru_scan(rows.data_ptr(), rows.stride(0), m.width, seq.gru[i].data_ptr(), mid.data_ptr(), self.act_code,
-                                                 mid.stride(0), T, self._stream()))
+                ops.mingru_scan(rows[:T], m.width, seq.gru[i], mid)
             self._dense(d["out"], T, mid, y)
             out, post = y, d["norm1b"]
             if l.mlp is not None:
@@ -453,12 +430,11 @@ class LayerListDecoder:
         def staged(lin, out, post, pre, c, unary=0):
             """The projection behind a sublayer border: residual add and norms while its input is staged."""
             nonlocal cur
-            d = self._dense_desc(lin, 1, None, c, L.F32, L.F32, unary)
-            d.res_x, d.norm_w, d.norm_groups, d.norm_eps = b["x"][cur].data_ptr(), pre.data_ptr(), cfg.norm_groups, cfg.norm_eps
-            if out is not None:
-                d.res_y, d.res_norm_w, d.res_out = out.data_ptr(), post.data_ptr(), b["x"][cur ^ 1].data_ptr()
-                cur ^= 1
-            return d
+            d = self._dense_desc(lin, 1, None, c, unary)
+            if out is None:
+                return ops.stage_input(d, b["x"][cur], pre, cfg.norm_groups, cfg.norm_eps)
+            cur ^= 1
+            return ops.stage_input(d, b["x"][cur ^ 1], pre, cfg.norm_groups, cfg.norm_eps, out, post, b["x"][cur])
 
         call("cutb_embedding_bigram", self._embed_desc(1, seq.state.data_ptr(), seq.state.data_ptr() + 4, b["x"][0]))
         out, post = None, None
@@ -470,11 +446,11 @@ class LayerListDecoder:
                 q = staged(d["in"], out, post, d["norm1"], b["mid"])
                 q.gru_state = seq.gru[i].data_ptr()
                 call("cutb_dense_matmul", q)
-            call("cutb_dense_matmul", self._dense_desc(d["out"], 1, b["mid"], b["y"], L.F32, L.F32))
+            call("cutb_dense_matmul", self._dense_desc(d["out"], 1, b["mid"], b["y"]))
             out, post = b["y"], d["norm1b"]
             if l.mlp is not None:
                 call("cutb_dense_matmul", staged(d["up"], out, post, d["norm2"], b["mid"], l.mlp.unary))
-                call("cutb_dense_matmul", self._dense_desc(d["down"], 1, b["mid"], b["y"], L.F32, L.F32))
+                call("cutb_dense_matmul", self._dense_desc(d["down"], 1, b["mid"], b["y"]))
                 out, post = b["y"], d["norm2b"]
         call("cutb_dense_matmul", staged(self.head, out, post, self.final_norm, b["logits"]))
         seqd.append(lambda: L.check(lib.cutb_argreduce(1, b["logits"].data_ptr(), b["next"].data_ptr(), cfg.vocab, self._stream())))

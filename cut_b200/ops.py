@@ -297,3 +297,121 @@ def glu_pairs(x: torch.Tensor, unary_op: int = 133, out: torch.Tensor | None = N
     L.check(L.lib().cutb_glu_pairs(x.data_ptr(), out.data_ptr(), rows, cols // 2, x.stride(0), out.stride(0), unary_op, _stream_ptr()))
     return out
 
+
+
+# ---- layer-list models: dense bf16 weights, windowed attention, gated recurrence ----
+def _el(t: torch.Tensor) -> int:
+    if t.dtype == torch.bfloat16:
+        return L.BF16
+    if t.dtype == torch.float32:
+        return L.F32
+    raise RuntimeError("element types here are float32 and bfloat16")
+
+
+def _ptr(t: torch.Tensor | None):
+    return t.data_ptr() if t is not None else None
+
+
+def dense_desc(A: torch.Tensor | None, W: torch.Tensor, K: int, out: torch.Tensor, *, bias=None, unary: int = 0, variant: int = L.DENSE_AUTO,
+               status=None, M: int | None = None, N: int | None = None):
+    """cutb_dense_desc of out[M, N] = unary(A[M, K] W[N, :K]^T + bias); W bf16 with rows padded to 8, out a 2-D view.  A may be
+    None when the input is staged from the residual stream (ops.stage_input)."""
+    d = L.DenseDesc()
+    d.M, d.K, d.N = (A.shape[0] if A is not None else 1) if M is None else M, K, W.shape[0] if N is None else N
+    d.a_dtype, d.c_dtype = _el(A) if A is not None else L.F32, _el(out)
+    if A is not None:
+        d.A, d.lda = A.data_ptr(), A.stride(0)
+    d.W, d.ldw, d.bias = W.data_ptr(), W.stride(0), _ptr(bias)
+    d.unary_op, d.C, d.ldc, d.variant, d.status = unary, out.data_ptr(), out.stride(0), variant, _ptr(status)
+    return d
+
+
+def stage_input(d, x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float, y=None, post_w=None, x_out=None):
+    """Makes the mat-vec of `d` read N(x + N(y; post_w); norm_w) instead of A (x + ... also goes to x_out)."""
+    d.res_x, d.norm_w, d.norm_groups, d.norm_eps = x.data_ptr(), norm_w.data_ptr(), groups, eps
+    d.res_y, d.res_norm_w, d.res_out = _ptr(y), _ptr(post_w), _ptr(x_out)
+    return d
+
+
+def dense_matmul(d) -> None:
+    """Launches a dense matmul, with a workspace of its own if the shape asks for one and the descriptor has none."""
+    need = int(L.lib().cutb_dense_workspace_bytes(C.byref(d)))
+    ws = None
+    if need and not d.workspace:
+        ws = torch.empty(need, dtype=torch.uint8, device="cuda")
+        d.workspace, d.workspace_bytes = ws.data_ptr(), need
+    L.check(L.lib().cutb_dense_matmul(C.byref(d), _stream_ptr()))
+    if ws is not None:
+        d.workspace, d.workspace_bytes = None, 0
+
+
+def residual_norm(x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float, *, dim: int | None = None, y=None, post_w=None, x_out=None,
+                  out: torch.Tensor | None = None, dtype=torch.float32, row_index=None) -> torch.Tensor:
+    """h = N(x + N(y; post_w); norm_w) row by row; the new residual goes to x_out when given (x itself is allowed)."""
+    d = L.ResidualNormDesc()
+    dim = x.shape[1] if dim is None else dim
+    rows = x.shape[0] if row_index is None else row_index.numel()
+    if out is None:
+        out = torch.zeros((rows, x.stride(0)), dtype=dtype, device=x.device)
+    d.x, d.ldx, d.pre_w, d.x_out = x.data_ptr(), x.stride(0), norm_w.data_ptr(), _ptr(x_out)
+    if y is not None:
+        d.y, d.ldy, d.post_w = y.data_ptr(), y.stride(0), post_w.data_ptr()
+    d.h, d.ldh, d.h_dtype, d.row_index = out.data_ptr(), out.stride(0), _el(out), _ptr(row_index)
+    d.rows, d.dim, d.groups, d.eps = rows, dim, groups, eps
+    L.check(L.lib().cutb_residual_norm(C.byref(d), _stream_ptr()))
+    return out
+
+
+def embedding_bigram(tokens: torch.Tensor, embed: torch.Tensor, *, prev=None, bigram=None, mul_prev: int = 0, mul_cur: int = 0,
+                     status=None) -> torch.Tensor:
+    """embed[token] + bigram[hash of (previous token, token)] for int32 tokens; prev: one-element int32 tensor or None."""
+    n, dim = tokens.numel(), embed.shape[1]
+    out = torch.empty((n, dim), dtype=torch.float32, device=embed.device)
+    d = L.EmbedDesc()
+    d.tokens, d.prev, d.embed, d.ld_embed, d.out, d.ldo = tokens.data_ptr(), _ptr(prev), embed.data_ptr(), embed.stride(0), out.data_ptr(), dim
+    if bigram is not None:
+        d.bigram, d.ld_bigram, d.buckets, d.mul_prev, d.mul_cur = bigram.data_ptr(), bigram.stride(0), bigram.shape[0] - 1, mul_prev, mul_cur
+    d.n, d.dim, d.vocab, d.status = n, dim, embed.shape[0], _ptr(status)
+    L.check(L.lib().cutb_embedding_bigram(C.byref(d), _stream_ptr()))
+    return out
+
+
+def mingru_scan(zxg: torch.Tensor, width: int, state: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """The recurrence over the rows of zxg ([T, >= 3 width] pre-activations); state is continued in place."""
+    L.check(L.lib().cutb_mingru_scan(zxg.data_ptr(), zxg.stride(0), width, state.data_ptr(), out.data_ptr(), _el(out), out.stride(0),
+                                     zxg.shape[0], _stream_ptr()))
+    return out
+
+
+def window_desc(qkv: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, vdim: int, k_cache: torch.Tensor, v_cache: torch.Tensor, *,
+                window: int, scale: float, out: torch.Tensor, cos_t=None, sin_t=None, rot_dims: int = 0, pairing: int = L.ROT_NEIGHBOURS,
+                max_pos: int, sink: bool = False, pos: int = 0, pos_ptr: int | None = None, v_first=None, v_mix: float = 0.0,
+                v_first_out=None, status=None):
+    """cutb_window_attn_desc over rows [q | k | v] of a stacked projection and ring caches [ring_rows, n_kv_heads * pad8(head)]."""
+    d = L.WindowAttnDesc()
+    d.kv_dtype, d.out_dtype = _el(k_cache), _el(out)
+    d.n_heads, d.n_kv_heads, d.dim, d.vdim = n_heads, n_kv_heads, dim, vdim
+    d.k_head, d.v_head, d.ring_rows = k_cache.shape[1] // n_kv_heads, v_cache.shape[1] // n_kv_heads, k_cache.shape[0]
+    d.window, d.rot_dims, d.max_pos, d.rot_pairing, d.sink = window, rot_dims, max_pos, pairing, int(sink)
+    d.scale, d.v_mix, d.cos_table, d.sin_table = scale, v_mix, _ptr(cos_t), _ptr(sin_t)
+    p, q_rows, k_rows = qkv.data_ptr(), n_heads * dim, n_kv_heads * dim
+    d.q, d.k, d.v, d.ldqkv = p, p + 4 * q_rows, p + 4 * (q_rows + k_rows), qkv.stride(0)
+    d.k_cache, d.v_cache = k_cache.data_ptr(), v_cache.data_ptr()
+    d.v_first, d.v_first_out = _ptr(v_first), _ptr(v_first_out)
+    first = v_first if v_first is not None else v_first_out
+    d.ld_first = first.stride(0) if first is not None else 0
+    d.pos_ptr, d.pos, d.n_tokens = pos_ptr, pos, qkv.shape[0]
+    d.out, d.ldo, d.status = out.data_ptr(), out.stride(0), _ptr(status)
+    return d
+
+
+def window_kv_write(d) -> None:
+    L.check(L.lib().cutb_window_kv_write(C.byref(d), _stream_ptr()))
+
+
+def window_attention(d) -> None:
+    L.check(L.lib().cutb_window_attention(C.byref(d), _stream_ptr()))
+
+
+def window_attention_decode(d) -> None:
+    L.check(L.lib().cutb_window_attention_decode(C.byref(d), _stream_ptr()))
