@@ -23,6 +23,7 @@ import torch
 
 from . import _lib as L
 from . import ops, synth
+from .decoding import RecordedStep
 
 UNARY_SILU, BINARY_ADD, BINARY_MUL = 133, 0, 2  # OperatorEnum codes (operators/runtime/ComputeOpsShared.h)
 
@@ -101,6 +102,13 @@ def synthetic_weights(cfg: LlamaConfig, seed: int = 0, distinct_layers: bool = T
             "embedding": (0.02 * rng.standard_normal((cfg.vocab, cfg.hidden))).astype(np.float32)}
 
 
+class LlamaSequence:
+    """The decoder's only sequence place: how far it is."""
+
+    def __init__(self):
+        self.pos, self.open = 0, True
+
+
 class LlamaDecoder:
     """Device state of one model and the recorded decode step.
 
@@ -151,7 +159,8 @@ class LlamaDecoder:
         self.fuse_rope = fuse_rope
         self._keep, self._descs, self.launches_per_step = [], [], 0
         self._plan()
-        self.graph = None
+        self.graph = self.recorded = None
+        self._opened = False
 
     # -- the recorded sequence: a list of closures over prepared descriptors --------------------
     def _matvec(self, A, W, N, out, fusion_type=L.FUSION_NONE, fusion_op=0, D=None, after_matvec=False, norm=None, glu=False):
@@ -309,21 +318,59 @@ class LlamaDecoder:
 
     def capture(self) -> None:
         """Records step + advance into one CUDA graph (call after at least one eager step)."""
-        torch.cuda.synchronize(self.dev)
         saved = (self.token.clone(), self.params.clone())
-        g = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(g):
-            self._run()
-            self._advance()
+        rec = RecordedStep([*self._seq, self._advance], self.dev)
+        rec.capture()
         self.token.copy_(saved[0])
         self.params.copy_(saved[1])
-        self.graph = g
+        self.recorded, self.graph = rec, rec.graph
 
     def replay(self, n: int) -> None:
         if self.graph is None:
             raise RuntimeError("capture() first")
-        for _ in range(n):
-            self.graph.replay()
+        self.recorded.replay(n)
+
+    # -- the interface of decoding.py: one sequence at a time -------------------------------------------------------------
+    def open(self) -> "LlamaSequence":
+        if self._opened:
+            raise RuntimeError("no free sequence place: this decoder serves one sequence at a time")
+        self._opened = True
+        return LlamaSequence()
+
+    def close(self, seq: "LlamaSequence") -> None:
+        if not seq.open:
+            raise RuntimeError("this sequence is not open")
+        seq.open = self._opened = False
+
+    def forward(self, seq: "LlamaSequence", tokens, want=()):
+        """The next tokens (more than one: as one batch); logits of the last one if it is wanted -- the batch computes no
+        others."""
+        tokens, want = [int(t) for t in tokens], [int(w) for w in want]
+        if not seq.open or not tokens or want not in ([], [len(tokens) - 1]):
+            raise ValueError("an open sequence, at least one token, and at most the last place wanted")
+        if any(not 0 <= t < self.cfg.vocab for t in tokens) or seq.pos + len(tokens) > self.cfg.max_seq:
+            raise ValueError("token past the vocabulary, or more tokens than the cache holds")
+        logits = self.step(tokens[0], seq.pos) if len(tokens) == 1 else self.prefill(tokens, seq.pos)
+        if len(tokens) == 1:  # as prefill leaves it: the pick is the next token
+            self._advance()
+        seq.pos += len(tokens)
+        return logits.view(1, -1) if want else None
+
+    def decode_greedy(self, seq: "LlamaSequence", n: int) -> list:
+        """n tokens: the arg-max of the last logits first, then one recorded step per further token."""
+        if seq.pos + n - 1 > self.cfg.max_seq:
+            raise ValueError("more tokens than the cache holds")
+        if self.graph is None and n > 1:
+            self.capture()
+        picks = torch.empty(n, dtype=torch.int32, device=self.dev)
+        for i in range(n):
+            picks[i].copy_(self.token[0])
+            if i + 1 < n:
+                self.replay(1)
+                seq.pos += 1
+        ids = picks.cpu().tolist()
+        self.check_status()
+        return ids
 
     def check_status(self) -> None:
         st = int(self.status.item())

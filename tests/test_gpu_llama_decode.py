@@ -221,3 +221,33 @@ def test_cpp_runner_batched_prefill_matches_composed_checker(tmp_path, fmt, T):
         rel = np.linalg.norm(got - want) / np.linalg.norm(want)
         assert np.isfinite(got).all() and rel <= 3e-3, (step, rel)
         assert int(out["tokens"][step]) == int(np.argmax(out["logits"][step]))
+
+
+def test_request_queue_over_the_llama_decoder():
+    """The shared generation loop (open, portions, recorded greedy steps, close) gives what step-by-step decoding gives."""
+    from cut_b200.decoding import RequestQueue
+    from cut_b200.llama_decode import LlamaConfig, LlamaDecoder, synthetic_weights
+
+    cfg = LlamaConfig(n_layers=2, hidden=256, n_heads=4, n_kv_heads=2, head_dim=64, ffn=512, vocab=512, max_seq=64, fmt=0)
+    w = synthetic_weights(cfg, seed=5)
+    w["embedding"] = (w["embedding"] * 50).astype(np.float32)
+    dec, ref = LlamaDecoder(cfg, w), LlamaDecoder(cfg, w)
+    prompts = [[3, 500, 17, 17], [9], [301, 42, 7]]
+    queue = RequestQueue(dec, portion=1)
+    requests = [queue.submit(p, 6) for p in prompts]
+    queue.run()
+    for r in requests:
+        fed, want = list(r.prompt), []
+        for pos in range(len(r.prompt) + 5):
+            logits = ref.step(fed[pos], pos)
+            if pos + 1 >= len(r.prompt):
+                want.append(int(ref.next_tok.item()))
+                fed.append(want[-1])
+        assert r.tokens == want
+    seq = dec.open()
+    with pytest.raises(RuntimeError, match="no free sequence place"):
+        dec.open()
+    with pytest.raises(ValueError):
+        dec.forward(seq, [512], [])
+    assert dec.forward(seq, [1, 2, 3], [2]).shape == (1, cfg.vocab)
+    dec.close(seq)
