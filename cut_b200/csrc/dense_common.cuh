@@ -23,8 +23,9 @@ __device__ __forceinline__ void store_out(void *C, int bf16, size_t i, float v) 
   if (bf16) reinterpret_cast<__nv_bfloat16 *>(C)[i] = __float2bfloat16_rn(v);
   else reinterpret_cast<float *>(C)[i] = v;
 }
-__device__ __forceinline__ float sigmoid(float x) { return 1.0f / (1.0f + expf(-x)); }
-__device__ __forceinline__ float silu(float x) { return x / (1.0f + expf(-x)); }
+// (__fdividef: within 2 ulp; a denominator past 2^126, x below -87, gives 0 like the exact quotient to fp32's last digits)
+__device__ __forceinline__ float sigmoid(float x) { return __fdividef(1.0f, 1.0f + expf(-x)); }
+__device__ __forceinline__ float silu(float x) { return __fdividef(x, 1.0f + expf(-x)); }
 
 // Elementwise epilogue: 0 none, CUTB_UNARY_RELU_SQUARE, or one of the unary codes of the quantized matmul.
 __device__ __forceinline__ float dense_unary(float x, int op) {

@@ -44,7 +44,7 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_
 
 // One block per row: x' = x + N(y), h = N(x') (norm_stage.cuh), h in bf16 or fp32.
 template <int IT>  // 16-byte pieces per thread of the register path; 0: any row
-__global__ void __launch_bounds__(256) residual_norm_kernel(NormStage n, uint64_t ldx, uint64_t ldy, const uint32_t *row_index, void *h,
+__global__ void __launch_bounds__(512) residual_norm_kernel(NormStage n, uint64_t ldx, uint64_t ldy, const uint32_t *row_index, void *h,
                                                             uint64_t ldh, int h_bf16) {
   extern __shared__ __align__(16) float rn_smem[];
   pdl_enter();
@@ -69,12 +69,14 @@ constexpr int SC_CH = 16, SC_SEG = 32, SC_L = 4, SC_THREADS = SC_CH * SC_SEG;
 
 __global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float *__restrict__ zxg, uint64_t ld, uint32_t width, float *state,
                                                                     void *out, uint64_t ldo, int out_bf16, uint32_t T) {
-  __shared__ float As[2][SC_SEG][SC_CH], Bs[2][SC_SEG][SC_CH];
+  __shared__ float As[SC_CH][SC_SEG + 1], Bs[SC_CH][SC_SEG + 1];  // the segments' maps, then (in Bs) their start states
   pdl_enter();
   const uint32_t c = threadIdx.x % SC_CH, seg = threadIdx.x / SC_CH, ch = blockIdx.x * SC_CH + c;
   const bool live = ch < width;
-  float carry = live ? state[ch] : 0.f;
-  uint32_t buf = 0;
+  // (warp w carries the state of channel w from turn to turn)
+  const uint32_t lane = threadIdx.x & 31, warp = threadIdx.x >> 5, wch = blockIdx.x * SC_CH + warp;
+  static_assert(SC_SEG == 32 && SC_THREADS / 32 == SC_CH, "one warp per channel, one lane per segment");
+  float carry = wch < width ? state[wch] : 0.f;
   float z1[SC_L], u1[SC_L], g1[SC_L];  // the next turn's pre-activations, in flight
   auto load = [&](uint32_t t0) {
 #pragma unroll
@@ -88,7 +90,7 @@ __global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float 
     }
   };
   load(0);
-  for (uint32_t t0 = 0; t0 < T; t0 += SC_SEG * SC_L, buf ^= 1) {
+  for (uint32_t t0 = 0; t0 < T; t0 += SC_SEG * SC_L) {
     float a[SC_L], b[SC_L], g[SC_L];
     float A = 1.f, B = 0.f;
 #pragma unroll
@@ -103,15 +105,22 @@ __global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float 
       A *= a[i];
       B = fmaf(a[i], B, b[i]);
     }
-    As[buf][seg][c] = A, Bs[buf][seg][c] = B;
+    As[c][seg] = A, Bs[c][seg] = B;
     __syncthreads();
-    float s = carry, mine = carry;
-#pragma unroll 8
-    for (uint32_t k = 0; k < SC_SEG; ++k) {
-      if (k == seg) mine = s;
-      s = fmaf(As[buf][k][c], s, Bs[buf][k][c]);
+    {  // warp w composes the maps of channel w, lane = segment
+      float pa = As[warp][lane], pb = Bs[warp][lane];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const float qa = __shfl_up_sync(0xffffffffu, pa, o), qb = __shfl_up_sync(0xffffffffu, pb, o);
+        if (lane >= (uint32_t)o) pb = fmaf(pa, qb, pb), pa *= qa;
+      }
+      const float after = fmaf(pa, carry, pb);  // state behind this lane's segment
+      const float start = __shfl_up_sync(0xffffffffu, after, 1);
+      Bs[warp][lane] = lane ? start : carry;
+      carry = __shfl_sync(0xffffffffu, after, 31);
     }
-    carry = s;
+    __syncthreads();
+    float mine = Bs[c][seg];
 #pragma unroll
     for (int i = 0; i < SC_L; ++i) {
       const uint32_t t = t0 + seg * SC_L + i;
@@ -119,7 +128,7 @@ __global__ void __launch_bounds__(SC_THREADS, 2) mingru_scan_kernel(const float 
       if (live && t < T) store_out(out, out_bf16, (size_t)t * ldo + ch, mine * silu(g[i]));
     }
   }
-  if (live && seg == 0) state[ch] = carry;
+  if (wch < width && lane == 0) state[wch] = carry;
 }
 
 __global__ void sequence_advance_kernel(cutb_sequence_state *s, const uint32_t *tokens, uint32_t n, const float *next) {
@@ -141,14 +150,15 @@ int embedding_bigram_launch(const cutb_embed_desc &d, cudaStream_t stream) {
 int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) {
   const NormStage n{d.x, d.y, d.post_w, d.pre_w, d.y ? d.x_out : nullptr, d.dim, d.groups, d.eps};
   const int bf16 = d.h_dtype == CUTB_BF16;
-  if (norm_stage_fits(d.dim, d.groups, 256, 8)) {  // the row stays in registers
+  if (norm_stage_fits(d.dim, d.groups, 512, 4)) {  // the row stays in registers
     const uint32_t small = 4 * (d.dim / 64);
-    auto go = [&](auto kernel) -> cudaError_t {
-      return launch_pdl(kernel, dim3(d.rows), dim3(256), small, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16);
+    auto go = [&](auto kernel, uint32_t threads) -> cudaError_t {
+      return launch_pdl(kernel, dim3(d.rows), dim3(threads), small, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16);
     };
-    if (d.dim <= 2048) CUTB_CUDA_TRY(go(residual_norm_kernel<2>));
-    else if (d.dim <= 4096) CUTB_CUDA_TRY(go(residual_norm_kernel<4>));
-    else CUTB_CUDA_TRY(go(residual_norm_kernel<8>));
+    if (d.dim <= 1024) CUTB_CUDA_TRY(go(residual_norm_kernel<2>, 128));
+    else if (d.dim <= 2048) CUTB_CUDA_TRY(go(residual_norm_kernel<2>, 256));
+    else if (d.dim <= 4096) CUTB_CUDA_TRY(go(residual_norm_kernel<2>, 512));
+    else CUTB_CUDA_TRY(go(residual_norm_kernel<4>, 512));
     return CUTB_OK;
   }
   const uint32_t smem = 4 * norm_stage_floats(d.dim, d.groups);
