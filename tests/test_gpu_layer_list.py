@@ -266,7 +266,8 @@ class Attn:
 
 
 ATTN = [(4, 2, 32, 24, 33, 150), (1, 1, 10, 7, 1, 40), (6, 2, 64, 64, 64, 200), (8, 1, 128, 128, 100, 260), (3, 3, 48, 96, 65, 130),
-        (2, 1, 130, 200, 50, 90), (16, 1, 24, 72, 700, 300), (5, 1, 100, 20, 200, 330)]
+        (2, 1, 130, 200, 50, 90), (16, 1, 24, 72, 700, 300), (5, 1, 100, 20, 200, 330),
+        (56, 4, 16, 8, 20, 40), (100, 2, 24, 24, 30, 50)]  # (many heads: two and four per block in decoding)
 
 
 @pytest.mark.parametrize("H,G,dim,vdim,window,T", ATTN)
