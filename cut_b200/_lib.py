@@ -14,6 +14,7 @@ OK, ERR_INVALID, ERR_UNSUPPORTED, ERR_CUDA, ERR_WORKSPACE, ERR_TIMEOUT, ERR_RANG
 Q8_0, Q4_0, Q4_K, Q5_K, Q6_K, BF16, Q4_1, Q5_0 = 0, 1, 2, 3, 4, 5, 6, 7  # from Q5_K on: cutb_dequant only
 F32, F16 = 0, 1
 UNARY_RELU_SQUARE, NO_TOKEN = 200, 0xFFFFFFFF
+GLU_NONE, GLU_CLAMPED = 0, 1
 DENSE_AUTO, DENSE_MATVEC, DENSE_TC, DENSE_SIMT = -1, 0, 1, 2
 ROT_HALVES, ROT_NEIGHBOURS = 0, 1
 LAYOUT_GGUF_BLOCKS, LAYOUT_KN_PLANES = 0, 1
@@ -38,6 +39,9 @@ EXPORTS = [
     "cutb_variant_name",
     "cutb_dense_select_variant", "cutb_dense_workspace_bytes", "cutb_dense_matmul", "cutb_residual_norm", "cutb_embedding_bigram",
     "cutb_mingru_scan", "cutb_sequence_advance", "cutb_window_kv_write", "cutb_window_attention", "cutb_window_attention_decode",
+    "cutb_latent_kv_write", "cutb_latent_attention", "cutb_latent_splits", "cutb_latent_workspace_bytes", "cutb_latent_values",
+    "cutb_latent_prefill_supported", "cutb_latent_prefill", "cutb_moe_route", "cutb_moe_scatter", "cutb_moe_matmul", "cutb_expert_up",
+    "cutb_expert_down",
 ]
 
 
@@ -73,6 +77,8 @@ class DenseDesc(C.Structure):
         ("res_out", C.c_void_p),
         ("norm_groups", C.c_uint32), ("norm_eps", C.c_float),
         ("gru_state", C.c_void_p),
+        ("norm_center", C.c_int32), ("res_scale", C.c_float), ("norm_out", C.c_void_p),
+        ("batch", C.c_uint32), ("a_batch", C.c_uint32), ("c_batch", C.c_uint32),
     ]
 
 
@@ -83,6 +89,9 @@ class ResidualNormDesc(C.Structure):
         ("ldx", C.c_uint64), ("ldy", C.c_uint64), ("ldh", C.c_uint64),
         ("rows", C.c_uint32), ("dim", C.c_uint32), ("groups", C.c_uint32),
         ("eps", C.c_float), ("h_dtype", C.c_int32),
+        ("center", C.c_int32), ("y_scale", C.c_float),
+        ("parts", C.c_void_p), ("part_rows", C.c_void_p), ("part_w", C.c_void_p), ("ld_parts", C.c_uint64),
+        ("n_parts", C.c_uint32), ("parts_dtype", C.c_int32),
     ]
 
 
@@ -92,7 +101,7 @@ class EmbedDesc(C.Structure):
         ("ld_embed", C.c_uint64), ("ld_bigram", C.c_uint64), ("ldo", C.c_uint64),
         ("n", C.c_uint32), ("dim", C.c_uint32), ("vocab", C.c_uint32), ("buckets", C.c_uint32),
         ("mul_prev", C.c_uint32), ("mul_cur", C.c_uint32),
-        ("status", C.c_void_p),
+        ("status", C.c_void_p), ("scale", C.c_float),
     ]
 
 
@@ -111,6 +120,52 @@ class WindowAttnDesc(C.Structure):
         ("pos_ptr", C.c_void_p), ("pos", C.c_uint32), ("n_tokens", C.c_uint32),
         ("out", C.c_void_p), ("ldo", C.c_uint64),
         ("status", C.c_void_p),
+    ]
+
+
+class LatentAttnDesc(C.Structure):
+    _fields_ = [
+        ("kv_dtype", C.c_int32), ("out_dtype", C.c_int32),
+        ("n_heads", C.c_uint32), ("dim", C.c_uint32), ("rot_dim", C.c_uint32), ("vdim", C.c_uint32), ("rank", C.c_uint32),
+        ("rot_at", C.c_uint32), ("q_rank", C.c_uint32), ("max_pos", C.c_uint32),
+        ("scale", C.c_float), ("eps", C.c_float),
+        ("sink", C.c_void_p), ("cos_table", C.c_void_p), ("sin_table", C.c_void_p),
+        ("lat", C.c_void_p), ("lat_norm_w", C.c_void_p), ("cq", C.c_void_p), ("cq_norm_w", C.c_void_p),
+        ("ld_lat", C.c_uint64), ("ld_cq", C.c_uint64), ("ld_cq_out", C.c_uint64),
+        ("cq_out", C.c_void_p),
+        ("q", C.c_void_p), ("qa", C.c_void_p), ("ldq", C.c_uint64), ("ld_qa", C.c_uint64),
+        ("cache", C.c_void_p), ("ld_cache", C.c_uint64),
+        ("k_exp", C.c_void_p), ("v_exp", C.c_void_p), ("ld_k", C.c_uint64), ("ld_v", C.c_uint64),
+        ("pos_ptr", C.c_void_p), ("pos", C.c_uint32), ("n_tokens", C.c_uint32),
+        ("out", C.c_void_p), ("ldo", C.c_uint64),
+        ("workspace", C.c_void_p), ("workspace_bytes", C.c_uint64),
+        ("status", C.c_void_p),
+        ("w_uv", C.c_void_p), ("ld_uv", C.c_uint64),
+    ]
+
+
+class MoeDesc(C.Structure):
+    _fields_ = [
+        ("n_tokens", C.c_uint32), ("experts", C.c_uint32), ("top", C.c_uint32), ("K", C.c_uint32), ("N", C.c_uint32),
+        ("logits", C.c_void_p), ("ld_logits", C.c_uint64),
+        ("weights", C.c_void_p), ("ids", C.c_void_p), ("slots", C.c_void_p), ("offsets", C.c_void_p),
+        ("a_dtype", C.c_int32), ("c_dtype", C.c_int32),
+        ("A", C.c_void_p), ("lda", C.c_uint64), ("W", C.c_void_p), ("ldw", C.c_uint32),
+        ("C", C.c_void_p), ("ldc", C.c_uint64),
+        ("glu", C.c_int32), ("alpha", C.c_float), ("beta", C.c_float), ("limit", C.c_float),
+        ("variant", C.c_int32), ("status", C.c_void_p),
+    ]
+
+
+class ExpertDesc(C.Structure):
+    _fields_ = [
+        ("experts", C.c_uint32), ("top", C.c_uint32), ("width", C.c_uint32), ("ff", C.c_uint32),
+        ("logits", C.c_void_p), ("ids", C.c_void_p), ("W", C.c_void_p), ("ldw", C.c_uint32),
+        ("x", C.c_void_p), ("act", C.c_void_p),
+        ("alpha", C.c_float), ("beta", C.c_float), ("limit", C.c_float),
+        ("Wd", C.c_void_p), ("Nd", C.c_uint32), ("Kd", C.c_uint32), ("ldwd", C.c_uint32),
+        ("xd", C.c_void_p), ("xd_norm_w", C.c_void_p), ("eps", C.c_float),
+        ("C", C.c_void_p), ("flags", C.c_uint32),
     ]
 
 
@@ -154,9 +209,15 @@ def _bind_layers(l: C.CDLL) -> None:
     l.cutb_device_sm_count.restype = C.c_int
     for name, desc in (("cutb_dense_matmul", DenseDesc), ("cutb_residual_norm", ResidualNormDesc), ("cutb_embedding_bigram", EmbedDesc),
                        ("cutb_window_kv_write", WindowAttnDesc), ("cutb_window_attention", WindowAttnDesc),
-                       ("cutb_window_attention_decode", WindowAttnDesc)):
+                       ("cutb_window_attention_decode", WindowAttnDesc), ("cutb_latent_kv_write", LatentAttnDesc),
+                       ("cutb_latent_attention", LatentAttnDesc), ("cutb_latent_values", LatentAttnDesc), ("cutb_latent_prefill", LatentAttnDesc),
+                       ("cutb_moe_route", MoeDesc), ("cutb_moe_scatter", MoeDesc), ("cutb_moe_matmul", MoeDesc), ("cutb_expert_up", ExpertDesc),
+                       ("cutb_expert_down", ExpertDesc)):
         getattr(l, name).restype = C.c_int
         getattr(l, name).argtypes = [C.POINTER(desc), C.c_void_p]
+    for name, kind in (("cutb_latent_splits", C.c_uint32), ("cutb_latent_workspace_bytes", C.c_uint64), ("cutb_latent_prefill_supported", C.c_int)):
+        getattr(l, name).restype = kind
+        getattr(l, name).argtypes = [C.POINTER(LatentAttnDesc)]
     l.cutb_dense_select_variant.restype = C.c_int
     l.cutb_dense_select_variant.argtypes = [C.POINTER(DenseDesc)]
     l.cutb_dense_workspace_bytes.restype = C.c_uint64

@@ -14,12 +14,14 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 LIB = os.path.join(HERE, "libcutb.so")
 # layer operators and the layer-list models over dense bf16 weights: what a model without quantized weights needs
-LAYER_SOURCES = ["cabi_layers.cu", "common.cu", "layer_ops.cu", "mixer_ops.cu", "dense_matvec.cu", "dense_gemm.cu", "window_attention.cu"]
+LAYER_SOURCES = ["cabi_layers.cu", "common.cu", "layer_ops.cu", "mixer_ops.cu", "dense_matvec.cu", "dense_gemm.cu", "window_attention.cu",
+                 "latent_attention.cu", "moe.cu", "expert_matvec.cu"]
 QUANT_SOURCES = ["cabi.cu", "qgemv_blocks.cu", "qmatmul_generic.cu", "dequant.cu", "transpose_q4.cu",
                  "qgemm_tc.cu", "qgemm_skinny.cu", "repack.cu", "attention.cu", "attention_prefill.cu", "qgemv_planes.cu"]
 SOURCES = QUANT_SOURCES + LAYER_SOURCES
 LAYERS_LIB = os.path.join(HERE, "libcutb_layers.so")
 HEADERS = ["common.cuh", "kernels.h", "tcgen05.cuh", "qgemm_tc_common.cuh", "dense_common.cuh", "norm_stage.cuh",
+           "attn_common.cuh", "moe_common.cuh",
            os.path.join("..", "..", "include", "cutb.h")]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC,-fvisibility=hidden"]

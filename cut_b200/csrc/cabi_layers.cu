@@ -3,6 +3,7 @@
 // quantized weights needs.
 #include "common.cuh"
 #include "kernels.h"
+#include "moe_common.cuh"
 
 namespace cutb {
 const char *last_error();
@@ -42,15 +43,20 @@ int check_dense(const cutb_dense_desc *d) {
     return CUTB_ERR_INVALID;
   }
   if (staged) {
-    if (d->M != 1 || !d->res_x || (d->res_y && !d->res_norm_w) || d->norm_groups == 0 || d->K % d->norm_groups || d->res_out == d->res_x) {
-      set_last_error("dense_matmul: a staged norm needs one row, res_x, the residual norm's weight with res_y, and groups that divide K");
+    if (d->M != 1 || !d->res_x || d->norm_groups == 0 || d->K % d->norm_groups || d->res_out == d->res_x) {
+      set_last_error("dense_matmul: a staged norm needs one row, res_x (not res_out), and groups that divide K");
       return CUTB_ERR_INVALID;
     }
-    for (const void *q : {(const void *)d->res_x, (const void *)d->res_y, (const void *)d->res_norm_w, (const void *)d->norm_w, (const void *)d->res_out})
+    for (const void *q : {(const void *)d->res_x, (const void *)d->res_y, (const void *)d->res_norm_w, (const void *)d->norm_w, (const void *)d->res_out, (const void *)d->norm_out})
       if (reinterpret_cast<uintptr_t>(q) % 16) {
         set_last_error("dense_matmul: operands of the staged norm must be 16-byte aligned");
         return CUTB_ERR_INVALID;
       }
+  }
+  if (d->batch > 1 && (staged || d->gru_state || d->bias || d->unary_op || d->lda < (uint64_t)(d->batch - 1) * d->a_batch + d->K ||
+                       (d->M > 1 && d->ldc < (uint64_t)(d->batch - 1) * d->c_batch + d->N))) {
+    set_last_error("dense_matmul: a batch of products has no bias, no elementwise op and no fused steps, and its columns lie within the rows");
+    return CUTB_ERR_INVALID;
   }
   if (d->gru_state && (d->M != 1 || d->N % 3)) {
     set_last_error("dense_matmul: the recurrence step needs one row and three stacked matrices");
@@ -65,6 +71,7 @@ int check_dense(const cutb_dense_desc *d) {
 
 int dense_select(const cutb_dense_desc &d) {
   if (d.variant != CUTB_DENSE_AUTO) return d.variant;
+  if (d.batch > 1) return d.M == 1 && dense_matvec_supported(d) ? CUTB_DENSE_MATVEC : CUTB_DENSE_SIMT;
   if (d.M == 1) return CUTB_DENSE_MATVEC;
   return dense_gemm_tc_supported(d) ? CUTB_DENSE_TC : CUTB_DENSE_SIMT;
 }
@@ -99,6 +106,56 @@ int check_window(const cutb_window_attn_desc *d, bool write, bool read) {
   }
   return CUTB_OK;
 }
+int check_latent(const cutb_latent_attn_desc *d, const char *what, bool reads) {
+  if (!d || !dtype_ok(d->kv_dtype) || !dtype_ok(d->out_dtype) || d->n_heads == 0 || d->n_tokens == 0 || d->max_pos == 0) {
+    set_last_error("%s: null descriptor, no heads, tokens or positions, or an element type that is not fp32 / bf16", what);
+    return CUTB_ERR_INVALID;
+  }
+  if (d->rank == 0 || d->rank > 1024 || d->rot_dim % 2 || d->rot_dim > 1024 || d->rot_at < d->rank || d->rot_at % 8 || d->ld_cache % 8 ||
+      d->ld_cache < d->rot_at + (uint64_t)(d->rot_dim + 7) / 8 * 8) {
+    set_last_error("%s: rank 1..1024, rot_dim even and at most 1024, rot_at and ld_cache multiples of 8 that hold both parts", what);
+    return CUTB_ERR_INVALID;
+  }
+  if (((reads || d->lat) && (!d->cache || reinterpret_cast<uintptr_t>(d->cache) % 32)) || (d->rot_dim && (!d->cos_table || !d->sin_table)) ||
+      (d->lat && (!d->lat_norm_w || d->ld_lat < d->rank + d->rot_dim))) {
+    set_last_error("%s: the cache must be 32-byte aligned; tables for the rotation, a norm weight and whole rows for the latents are needed", what);
+    return CUTB_ERR_INVALID;
+  }
+  return CUTB_OK;
+}
+
+int check_moe(const cutb_moe_desc *d, const char *what) {
+  if (!d || d->n_tokens == 0 || d->top == 0 || d->experts < d->top || d->experts > MOE_MAX_EXPERTS || (uint64_t)d->n_tokens * d->top > 0x7fffffffu) {
+    set_last_error("%s: null descriptor, no tokens, or not 1 <= top <= experts <= %u", what, MOE_MAX_EXPERTS);
+    return CUTB_ERR_INVALID;
+  }
+  return CUTB_OK;
+}
+
+int check_expert(const cutb_expert_desc *d, bool up) {
+  const char *what = up ? "expert_up" : "expert_down";
+  if (!d || d->top == 0 || d->experts < d->top || d->experts > MOE_MAX_EXPERTS || d->width == 0 || d->ff == 0 || !d->ids || !d->W || !d->act ||
+      (up && (!d->logits || !d->x)) || (!up && !d->C)) {
+    set_last_error("%s: null pointer, an empty size, or not 1 <= top <= experts <= %u", what, MOE_MAX_EXPERTS);
+    return CUTB_ERR_INVALID;
+  }
+  if (d->ldw % 8 || d->ldw < (up ? d->width : d->ff) || reinterpret_cast<uintptr_t>(d->W) % 16 ||
+      (d->Wd && (d->Nd == 0 || d->Kd == 0 || d->ldwd % 8 || d->ldwd < d->Kd || reinterpret_cast<uintptr_t>(d->Wd) % 16 || !d->xd || !d->C))) {
+    set_last_error("%s: weight rows must be 16-byte aligned and hold their elements; the dense matrix needs an input and an output", what);
+    return CUTB_ERR_INVALID;
+  }
+  if ((up && d->Wd && d->xd_norm_w && (reinterpret_cast<uintptr_t>(d->xd) | reinterpret_cast<uintptr_t>(d->xd_norm_w)) % 16) ||
+      (!up && d->Wd && d->Nd != d->width)) {
+    set_last_error("%s: the normed input must be 16-byte aligned; the dense matrix of expert_down has width rows", what);
+    return CUTB_ERR_INVALID;
+  }
+  if (!expert_matvec_supported(*d, up)) {
+    set_last_error("%s: the input does not fit in shared memory, or more than 64 experts per token", what);
+    return CUTB_ERR_UNSUPPORTED;
+  }
+  return CUTB_OK;
+}
+
 // the kernels compare positions with the window in 32 bits
 cutb_window_attn_desc clamp_window(const cutb_window_attn_desc *d) {
   cutb_window_attn_desc c = *d;
@@ -238,8 +295,10 @@ int cutb_dense_matmul(const cutb_dense_desc *desc, void *stream) {
 }
 
 int cutb_residual_norm(const cutb_residual_norm_desc *d, void *stream) {
-  if (!d || !d->x || !d->pre_w || !d->h || (d->y && !d->post_w) || !dtype_ok(d->h_dtype)) {
-    set_last_error("residual_norm: null pointer, or an output type that is not fp32 / bf16");
+  if (!d || !d->x || !d->pre_w || !d->h || !dtype_ok(d->h_dtype) ||
+      (d->n_parts && (!d->parts || !d->part_rows || !d->part_w || !dtype_ok(d->parts_dtype) || d->ld_parts % 4 || d->ld_parts < d->dim ||
+                      reinterpret_cast<uintptr_t>(d->parts) % 16))) {
+    set_last_error("residual_norm: null pointer, an element type that is not fp32 / bf16, or parts that are not 16-byte aligned rows");
     return CUTB_ERR_INVALID;
   }
   if (d->rows == 0) return CUTB_OK;
@@ -301,6 +360,124 @@ int cutb_window_attention_decode(const cutb_window_attn_desc *d, void *stream) {
     return CUTB_ERR_INVALID;
   }
   return window_attention_decode_launch(clamp_window(d), reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_latent_kv_write(const cutb_latent_attn_desc *d, void *stream) {
+  if (int rc = check_latent(d, "latent_kv_write", false)) return rc;
+  if ((!d->lat && !d->cq) || (d->cq && (!d->cq_norm_w || !d->cq_out || d->q_rank == 0 || d->ld_cq < d->q_rank || d->ld_cq_out < d->q_rank))) {
+    set_last_error("latent_kv_write: nothing to do, or no norm weight, output or whole rows for the latent queries");
+    return CUTB_ERR_INVALID;
+  }
+  return latent_kv_write_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+uint32_t cutb_latent_splits(const cutb_latent_attn_desc *d) { return check_latent(d, "latent_splits", false) == CUTB_OK ? latent_splits(*d) : 0; }
+
+uint64_t cutb_latent_workspace_bytes(const cutb_latent_attn_desc *d) {
+  if (check_latent(d, "latent_workspace", false) != CUTB_OK || d->n_tokens != 1) return 0;
+  const uint64_t n = (uint64_t)d->n_heads * latent_splits(*d);
+  return ((2 * n + 3) / 4 * 4 + n * ((d->rank + 3) / 4 * 4)) * sizeof(float);
+}
+
+int cutb_latent_attention(const cutb_latent_attn_desc *d, void *stream) {
+  if (int rc = check_latent(d, "latent_attention", true)) return rc;
+  if (!d->q || !d->qa || (d->lat && d->n_tokens != 1) || (d->n_tokens != 1 && (!d->out || d->ldo < (uint64_t)d->n_heads * d->rank)) ||
+      (d->n_tokens > 1 && (d->ldq < (uint64_t)d->n_heads * (d->dim + d->rot_dim) || d->ld_qa < (uint64_t)d->n_heads * d->rank))) {
+    set_last_error("latent_attention: null pointer, short rows, or a cache row to make for more than one token");
+    return CUTB_ERR_INVALID;
+  }
+  if (d->n_tokens > 65535) {
+    set_last_error("latent_attention: at most 65535 tokens per call");
+    return CUTB_ERR_UNSUPPORTED;
+  }
+  if (d->n_tokens == 1 && (!d->workspace || d->workspace_bytes < cutb_latent_workspace_bytes(d) || reinterpret_cast<uintptr_t>(d->workspace) % 16)) {
+    set_last_error("latent_attention: one token needs a workspace of cutb_latent_workspace_bytes(), 16-byte aligned");
+    return CUTB_ERR_WORKSPACE;
+  }
+  return latent_attention_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_latent_values(const cutb_latent_attn_desc *d, void *stream) {
+  if (int rc = check_latent(d, "latent_values", false)) return rc;
+  if (d->n_tokens != 1 || d->vdim == 0 || !d->w_uv || d->ld_uv % 8 || d->ld_uv < d->rank || reinterpret_cast<uintptr_t>(d->w_uv) % 16 || !d->out ||
+      !d->workspace || d->workspace_bytes < cutb_latent_workspace_bytes(d)) {
+    set_last_error("latent_values: one token, its workspace, and 16-byte aligned rows of W_uv are needed");
+    return CUTB_ERR_INVALID;
+  }
+  return latent_values_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_latent_prefill_supported(const cutb_latent_attn_desc *d) { return d && latent_prefill_supported(*d) ? 1 : 0; }
+
+int cutb_latent_prefill(const cutb_latent_attn_desc *d, void *stream) {
+  if (int rc = check_latent(d, "latent_prefill", true)) return rc;
+  const uint64_t H = d->n_heads;
+  if (!d->q || !d->k_exp || !d->v_exp || !d->out || d->ldq < H * (d->dim + d->rot_dim) || d->ld_k < H * d->dim || d->ld_v < H * d->vdim ||
+      d->ldo < H * d->vdim || d->ld_k % 8 || d->ld_v % 8 ||
+      (reinterpret_cast<uintptr_t>(d->k_exp) | reinterpret_cast<uintptr_t>(d->v_exp)) % 16) {
+    set_last_error("latent_prefill: null pointer, short rows, or keys and values that are not 16-byte aligned");
+    return CUTB_ERR_INVALID;
+  }
+  if (!latent_prefill_supported(*d)) {
+    set_last_error("latent_prefill: bf16, head parts that are multiples of 8, dim + rot_dim <= 256 and vdim <= 256");
+    return CUTB_ERR_UNSUPPORTED;
+  }
+  return latent_prefill_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_moe_route(const cutb_moe_desc *d, void *stream) {
+  if (int rc = check_moe(d, "moe_route")) return rc;
+  if (!d->logits || !d->weights || !d->ids || !d->slots || !d->offsets || d->ld_logits < d->experts) {
+    set_last_error("moe_route: null pointer, or short rows of logits");
+    return CUTB_ERR_INVALID;
+  }
+  return moe_route_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_moe_scatter(const cutb_moe_desc *d, void *stream) {
+  if (int rc = check_moe(d, "moe_scatter")) return rc;
+  if (!d->A || !d->C || !d->slots || !dtype_ok(d->a_dtype) || d->c_dtype != d->a_dtype || d->K == 0 || d->lda < d->K || d->ldc < d->K) {
+    set_last_error("moe_scatter: null pointer, short rows, or different element types");
+    return CUTB_ERR_INVALID;
+  }
+  return moe_scatter_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_moe_matmul(const cutb_moe_desc *d, void *stream) {
+  if (int rc = check_moe(d, "moe_matmul")) return rc;
+  const uint32_t cols = d->glu ? d->N / 2 : d->N;
+  if (!d->A || !d->W || !d->C || !d->offsets || !dtype_ok(d->a_dtype) || !dtype_ok(d->c_dtype) || d->K == 0 || d->N == 0 || d->lda < d->K ||
+      d->ldc < cols || (d->glu && d->N % 2) || d->glu < CUTB_GLU_NONE || d->glu > CUTB_GLU_CLAMPED) {
+    set_last_error("moe_matmul: null pointer, short rows, an unknown element type or gated unit, or an odd number of paired rows");
+    return CUTB_ERR_INVALID;
+  }
+  if (d->ldw % 8 || d->ldw < d->K || reinterpret_cast<uintptr_t>(d->W) % 16 || reinterpret_cast<uintptr_t>(d->A) % 16 ||
+      (d->ldc % 8 == 0 && reinterpret_cast<uintptr_t>(d->C) % 16)) {
+    set_last_error("moe_matmul: A, C and the weight rows must be 16-byte aligned and hold K elements (ldw=%u)", d->ldw);
+    return CUTB_ERR_INVALID;
+  }
+  if (d->variant == CUTB_DENSE_TC) {
+    if (d->a_dtype != CUTB_BF16 || d->lda % 8) {
+      set_last_error("moe_matmul: the tensor cores read bf16 rows, 16-byte aligned");
+      return CUTB_ERR_UNSUPPORTED;
+    }
+    return moe_gemm_tc_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+  }
+  if (d->variant != CUTB_DENSE_SIMT) {
+    set_last_error("moe_matmul: unknown variant %d", d->variant);
+    return CUTB_ERR_INVALID;
+  }
+  return moe_gemm_simt_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_expert_up(const cutb_expert_desc *d, void *stream) {
+  if (int rc = check_expert(d, true)) return rc;
+  return expert_up_launch(*d, reinterpret_cast<cudaStream_t>(stream));
+}
+
+int cutb_expert_down(const cutb_expert_desc *d, void *stream) {
+  if (int rc = check_expert(d, false)) return rc;
+  return expert_down_launch(*d, reinterpret_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

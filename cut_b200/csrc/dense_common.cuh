@@ -19,6 +19,17 @@ __device__ __forceinline__ uint4 ld_stream(const uint4 *p) {
   asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
   return v;
 }
+// eight bf16 weights times eight activations
+__device__ __forceinline__ void fma8(float &acc, const uint4 w, const float4 a, const float4 b) {
+  acc = fmaf(bf16_lo(w.x), a.x, acc);
+  acc = fmaf(bf16_hi(w.x), a.y, acc);
+  acc = fmaf(bf16_lo(w.y), a.z, acc);
+  acc = fmaf(bf16_hi(w.y), a.w, acc);
+  acc = fmaf(bf16_lo(w.z), b.x, acc);
+  acc = fmaf(bf16_hi(w.z), b.y, acc);
+  acc = fmaf(bf16_lo(w.w), b.z, acc);
+  acc = fmaf(bf16_hi(w.w), b.w, acc);
+}
 __device__ __forceinline__ void store_out(void *C, int bf16, size_t i, float v) {
   if (bf16) reinterpret_cast<__nv_bfloat16 *>(C)[i] = __float2bfloat16_rn(v);
   else reinterpret_cast<float *>(C)[i] = v;
@@ -35,6 +46,16 @@ __device__ __forceinline__ float dense_unary(float x, int op) {
     return r * r;
   }
   return apply_epilogue(x, CUTB_FUSION_UNARY, op, 0.f);
+}
+
+// The gated unit of a feed-forward's element: the gate clamped from above, the up value from both sides.
+struct GluParams {
+  int kind;  // CUTB_GLU_*
+  float alpha, beta, limit;
+};
+__device__ __forceinline__ float glu(const GluParams &p, float g, float u) {
+  g = fminf(g, p.limit), u = fminf(fmaxf(u, -p.limit), p.limit);
+  return __fdividef(g, 1.0f + expf(-p.alpha * g)) * (u + p.beta);
 }
 
 // The gated recurrence of one channel: gate z and candidate c from this token's pre-activations.

@@ -15,6 +15,11 @@
 //    prefetched before the wait;
 //  * output: bias and one elementwise op, or the gated recurrence  s = (1 - z) s + z c  of one token with its state update
 //    and output gate (rows z, x, g of channel j are rows j, width + j, 2 width + j of the stacked weight).
+//
+// head_matvec_kernel: the same for a batch of small products, a matrix and a slice of the row per head (latent attention's
+// W_uk^T q and W_uv o).  4 .. 32 lanes share a row by its length, a block takes consecutive rows and stages the slices of their
+// heads only.  A slice may be made here from the partial sums that the blocks of an attention left (each with its maximum and
+// weight sum).
 #include <cuda_bf16.h>
 
 #include "common.cuh"
@@ -38,22 +43,12 @@ struct MvParams {
   uint32_t row_step; // distance of a tile's rows (1, or width for the recurrence)
   int a_bf16, c_bf16, unary;
   NormStage norm;  // norm.pre_w != null: the input is staged from the residual stream
+  float *norm_out;
 };
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
-__device__ __forceinline__ void fma8(float &acc, const uint4 w, const float4 a, const float4 b) {
-  acc = fmaf(bf16_lo(w.x), a.x, acc);
-  acc = fmaf(bf16_hi(w.x), a.y, acc);
-  acc = fmaf(bf16_lo(w.y), a.z, acc);
-  acc = fmaf(bf16_hi(w.y), a.w, acc);
-  acc = fmaf(bf16_lo(w.z), b.x, acc);
-  acc = fmaf(bf16_hi(w.z), b.y, acc);
-  acc = fmaf(bf16_lo(w.w), b.z, acc);
-  acc = fmaf(bf16_hi(w.w), b.w, acc);
-}
-
 template <int R, int UNR, bool GRU>
 __global__ void __launch_bounds__(MV_MAX_THREADS, 1) dense_matvec_kernel(const MvParams p) {
   extern __shared__ __align__(16) float mv_smem[];
@@ -99,11 +94,20 @@ __global__ void __launch_bounds__(MV_MAX_THREADS, 1) dense_matvec_kernel(const M
   // ---- the activation row -> two planes, zero past K ----
   auto put1 = [&](uint32_t i, float v) { mv_smem[(i & 4 ? 4 * p.K8 : 0) + (i >> 3) * 4 + (i & 3)] = v; };
   auto put4 = [&](uint32_t i, float4 v) { (i & 4 ? hi : lo)[i >> 3] = v; };
+  float *keep = blockIdx.x == 0 ? p.norm_out : nullptr;
+  auto norm1 = [&](uint32_t i, float v) {
+    put1(i, v);
+    if (keep) keep[i] = v;
+  };
+  auto norm4 = [&](uint32_t i, float4 v) {
+    put4(i, v);
+    if (keep) *reinterpret_cast<float4 *>(keep + i) = v;
+  };
   for (uint32_t i = p.K + tid; i < 8 * p.K8; i += nt) put1(i, 0.f);
   if (fast_norm) {
-    stage_norm_regs<2>(p.norm, stage + 2 * p.K, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, put4);
+    stage_norm_regs<2>(p.norm, stage + 2 * p.K, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, norm4);
   } else if (p.norm.pre_w) {
-    stage_norm(p.norm, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, put4, put1);
+    stage_norm(p.norm, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, norm4, norm1);
   } else if (p.a_bf16) {
     const __nv_bfloat16 *a = reinterpret_cast<const __nv_bfloat16 *>(p.A);
     for (uint32_t i = tid; i < p.K; i += nt) put1(i, __bfloat162float(a[i]));
@@ -196,6 +200,84 @@ template <int R, int UNR, bool GRU> int mv_launch(MvParams &p, uint32_t smem, ui
   return CUTB_OK;
 }
 
+// ---- a product per head ------------------------------------------------------------------------------------------------
+constexpr int HV_THREADS = 256;
+
+template <int LPR> __global__ void __launch_bounds__(HV_THREADS) head_matvec_kernel(const HeadMvParams p, uint32_t rows_per_block) {
+  extern __shared__ __align__(16) float hv_smem[];
+  constexpr uint32_t RPW = 32 / LPR, PASS = HV_THREADS / 32 * RPW;  // rows of a warp and of the block at a time
+  constexpr int U = 4;
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane % LPR;
+  const uint32_t total = p.batch * p.N, r0 = blockIdx.x * rows_per_block, r1 = min(r0 + rows_per_block, total);
+  const uint32_t h0 = r0 / p.N, nh = (r1 - 1) / p.N - h0 + 1, K8 = p.K8, plane = nh * K8;
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  float4 *lo = reinterpret_cast<float4 *>(hv_smem), *hi = lo + plane;
+  const uint4 *W4 = reinterpret_cast<const uint4 *>(p.W);
+  // the first row's weights are on their way before the wait for the previous kernel
+  uint4 w[U];
+  auto load = [&](uint32_t row, uint32_t k) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) w[u] = row < r1 && k + LPR * u < K8 ? ld_stream(W4 + (size_t)row * p.ldw8 + k + LPR * u) : make_uint4(0, 0, 0, 0);
+  };
+  const uint32_t first = r0 + warp * RPW + lane / LPR;
+  load(first, sub);
+  pdl_enter();
+  auto put = [&](uint32_t h, uint32_t k, float v) { hv_smem[(k & 4 ? 4 * plane : 0) + (h * K8 + (k >> 3)) * 4 + (k & 3)] = v; };
+  for (uint32_t h = 0; h < nh; ++h) {
+    if (p.splits) {
+      const float2 *ml = p.ml + (size_t)(h0 + h) * p.splits;
+      const float *part = p.part + (size_t)(h0 + h) * p.splits * p.ld_part;
+      float m = -1e30f, l = 0.f;
+      for (uint32_t s = 0; s < p.splits; ++s) m = fmaxf(m, ml[s].x);
+      for (uint32_t s = 0; s < p.splits; ++s) l = fmaf(exp2f(ml[s].x - m), ml[s].y, l);
+      const float inv = 1.0f / l;
+      for (uint32_t k = tid; k < 8 * K8; k += HV_THREADS) {
+        float v = 0.f;
+        if (k < p.K) {
+#pragma unroll 8
+          for (uint32_t s = 0; s < p.splits; ++s) v = fmaf(exp2f(ml[s].x - m), part[(size_t)s * p.ld_part + k], v);
+        }
+        put(h, k, v * inv);
+      }
+    } else {
+      const float *x = p.x + (size_t)(h0 + h) * p.x_batch;
+      for (uint32_t k = tid; k < 8 * K8; k += HV_THREADS) put(h, k, k < p.K ? x[k] : 0.f);
+    }
+  }
+  __syncthreads();
+  for (uint32_t row = first; row - lane / LPR < r1; row += PASS) {  // (the same number of turns in every lane)
+    const uint32_t h = min(row, r1 - 1) / p.N - h0;
+    const float4 *xl = lo + h * K8, *xh = hi + h * K8;
+    float acc = 0.f;
+    for (uint32_t k = sub; k < K8 + sub; k += LPR * U) {
+      if (!(row == first && k == sub)) load(row, k);
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (k + LPR * u < K8) fma8(acc, w[u], xl[k + LPR * u], xh[k + LPR * u]);
+    }
+#pragma unroll
+    for (int o = LPR / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+    if (sub == 0 && row < r1) store_out(p.C, p.c_bf16, (size_t)(row / p.N) * p.c_batch + row % p.N, acc);
+  }
+}
+
+template <int LPR> int hv_launch(const HeadMvParams &p, uint32_t sms, cudaStream_t stream) {
+  constexpr uint32_t PASS = HV_THREADS / 32 * (32 / LPR);
+  const uint32_t total = p.batch * p.N;
+  uint32_t rows = (total + 2 * sms - 1) / (2 * sms);
+  rows = (rows + PASS - 1) / PASS * PASS;
+  auto smem_of = [&](uint32_t r) { return 32 * p.K8 * (r / p.N + 2 < p.batch ? r / p.N + 2 : p.batch); };
+  while (rows > PASS && smem_of(rows) > 96 * 1024) rows -= PASS;
+  const uint32_t smem = smem_of(rows);
+  if (smem > 200 * 1024) {
+    set_last_error("head mat-vec: the slices of %u rows of %u elements do not fit in shared memory", rows, p.K);
+    return CUTB_ERR_UNSUPPORTED;
+  }
+  if (smem > 48 * 1024) CUTB_CUDA_TRY(cudaFuncSetAttribute(head_matvec_kernel<LPR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  CUTB_CUDA_TRY(launch_pdl(head_matvec_kernel<LPR>, dim3((total + rows - 1) / rows), dim3(HV_THREADS), smem, stream, p, rows));
+  return CUTB_OK;
+}
+
 uint32_t mv_smem_bytes(const cutb_dense_desc &d) {
   const uint32_t K8 = (d.K + 7) / 8;
   return 4 * (8 * K8 + (d.norm_w ? norm_stage_floats(d.K, d.norm_groups) : 0));
@@ -203,16 +285,37 @@ uint32_t mv_smem_bytes(const cutb_dense_desc &d) {
 
 }  // namespace
 
-bool dense_matvec_supported(const cutb_dense_desc &d) { return d.M == 1 && mv_smem_bytes(d) <= 220 * 1024; }
+bool dense_matvec_supported(const cutb_dense_desc &d) {
+  if (d.batch > 1) return d.M == 1 && d.a_dtype == CUTB_F32 && !d.bias && !d.unary_op;
+  return d.M == 1 && mv_smem_bytes(d) <= 220 * 1024;
+}
+
+int head_matvec_launch(const HeadMvParams &p, cudaStream_t stream) {
+  DeviceInfo di;
+  if (int rc = get_device_info(&di)) return rc;
+  const uint32_t sms = (uint32_t)di.sm_count;
+  // about four 16-byte pieces per lane
+  if (p.K8 <= 16) return hv_launch<4>(p, sms, stream);
+  if (p.K8 <= 32) return hv_launch<8>(p, sms, stream);
+  if (p.K8 <= 64) return hv_launch<16>(p, sms, stream);
+  return hv_launch<32>(p, sms, stream);
+}
 
 int dense_matvec_launch(const cutb_dense_desc &d, cudaStream_t stream) {
   DeviceInfo di;
   if (int rc = get_device_info(&di)) return rc;
+  if (d.batch > 1) {
+    HeadMvParams h{};
+    h.x = reinterpret_cast<const float *>(d.A), h.x_batch = d.a_batch, h.W = d.W, h.C = d.C, h.c_bf16 = d.c_dtype == CUTB_BF16;
+    h.batch = d.batch, h.K = d.K, h.K8 = (d.K + 7) / 8, h.N = d.N, h.ldw8 = d.ldw / 8, h.c_batch = d.c_batch;
+    return head_matvec_launch(h, stream);
+  }
   MvParams p{};
   p.A = d.A, p.W = reinterpret_cast<const __nv_bfloat16 *>(d.W), p.bias = d.bias, p.C = d.C, p.state = d.gru_state;
   p.K = d.K, p.K8 = (d.K + 7) / 8, p.N = d.N, p.ldw8 = d.ldw / 8;
   p.a_bf16 = d.a_dtype == CUTB_BF16, p.c_bf16 = d.c_dtype == CUTB_BF16, p.unary = d.unary_op;
-  p.norm = NormStage{d.res_x, d.res_y, d.res_norm_w, d.norm_w, d.res_out, d.K, d.norm_groups ? d.norm_groups : 1, d.norm_eps};
+  p.norm = NormStage{d.res_x, d.res_y, d.res_norm_w, d.norm_w, d.res_out, d.K, d.norm_groups ? d.norm_groups : 1, d.norm_eps, d.norm_center, d.res_scale};
+  p.norm_out = d.norm_out;
   const bool gru = d.gru_state != nullptr;
   const uint32_t sms = (uint32_t)di.sm_count;
   const uint32_t sms_all = sms * MV_MAX_WARPS;

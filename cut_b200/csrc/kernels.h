@@ -82,7 +82,34 @@ int attention_decode_launch(int kv_dtype, const float *q, const void *kC, const 
                             uint32_t nHeads, uint32_t nKvHeads, uint32_t headDim, uint64_t ld, uint32_t max_seq, float scale,
                             void *workspace, int *status, cudaStream_t stream);
 
-// Layer-list models over dense bf16 weights (dense_matvec.cu, dense_gemm.cu, mixer_ops.cu, window_attention.cu).
+// Layer-list models over dense bf16 weights (dense_matvec.cu, dense_gemm.cu, mixer_ops.cu, window_attention.cu,
+// latent_attention.cu, moe.cu, expert_matvec.cu).
+// A product per head for one token: C[b * c_batch + n] = W[b * N + n] . x[b * x_batch ..], or (splits > 0) x made from the partial
+// sums part [b][splits][ld_part] with {maximum (log2 units), weight sum} ml [b][splits].
+struct HeadMvParams {
+  const float *x;
+  const void *W;
+  void *C;
+  uint32_t batch, K, K8, N, ldw8, x_batch, c_batch;
+  int c_bf16;
+  const float2 *ml;
+  const float *part;
+  uint32_t splits, ld_part;
+};
+int head_matvec_launch(const HeadMvParams &p, cudaStream_t stream);
+int moe_gemm_tc_launch(const cutb_moe_desc &d, cudaStream_t stream);
+int moe_gemm_simt_launch(const cutb_moe_desc &d, cudaStream_t stream);
+int moe_route_launch(const cutb_moe_desc &d, cudaStream_t stream);
+int moe_scatter_launch(const cutb_moe_desc &d, cudaStream_t stream);
+bool expert_matvec_supported(const cutb_expert_desc &d, bool up);
+int expert_up_launch(const cutb_expert_desc &d, cudaStream_t stream);
+int expert_down_launch(const cutb_expert_desc &d, cudaStream_t stream);
+uint32_t latent_splits(const cutb_latent_attn_desc &d);
+int latent_kv_write_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);
+int latent_attention_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);
+int latent_values_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);
+bool latent_prefill_supported(const cutb_latent_attn_desc &d);
+int latent_prefill_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);
 bool dense_matvec_supported(const cutb_dense_desc &d);
 int dense_matvec_launch(const cutb_dense_desc &d, cudaStream_t stream);
 bool dense_gemm_tc_supported(const cutb_dense_desc &d);

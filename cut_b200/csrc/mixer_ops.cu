@@ -10,7 +10,7 @@
 namespace cutb {
 namespace {
 
-// out[i, :] = embed[token_i] + bigram[(prev_i * mul_prev + token_i * mul_cur) mod buckets]; a sequence's first token has no
+// out[i, :] = scale embed[token_i] + bigram[(prev_i * mul_prev + token_i * mul_cur) mod buckets]; a sequence's first token has no
 // previous one and takes row `buckets`.  One block per token.
 __global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_desc d, int vec) {
   pdl_enter();
@@ -34,15 +34,17 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_
     for (uint32_t c = threadIdx.x; c < d.dim / 8; c += 256) {
       const uint4 x = __ldg(reinterpret_cast<const uint4 *>(e) + c), y = b ? __ldg(reinterpret_cast<const uint4 *>(b) + c) : make_uint4(0, 0, 0, 0);
       float4 *o = reinterpret_cast<float4 *>(out) + 2 * c;
-      o[0] = make_float4(bf16_lo(x.x) + bf16_lo(y.x), bf16_hi(x.x) + bf16_hi(y.x), bf16_lo(x.y) + bf16_lo(y.y), bf16_hi(x.y) + bf16_hi(y.y));
-      o[1] = make_float4(bf16_lo(x.z) + bf16_lo(y.z), bf16_hi(x.z) + bf16_hi(y.z), bf16_lo(x.w) + bf16_lo(y.w), bf16_hi(x.w) + bf16_hi(y.w));
+      o[0] = make_float4(fmaf(d.scale, bf16_lo(x.x), bf16_lo(y.x)), fmaf(d.scale, bf16_hi(x.x), bf16_hi(y.x)),
+                         fmaf(d.scale, bf16_lo(x.y), bf16_lo(y.y)), fmaf(d.scale, bf16_hi(x.y), bf16_hi(y.y)));
+      o[1] = make_float4(fmaf(d.scale, bf16_lo(x.z), bf16_lo(y.z)), fmaf(d.scale, bf16_hi(x.z), bf16_hi(y.z)),
+                         fmaf(d.scale, bf16_lo(x.w), bf16_lo(y.w)), fmaf(d.scale, bf16_hi(x.w), bf16_hi(y.w)));
     }
     return;
   }
-  for (uint32_t c = threadIdx.x; c < d.dim; c += 256) out[c] = __bfloat162float(e[c]) + (b ? __bfloat162float(b[c]) : 0.f);
+  for (uint32_t c = threadIdx.x; c < d.dim; c += 256) out[c] = fmaf(d.scale, __bfloat162float(e[c]), b ? __bfloat162float(b[c]) : 0.f);
 }
 
-// One block per row: x' = x + N(y), h = N(x') (norm_stage.cuh), h in bf16 or fp32.
+// One block per row: x' = x + y_scale P(y + gathered parts), h = N(x') (norm_stage.cuh), h in bf16 or fp32.
 template <int IT>  // 16-byte pieces per thread of the register path; 0: any row
 __global__ void __launch_bounds__(512) residual_norm_kernel(NormStage n, uint64_t ldx, uint64_t ldy, const uint32_t *row_index, void *h,
                                                             uint64_t ldh, int h_bf16) {
@@ -51,6 +53,7 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(NormStage n, uint64_
   const uint32_t row = blockIdx.x, src = row_index ? __ldg(row_index + row) : row;
   n.x += src * ldx;
   if (n.y) n.y += src * ldy;
+  n.part_rows += src * n.n_parts, n.part_w += src * n.n_parts;
   if (n.x_out) n.x_out += src * ldx;
   const size_t base = (size_t)row * ldh;
   auto put4 = [&](uint32_t i, float4 v) {
@@ -148,10 +151,11 @@ int embedding_bigram_launch(const cutb_embed_desc &d, cudaStream_t stream) {
 }
 
 int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) {
-  const NormStage n{d.x, d.y, d.post_w, d.pre_w, d.y ? d.x_out : nullptr, d.dim, d.groups, d.eps};
+  const NormStage n{d.x, d.y, d.post_w, d.pre_w, d.y || d.n_parts ? d.x_out : nullptr, d.dim, d.groups, d.eps, d.center, d.y_scale,
+                    d.parts, d.part_rows, d.part_w, d.ld_parts, d.n_parts, d.parts_dtype == CUTB_BF16};
   const int bf16 = d.h_dtype == CUTB_BF16;
   if (norm_stage_fits(d.dim, d.groups, 512, 4)) {  // the row stays in registers
-    const uint32_t small = 4 * (d.dim / 64);
+    const uint32_t small = 4 * (d.dim / 32);
     auto go = [&](auto kernel, uint32_t threads) -> cudaError_t {
       return launch_pdl(kernel, dim3(d.rows), dim3(threads), small, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16);
     };

@@ -9,7 +9,7 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from . import bigerax
+from . import bigerax, lenesun
 from .layer_list import LayerListDecoder
 from .safetensors_io import SafetensorsFile
 
@@ -24,6 +24,7 @@ class ModelEntry:
 
 REGISTRY = {
     bigerax.ARCHITECTURE: ModelEntry(bigerax.parse_config, bigerax.gather_weights, LayerListDecoder, ("bfloat16", "float32")),
+    lenesun.ARCHITECTURE: ModelEntry(lenesun.parse_config, lenesun.gather_weights, LayerListDecoder, ("bfloat16", "float32")),
 }
 
 

@@ -326,10 +326,19 @@ def dense_desc(A: torch.Tensor | None, W: torch.Tensor, K: int, out: torch.Tenso
     return d
 
 
-def stage_input(d, x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float, y=None, post_w=None, x_out=None):
-    """Makes the mat-vec of `d` read N(x + N(y; post_w); norm_w) instead of A (x + ... also goes to x_out)."""
-    d.res_x, d.norm_w, d.norm_groups, d.norm_eps = x.data_ptr(), norm_w.data_ptr(), groups, eps
-    d.res_y, d.res_norm_w, d.res_out = _ptr(y), _ptr(post_w), _ptr(x_out)
+def stage_input(d, x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float, y=None, post_w=None, x_out=None, center: bool = False,
+                y_scale: float = 1.0, norm_out=None):
+    """Makes the mat-vec of `d` read N(x + y_scale P(y); norm_w) instead of A, P = N(.; post_w) or without post_w the identity, N =
+    RMS norm or (center) layer norm; x + ... also goes to x_out, the normed row to norm_out."""
+    d.res_x, d.norm_w, d.norm_groups, d.norm_eps, d.norm_center, d.res_scale = x.data_ptr(), norm_w.data_ptr(), groups, eps, int(center), y_scale
+    d.res_y, d.res_norm_w, d.res_out, d.norm_out = _ptr(y), _ptr(post_w), _ptr(x_out), _ptr(norm_out)
+    return d
+
+
+def batch_desc(A: torch.Tensor, W: torch.Tensor, K: int, out: torch.Tensor, heads: int, a_step: int, c_step: int, *, status=None):
+    """cutb_dense_desc of `heads` products: number b maps columns b * a_step .. + K of A by rows b N .. of W to columns b * c_step .. of out."""
+    d = dense_desc(A, W, K, out, status=status, N=W.shape[0] // heads)
+    d.batch, d.a_batch, d.c_batch = heads, a_step, c_step
     return d
 
 
@@ -346,8 +355,11 @@ def dense_matmul(d) -> None:
 
 
 def residual_norm(x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float, *, dim: int | None = None, y=None, post_w=None, x_out=None,
-                  out: torch.Tensor | None = None, dtype=torch.float32, row_index=None) -> torch.Tensor:
-    """h = N(x + N(y; post_w); norm_w) row by row; the new residual goes to x_out when given (x itself is allowed)."""
+                  out: torch.Tensor | None = None, dtype=torch.float32, row_index=None, center: bool = False, y_scale: float = 1.0,
+                  parts=None) -> torch.Tensor:
+    """h = N(x + y_scale P(y + parts); norm_w) row by row (P = N(.; post_w), or the identity without post_w; N = RMS norm, or layer norm
+    with center); the new residual goes to x_out when given (x itself is allowed).  parts: (matrix, rows [., n] int32, weights [., n]):
+    row r gains sum_k weights[r, k] * matrix[rows[r, k]]."""
     d = L.ResidualNormDesc()
     dim = x.shape[1] if dim is None else dim
     rows = x.shape[0] if row_index is None else row_index.numel()
@@ -355,7 +367,12 @@ def residual_norm(x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float
         out = torch.zeros((rows, x.stride(0)), dtype=dtype, device=x.device)
     d.x, d.ldx, d.pre_w, d.x_out = x.data_ptr(), x.stride(0), norm_w.data_ptr(), _ptr(x_out)
     if y is not None:
-        d.y, d.ldy, d.post_w = y.data_ptr(), y.stride(0), post_w.data_ptr()
+        d.y, d.ldy = y.data_ptr(), y.stride(0)
+    if parts is not None:
+        m, part_rows, part_w = parts
+        d.parts, d.parts_dtype, d.ld_parts = m.data_ptr(), _el(m), m.stride(0)
+        d.part_rows, d.part_w, d.n_parts = part_rows.data_ptr(), part_w.data_ptr(), part_w.shape[1]
+    d.post_w, d.center, d.y_scale = _ptr(post_w), int(center), y_scale
     d.h, d.ldh, d.h_dtype, d.row_index = out.data_ptr(), out.stride(0), _el(out), _ptr(row_index)
     d.rows, d.dim, d.groups, d.eps = rows, dim, groups, eps
     L.check(L.lib().cutb_residual_norm(C.byref(d), _stream_ptr()))
@@ -363,15 +380,15 @@ def residual_norm(x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: float
 
 
 def embedding_bigram(tokens: torch.Tensor, embed: torch.Tensor, *, prev=None, bigram=None, mul_prev: int = 0, mul_cur: int = 0,
-                     status=None) -> torch.Tensor:
-    """embed[token] + bigram[hash of (previous token, token)] for int32 tokens; prev: one-element int32 tensor or None."""
+                     status=None, scale: float = 1.0) -> torch.Tensor:
+    """scale * embed[token] + bigram[hash of (previous token, token)] for int32 tokens; prev: one-element int32 tensor or None."""
     n, dim = tokens.numel(), embed.shape[1]
     out = torch.empty((n, dim), dtype=torch.float32, device=embed.device)
     d = L.EmbedDesc()
     d.tokens, d.prev, d.embed, d.ld_embed, d.out, d.ldo = tokens.data_ptr(), _ptr(prev), embed.data_ptr(), embed.stride(0), out.data_ptr(), dim
     if bigram is not None:
         d.bigram, d.ld_bigram, d.buckets, d.mul_prev, d.mul_cur = bigram.data_ptr(), bigram.stride(0), bigram.shape[0] - 1, mul_prev, mul_cur
-    d.n, d.dim, d.vocab, d.status = n, dim, embed.shape[0], _ptr(status)
+    d.n, d.dim, d.vocab, d.status, d.scale = n, dim, embed.shape[0], _ptr(status), scale
     L.check(L.lib().cutb_embedding_bigram(C.byref(d), _stream_ptr()))
     return out
 
@@ -415,3 +432,78 @@ def window_attention(d) -> None:
 
 def window_attention_decode(d) -> None:
     L.check(L.lib().cutb_window_attention_decode(C.byref(d), _stream_ptr()))
+
+
+# ---- latent attention, mixtures of experts ----
+def latent_desc(cache: torch.Tensor, n_heads: int, dim: int, rot_dim: int, vdim: int, rank: int, *, scale: float, eps: float, max_pos: int,
+                n_tokens: int, cos_t=None, sin_t=None, sink=None, pos: int = 0, pos_ptr: int | None = None, lat=None, lat_norm_w=None, cq=None,
+                cq_norm_w=None, cq_out=None, q=None, qa=None, k_exp=None, v_exp=None, out=None, workspace=None, w_uv=None, status=None):
+    """cutb_latent_attn_desc over a cache [rows, pad8(rank) + pad8(rot_dim)]; what a call does not use may be missing."""
+    d = L.LatentAttnDesc()
+    shape = out if out is not None else cq_out
+    d.kv_dtype, d.out_dtype = _el(cache), _el(shape) if shape is not None else L.F32
+    d.n_heads, d.dim, d.rot_dim, d.vdim, d.rank, d.rot_at, d.max_pos = n_heads, dim, rot_dim, vdim, rank, (rank + 7) // 8 * 8, max_pos
+    d.scale, d.eps, d.sink, d.cos_table, d.sin_table = scale, eps, _ptr(sink), _ptr(cos_t), _ptr(sin_t)
+    d.cache, d.ld_cache, d.n_tokens, d.pos, d.pos_ptr, d.status = cache.data_ptr(), cache.stride(0), n_tokens, pos, pos_ptr, _ptr(status)
+    if lat is not None:
+        d.lat, d.ld_lat, d.lat_norm_w = lat.data_ptr(), lat.stride(0), lat_norm_w.data_ptr()
+    if cq is not None:
+        d.cq, d.ld_cq, d.q_rank, d.cq_norm_w = cq.data_ptr(), cq.stride(0), cq_norm_w.numel(), cq_norm_w.data_ptr()
+        d.cq_out, d.ld_cq_out = cq_out.data_ptr(), cq_out.stride(0)
+    for name, t in (("q", q), ("qa", qa), ("k_exp", k_exp), ("v_exp", v_exp), ("out", out), ("w_uv", w_uv)):
+        if t is not None:
+            setattr(d, name, t.data_ptr())
+            setattr(d, {"q": "ldq", "qa": "ld_qa", "k_exp": "ld_k", "v_exp": "ld_v", "out": "ldo", "w_uv": "ld_uv"}[name], t.stride(0))
+    if workspace is not None:
+        d.workspace, d.workspace_bytes = workspace.data_ptr(), workspace.numel() * workspace.element_size()
+    return d
+
+
+def latent_workspace_bytes(d) -> int:
+    return int(L.lib().cutb_latent_workspace_bytes(C.byref(d)))
+
+
+def moe_route_desc(logits: torch.Tensor, experts: int, top: int, weights, ids, slots, offsets):
+    """cutb_moe_desc of a batch's routing: logits [T, >= experts]; weights, ids, slots [T, top], offsets [experts + 1] are written."""
+    d = L.MoeDesc()
+    d.n_tokens, d.experts, d.top = logits.shape[0], experts, top
+    d.logits, d.ld_logits = logits.data_ptr(), logits.stride(0)
+    d.weights, d.ids, d.slots, d.offsets = weights.data_ptr(), ids.data_ptr(), slots.data_ptr(), offsets.data_ptr()
+    return d
+
+
+def moe_scatter_desc(x: torch.Tensor, K: int, slots: torch.Tensor, experts: int, out: torch.Tensor):
+    """out[slots[t, k]] = x[t, :K]."""
+    d = L.MoeDesc()
+    d.n_tokens, d.top, d.experts, d.K = slots.shape[0], slots.shape[1], experts, K
+    d.A, d.lda, d.a_dtype, d.C, d.ldc, d.c_dtype, d.slots = x.data_ptr(), x.stride(0), _el(x), out.data_ptr(), out.stride(0), _el(out), slots.data_ptr()
+    return d
+
+
+def moe_matmul_desc(A: torch.Tensor, W: torch.Tensor, K: int, offsets: torch.Tensor, experts: int, tokens: int, top: int, out: torch.Tensor, *,
+                    glu: int = L.GLU_NONE, alpha: float = 0.0, beta: float = 0.0, limit: float = 0.0, variant: int = L.DENSE_SIMT, status=None):
+    """The grouped product of expert-sorted rows A [tokens * top, K] with the experts' stacked matrices W [experts * N, ldw]."""
+    d = L.MoeDesc()
+    d.n_tokens, d.top, d.experts, d.K, d.N = tokens, top, experts, K, W.shape[0] // experts
+    d.A, d.lda, d.a_dtype, d.W, d.ldw, d.C, d.ldc, d.c_dtype = A.data_ptr(), A.stride(0), _el(A), W.data_ptr(), W.stride(0), out.data_ptr(), out.stride(0), _el(out)
+    d.offsets, d.glu, d.alpha, d.beta, d.limit, d.variant, d.status = offsets.data_ptr(), glu, alpha, beta, limit, variant, _ptr(status)
+    return d
+
+
+def expert_desc(experts: int, top: int, width: int, ff: int, W: torch.Tensor, ids: torch.Tensor, act: torch.Tensor, *, logits=None, x=None,
+                alpha: float = 0.0, beta: float = 0.0, limit: float = 0.0, dense=None, dense_K: int = 0, xd=None, xd_norm_w=None, eps: float = 0.0,
+                out=None):
+    """cutb_expert_desc of one token's expert mat-vecs (logits and x: cutb_expert_up); dense: the companion matrix."""
+    d = L.ExpertDesc()
+    d.experts, d.top, d.width, d.ff, d.W, d.ldw = experts, top, width, ff, W.data_ptr(), W.stride(0)
+    d.ids, d.act, d.logits, d.x, d.alpha, d.beta, d.limit = ids.data_ptr(), act.data_ptr(), _ptr(logits), _ptr(x), alpha, beta, limit
+    if dense is not None:
+        d.Wd, d.Nd, d.Kd, d.ldwd = dense.data_ptr(), dense.shape[0], dense_K, dense.stride(0)
+        d.xd, d.xd_norm_w, d.eps = xd.data_ptr(), _ptr(xd_norm_w), eps
+    d.C = _ptr(out)
+    return d
+
+
+def launch_layer_op(name: str, d) -> None:
+    """Launches a layer operator (an entry point that takes a descriptor and a stream)."""
+    L.check(getattr(L.lib(), name)(C.byref(d), _stream_ptr()))

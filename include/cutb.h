@@ -429,7 +429,8 @@ CUTB_API int cutb_attention_decode(int kv_dtype, const float *q, const void *k_c
 
 /*
  * Layer-list models over dense bf16 weights (a model whose configuration lists its layers, each with a mixer -- windowed
- * attention or a gated recurrence -- and an optional feed-forward, with norms before and after each).  These entry points
+ * attention, latent attention or a gated recurrence -- and an optional feed-forward, dense or a mixture of experts, with norms
+ * around each or one norm for both).  These entry points
  * have no counterpart in the reference, whose runner covers llama-style GGUF models.  Element types: CUTB_F32 or CUTB_BF16
  * wherever a *_dtype field says so; weights are always bf16, everything the recurrences, norms and softmaxes read is fp32.
  */
@@ -441,13 +442,16 @@ enum { CUTB_DENSE_AUTO = -1, CUTB_DENSE_MATVEC = 0, CUTB_DENSE_TC = 1, CUTB_DENS
  * C[M, N] = unary(A[M, K] W[N, K]^T + bias), W bf16 with rows of ldw elements (a multiple of 8, zero past K, 16-byte
  * aligned), fp32 accumulation.
  *   CUTB_DENSE_MATVEC  one row; A fp32 or bf16, used as it is (no rounding).  Fused input: with norm_w set, A is ignored and
- *     the row is N(x'; norm_w) of x' = res_x + N(res_y; res_norm_w) (res_y may be null: x' = res_x), N = RMS norm in
- *     norm_groups equal parts; x' is stored to res_out when that is not null (res_out != res_x).  Fused output: with
+ *     the row is N(x'; norm_w) of x' = res_x + res_scale * N(res_y; res_norm_w) (res_y may be null: x' = res_x; res_norm_w may
+ *     be null: res_y as it is), N = RMS norm in norm_groups equal parts, or a layer norm of each part with norm_center; x' is
+ *     stored to res_out when that is not null (res_out != res_x), the normed row to norm_out (fp32).  Fused output: with
  *     gru_state set, W stacks three matrices (z, x, g; N / 3 rows each) and the call is one token of the recurrence
  *     s = (1 - z) s + z c,  C[j] = s silu(g), over the fp32 states gru_state[N / 3]; C then has N / 3 elements.
  *   CUTB_DENSE_TC      tcgen05 tensor cores, A bf16 (rows 16-byte aligned, lda % 8 == 0): prefill.
  *   CUTB_DENSE_SIMT    fp32 fused multiply-adds, A fp32 or bf16: the true 32-bit path of a prefill.
  * CUTB_DENSE_AUTO: one row -> mat-vec, more bf16 rows -> tensor cores, fp32 rows -> SIMT.
+ * batch > 1 (mat-vec and SIMT; no fused steps): `batch` products of these sizes, number b over the columns b * a_batch on of A,
+ * the rows b * N on of W and the columns b * c_batch on of C (a matrix per head).
  */
 typedef struct cutb_dense_desc {
   int32_t a_dtype, c_dtype;
@@ -470,13 +474,19 @@ typedef struct cutb_dense_desc {
   uint32_t norm_groups;
   float norm_eps;
   float *gru_state;
+  int32_t norm_center;
+  float res_scale;
+  float *norm_out;
+  uint32_t batch, a_batch, c_batch;
 } cutb_dense_desc;
 CUTB_API int cutb_dense_select_variant(const cutb_dense_desc *desc);
 CUTB_API uint64_t cutb_dense_workspace_bytes(const cutb_dense_desc *desc);
 CUTB_API int cutb_dense_matmul(const cutb_dense_desc *desc, void *stream);
 
-/* The step between two sublayers for `rows` rows: x' = x + N(y; post_w) (y null: x' = x), h = N(x'; pre_w); x' goes to x_out
- * (may be x; null: not kept).  row_index (device, optional): row r of h comes from row row_index[r] of x and y. */
+/* The step between two sublayers for `rows` rows: x' = x + y_scale * P(y + sum_k part_w[r][k] * parts[part_rows[r][k]]), P =
+ * N(.; post_w) or (post_w null) the identity; y null and n_parts 0: x' = x.  h = N(x'; pre_w), N = RMS norm in `groups` equal
+ * parts, or a layer norm of each with `center`.  x' goes to x_out (may be x; null: not kept).  row_index (device, optional):
+ * row r of h comes from row row_index[r] of x, y, part_rows and part_w. */
 typedef struct cutb_residual_norm_desc {
   const float *x, *y, *post_w, *pre_w;
   float *x_out;
@@ -486,10 +496,18 @@ typedef struct cutb_residual_norm_desc {
   uint32_t rows, dim, groups;
   float eps;
   int32_t h_dtype;
+  int32_t center;
+  float y_scale;
+  const void *parts; /* parts_dtype, rows of ld_parts elements */
+  const uint32_t *part_rows;
+  const float *part_w;
+  uint64_t ld_parts;
+  uint32_t n_parts;
+  int32_t parts_dtype;
 } cutb_residual_norm_desc;
 CUTB_API int cutb_residual_norm(const cutb_residual_norm_desc *desc, void *stream);
 
-/* out[i, :] = embed[tokens[i]] + bigram[(previous token * mul_prev + tokens[i] * mul_cur) mod buckets]; the token before
+/* out[i, :] = scale * embed[tokens[i]] + bigram[(previous token * mul_prev + tokens[i] * mul_cur) mod buckets]; the token before
  * tokens[0] is *prev (device; null or CUTB_NO_TOKEN: none, which takes table row `buckets`).  bigram null: embed only.  A
  * token past the vocabulary writes zeros and sets *status to CUTB_ERR_INVALID. */
 typedef struct cutb_embed_desc {
@@ -499,6 +517,7 @@ typedef struct cutb_embed_desc {
   uint64_t ld_embed, ld_bigram, ldo;
   uint32_t n, dim, vocab, buckets, mul_prev, mul_cur;
   int *status;
+  float scale;
 } cutb_embed_desc;
 CUTB_API int cutb_embedding_bigram(const cutb_embed_desc *desc, void *stream);
 
@@ -556,6 +575,117 @@ typedef struct cutb_window_attn_desc {
 CUTB_API int cutb_window_kv_write(const cutb_window_attn_desc *desc, void *stream);
 CUTB_API int cutb_window_attention(const cutb_window_attn_desc *desc, void *stream);
 CUTB_API int cutb_window_attention_decode(const cutb_window_attn_desc *desc, void *stream);
+
+/*
+ * Latent attention: a token's keys and values of all heads come from one latent vector c (`rank` elements) and one rotated key
+ * part r (`rot_dim`) that all heads share.  Only [c | r] is cached: row p of the cache holds position p, c in columns 0 .. rank
+ * - 1, r from column rot_at on, zeros in between (rot_at and ld_cache multiples of 8).  Head h's score of position j is
+ *   scale * (q_h . W_uk,h c_j + turned q'_h . r_j)  =  scale * ([W_uk,h^T q_h | turned q'_h] . [c_j | r_j]),
+ * causal, with exp(sink[h]) added to the softmax denominator when sink is not null (a key without a value, not scaled).
+ * Rotation: all rot_dim elements, neighbours paired, tables [max_pos][rot_dim / 2].  The first token's position is *pos_ptr
+ * (device), or pos when pos_ptr is null; positions past max_pos (the cache's rows) set *status and touch nothing.
+ *   cutb_latent_kv_write    n_tokens rows: cache row = [N(lat; lat_norm_w) | turned lat tail], lat [T][ld_lat] = rank + rot_dim
+ *       pre-activations (lat null: nothing is cached); and the latent queries cq_out = N(cq; cq_norm_w), q_rank elements (cq
+ *       null: none).  N = RMS norm.
+ *   cutb_latent_attention   absorbed form: q [T][ldq] holds each head's dim + rot_dim elements (the turned part is read), qa
+ *       [T][ld_qa] each head's W_uk,h^T q_h (rank elements); out [T][ldo] = each head's weighted sum of latents.  With lat
+ *       set (one token only) the call also makes, uses and stores that token's cache row.  For one token the keys are shared
+ *       out over cutb_latent_splits() blocks per head group: their partial sums go to `workspace`, and the product over W_uv
+ *       that follows reads them there (cutb_latent_values).
+ *   cutb_latent_values      one token: out[h] = W_uv,h * (weighted sum of latents), from the workspace of cutb_latent_attention
+ *   cutb_latent_prefill     expanded form, bf16: k_exp [positions][ld_k] = W_uk c of every head (dim elements), v_exp
+ *       [positions][ld_v] = W_uv c, r from the cache; out [T][ldo] = each head's vdim elements.  dim, rot_dim and vdim
+ *       multiples of 8, dim + rot_dim <= 256, vdim <= 256 (cutb_latent_prefill_supported).
+ */
+typedef struct cutb_latent_attn_desc {
+  int32_t kv_dtype, out_dtype;
+  uint32_t n_heads, dim, rot_dim, vdim, rank, rot_at, q_rank, max_pos;
+  float scale, eps;
+  const float *sink, *cos_table, *sin_table;
+  const float *lat, *lat_norm_w, *cq, *cq_norm_w;
+  uint64_t ld_lat, ld_cq, ld_cq_out;
+  void *cq_out; /* out_dtype */
+  const float *q, *qa;
+  uint64_t ldq, ld_qa;
+  void *cache;
+  uint64_t ld_cache;
+  const void *k_exp, *v_exp;
+  uint64_t ld_k, ld_v;
+  const uint32_t *pos_ptr;
+  uint32_t pos, n_tokens;
+  void *out;
+  uint64_t ldo;
+  void *workspace;
+  uint64_t workspace_bytes;
+  int *status;
+  const void *w_uv; /* cutb_latent_values: bf16 [n_heads * vdim][ld_uv] */
+  uint64_t ld_uv;
+} cutb_latent_attn_desc;
+CUTB_API int cutb_latent_kv_write(const cutb_latent_attn_desc *desc, void *stream);
+CUTB_API int cutb_latent_attention(const cutb_latent_attn_desc *desc, void *stream);
+CUTB_API uint32_t cutb_latent_splits(const cutb_latent_attn_desc *desc);
+CUTB_API uint64_t cutb_latent_workspace_bytes(const cutb_latent_attn_desc *desc);
+CUTB_API int cutb_latent_values(const cutb_latent_attn_desc *desc, void *stream);
+CUTB_API int cutb_latent_prefill_supported(const cutb_latent_attn_desc *desc);
+CUTB_API int cutb_latent_prefill(const cutb_latent_attn_desc *desc, void *stream);
+
+/*
+ * Mixture of experts: of `experts` feed-forwards a token uses the `top` with the largest router logits (ties: the lower index),
+ * weighted by the softmax over those logits.  Expert e: act = glu(W_gu x), out = W_down act, where rows 2 j and 2 j + 1 of W_gu
+ * are the gate and the up row of element j, and (CUTB_GLU_CLAMPED)
+ *   glu(g, u) = g' sigmoid(alpha g') (u' + beta),  g' = min(g, limit), u' = clamp(u, -limit, limit).
+ * A batch of tokens:
+ *   cutb_moe_route    logits [T][ld] -> ids and weights [T][top], and slots [T][top]: the rows of the expert-sorted arrays, where the rows of
+ *       expert e are the offsets[e] .. offsets[e + 1] - 1 (offsets: experts + 1, written); order: expert, then token.
+ *   cutb_moe_scatter  sorted[slots[t][k]] = x[t] (16- or 32-bit elements, a copy)
+ *   cutb_moe_matmul   C[i] = f(W_e A[i]) for the rows i of every expert e; W stacks the experts' N rows; f = glu of
+ *       neighbouring outputs (C then has N / 2 columns) or the identity.  TC: bf16 A; SIMT: fp32 or bf16 A.
+ *       (the weighted sum of a token's rows is cutb_residual_norm's parts)
+ * One token, each call with an optional dense companion, so that both sublayers of a layer share two launches:
+ *   cutb_expert_up    C = Wd N(xd; xd_norm_w) (RMS norm; Wd null: none); ids, act [top][ff] = softmax weight * glu(W_gu,e x)
+ *   cutb_expert_down  C = Wd xd + sum_k W_down,ids[k] act[k]
+ */
+enum { CUTB_GLU_NONE = 0, CUTB_GLU_CLAMPED = 1 };
+typedef struct cutb_moe_desc {
+  uint32_t n_tokens, experts, top, K, N;
+  const float *logits;
+  uint64_t ld_logits;
+  float *weights;
+  uint32_t *ids, *slots, *offsets; /* ids [T][top]: the chosen experts, by falling logit */
+  int32_t a_dtype, c_dtype;
+  const void *A; /* cutb_moe_scatter: the tokens' rows; cutb_moe_matmul: the sorted rows */
+  uint64_t lda;
+  const void *W; /* bf16, rows of ldw elements (a multiple of 8, zero past K, 16-byte aligned) */
+  uint32_t ldw;
+  void *C;
+  uint64_t ldc;
+  int32_t glu;
+  float alpha, beta, limit;
+  int32_t variant; /* CUTB_DENSE_TC or CUTB_DENSE_SIMT */
+  int *status;
+} cutb_moe_desc;
+CUTB_API int cutb_moe_route(const cutb_moe_desc *desc, void *stream);
+CUTB_API int cutb_moe_scatter(const cutb_moe_desc *desc, void *stream);
+CUTB_API int cutb_moe_matmul(const cutb_moe_desc *desc, void *stream);
+
+typedef struct cutb_expert_desc {
+  uint32_t experts, top, width, ff;
+  const float *logits; /* cutb_expert_up */
+  uint32_t *ids;       /* written by cutb_expert_up, read by cutb_expert_down */
+  const void *W;       /* W_gu [experts * 2 ff][ldw], or W_down [experts * width][ldw] */
+  uint32_t ldw;
+  const float *x; /* cutb_expert_up: [width] */
+  float *act;     /* [top][ff] */
+  float alpha, beta, limit;
+  const void *Wd; /* dense companion, [Nd][ldwd] */
+  uint32_t Nd, Kd, ldwd;
+  const float *xd, *xd_norm_w;
+  float eps;
+  float *C; /* cutb_expert_up: [Nd]; cutb_expert_down: [width] (Nd = width with Wd) */
+  uint32_t flags;
+} cutb_expert_desc;
+CUTB_API int cutb_expert_up(const cutb_expert_desc *desc, void *stream);
+CUTB_API int cutb_expert_down(const cutb_expert_desc *desc, void *stream);
 
 CUTB_API int cutb_version(void);
 CUTB_API const char *cutb_status_string(int status);
