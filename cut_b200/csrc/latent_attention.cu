@@ -4,7 +4,11 @@
 //  * latent_kv_write_kernel: a batch of tokens into the cache, and the norm of the latent queries;
 //  * latent_attention_simt_kernel: the absorbed form (every head's query against the cache row itself) in fp32 arithmetic, for
 //    any size, either cache type, and any number of tokens.  For one token the keys are shared out over blocks, which leave
-//    partial sums; the values' mat-vec behind it merges them while it stages its input (head_matvec_kernel).
+//    partial sums; the values' mat-vec behind it merges them while it stages its input (head_matvec_kernel);
+//  * latent_prefill_tc_kernel: many tokens over expanded keys and values (a GEMM over the cache makes them), bf16.  A block of
+//    eight warps owns 128 consecutive tokens of one head; tiles of 64 keys -- the head's own part, and the shared rotated part
+//    straight from the cache -- stream through a two-deep cp.async ring, products are m16n8k16 warp MMAs with fp32
+//    accumulators, the softmax runs online.  The weights enter the value product as the sum of two bf16 terms.
 #include <cuda_bf16.h>
 
 #include "attn_common.cuh"
@@ -205,6 +209,207 @@ template <typename KV> __global__ void __launch_bounds__(LA_THREADS) latent_atte
   if (sp.part && tid < nh) sp.ml[(size_t)(h0 + tid) * sp.splits + split] = make_float2(head_m[tid], head_l[tid]);
 }
 
+// ---- expanded form on the tensor cores ---------------------------------------------------------------------------------
+constexpr int LP_BM = 128, LP_BN = 64, LP_THREADS = 256, LP_PAD = 8;
+
+template <int DK, int DV> __global__ void __launch_bounds__(LP_THREADS, 1) latent_prefill_tc_kernel(const cutb_latent_attn_desc d) {
+  constexpr int LK = DK + LP_PAD, LV = DV + LP_PAD, KS = DK / 16, KC = DK / 8, VC = DV / 8;
+  constexpr uint32_t KT = LP_BN * LK * 2, VT = LP_BN * LV * 2;
+  constexpr bool Q_IN_REGS = DK <= 128;
+  extern __shared__ __align__(16) uint8_t lp_smem[];
+  __nv_bfloat16 *Qs = reinterpret_cast<__nv_bfloat16 *>(lp_smem);
+  const uint32_t qs_u = smem_u32(lp_smem), k_u = qs_u + LP_BM * LK * 2, v_u = k_u + 2 * KT;
+
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  // later tokens (which see more keys) first
+  const uint32_t tok0 = (gridDim.y - 1 - blockIdx.y) * LP_BM, h = blockIdx.x;
+  pdl_enter();
+  const uint32_t p0 = (d.pos_ptr ? *d.pos_ptr : d.pos) + tok0, ntok = min((uint32_t)LP_BM, d.n_tokens - tok0);
+  if (p0 + ntok > d.max_pos) {  // no table rows: the cache write has done nothing for them either
+    if (d.status && tid == 0 && h == 0) atomicExch(d.status, (int)CUTB_ERR_INVALID);
+    return;
+  }
+  const uint32_t p_last = p0 + ntok - 1, t_end = p_last / LP_BN + 1, width = d.dim + d.rot_dim;
+  const __nv_bfloat16 *kbase = reinterpret_cast<const __nv_bfloat16 *>(d.k_exp) + (size_t)h * d.dim;
+  const __nv_bfloat16 *vbase = reinterpret_cast<const __nv_bfloat16 *>(d.v_exp) + (size_t)h * d.vdim;
+  const __nv_bfloat16 *rbase = reinterpret_cast<const __nv_bfloat16 *>(d.cache) + d.rot_at;
+  // Keys past the block's last token are zero (a weight of zero times a stray NaN would not be); so are columns past the head's.
+  auto load_tile = [&](uint32_t t, uint32_t buf) {
+    const uint32_t key0 = t * LP_BN;
+#pragma unroll
+    for (uint32_t i = tid; i < LP_BN * KC; i += LP_THREADS) {
+      const uint32_t r = i / KC, c = i % KC * 8, key = key0 + r;
+      const __nv_bfloat16 *src = c < d.dim ? kbase + key * d.ld_k + c : rbase + key * d.ld_cache + (c - d.dim);
+      const uint32_t off = buf * KT + (r * LK + c) * 2;
+      if (key <= p_last && c < width) cp_async16(k_u + off, src);
+      else *reinterpret_cast<uint4 *>(lp_smem + (k_u - qs_u) + off) = make_uint4(0, 0, 0, 0);
+    }
+#pragma unroll
+    for (uint32_t i = tid; i < LP_BN * VC; i += LP_THREADS) {
+      const uint32_t r = i / VC, c = i % VC * 8, key = key0 + r;
+      const uint32_t off = buf * VT + (r * LV + c) * 2;
+      if (key <= p_last && c < d.vdim) cp_async16(v_u + off, vbase + key * d.ld_v + c);
+      else *reinterpret_cast<uint4 *>(lp_smem + (v_u - qs_u) + off) = make_uint4(0, 0, 0, 0);
+    }
+    cp_async_commit();
+  };
+  load_tile(0, 0);
+
+  // queries: the rotated part turned at their own positions, rounded to bf16; pairs of neighbours
+  {
+    constexpr uint32_t PP = DK / 2;
+    const float *q0 = d.q + (size_t)tok0 * d.ldq + (size_t)h * width;
+    const uint32_t half = d.rot_dim / 2;
+#pragma unroll 4
+    for (uint32_t i = tid; i < LP_BM * PP; i += LP_THREADS) {
+      const uint32_t r = i / PP, e = i % PP * 2, rc = min(r, ntok - 1);  // (rows past the last token repeat it)
+      float u = 0.f, v = 0.f;
+      if (e < width) {
+        u = __ldg(q0 + rc * d.ldq + e), v = __ldg(q0 + rc * d.ldq + e + 1);
+        if (e >= d.dim) {
+          const size_t at = (size_t)(p0 + rc) * half + (e - d.dim) / 2;
+          const float c = __ldg(d.cos_table + at), s = __ldg(d.sin_table + at), u0 = u;
+          u = u0 * c - v * s, v = v * c + u0 * s;
+        }
+      }
+      *reinterpret_cast<uint32_t *>(Qs + r * LK + e) = pack_bf16(u, v);
+    }
+  }
+  __syncthreads();
+
+  const uint32_t g = lane >> 2, tg = lane & 3, mat = lane >> 3, mr = lane & 7;
+  const uint32_t q_row = warp * 16 + (mat & 1) * 8 + mr;
+  uint32_t qa[Q_IN_REGS ? KS : 1][4];
+  if constexpr (Q_IN_REGS) {
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks) ldsm_x4(qs_u + (q_row * LK + ks * 16 + (mat >> 1) * 8) * 2, qa[ks][0], qa[ks][1], qa[ks][2], qa[ks][3]);
+  }
+  const uint32_t row_lo = warp * 16 + g, row_hi = row_lo + 8;
+  const uint32_t pos_lo = p0 + row_lo, pos_hi = p0 + row_hi;          // (rows past ntok compute and are not stored)
+  const uint32_t wp_first = p0 + warp * 16, wp_last = wp_first + 15;  // this warp's positions
+  const float scale_log2 = d.scale * LA_LOG2E;
+
+  float o[DV / 8][4];
+#pragma unroll
+  for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  // running maxima (log2 units) and sums; a sink is a key without a value seen before all others
+  const float sink = d.sink ? __ldg(d.sink + h) * LA_LOG2E : LA_NEG;
+  float m_lo = sink, m_hi = sink, l_lo = 0.f, l_hi = 0.f;
+
+  for (uint32_t t = 0; t < t_end; ++t) {
+    const uint32_t buf = t & 1;
+    if (t + 1 < t_end) {
+      load_tile(t + 1, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const uint32_t kt_u = k_u + buf * KT, vt_u = v_u + buf * VT, key0 = t * LP_BN;
+    if (key0 <= wp_last) {  // this warp sees the tile
+      float s[LP_BN / 8][4];
+#pragma unroll
+      for (int j = 0; j < LP_BN / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < KS; ++ks) {
+        uint32_t (&a)[4] = qa[Q_IN_REGS ? ks : 0];
+        if constexpr (!Q_IN_REGS) ldsm_x4(qs_u + (q_row * LK + ks * 16 + (mat >> 1) * 8) * 2, a[0], a[1], a[2], a[3]);
+#pragma unroll
+        for (int j2 = 0; j2 < LP_BN / 16; ++j2) {
+          const uint32_t row = j2 * 16 + (mat >> 1) * 8 + mr, col = ks * 16 + (mat & 1) * 8;
+          uint32_t b0, b1, b2, b3;
+          ldsm_x4(kt_u + (row * LK + col) * 2, b0, b1, b2, b3);
+          mma_bf16(s[2 * j2], a, b0, b1);
+          mma_bf16(s[2 * j2 + 1], a, b2, b3);
+        }
+      }
+      float mx_lo = LA_NEG, mx_hi = LA_NEG;
+      const bool all = key0 + LP_BN - 1 <= wp_first;  // every key seen by every token of the warp
+#pragma unroll
+      for (int j = 0; j < LP_BN / 8; ++j) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const uint32_t key = key0 + j * 8 + 2 * tg + (e & 1), pos = e < 2 ? pos_lo : pos_hi;
+          const float v = all || key <= pos ? s[j][e] * scale_log2 : -INFINITY;
+          s[j][e] = v;
+          if (e < 2) mx_lo = fmaxf(mx_lo, v);
+          else mx_hi = fmaxf(mx_hi, v);
+        }
+      }
+      mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
+      mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+      mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
+      mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+      const float mn_lo = fmaxf(m_lo, mx_lo), mn_hi = fmaxf(m_hi, mx_hi);
+      const float al_lo = exp2f(m_lo - mn_lo), al_hi = exp2f(m_hi - mn_hi);
+      m_lo = mn_lo, m_hi = mn_hi;
+      float sum_lo = 0.f, sum_hi = 0.f;
+#pragma unroll
+      for (int j = 0; j < LP_BN / 8; ++j) {
+        s[j][0] = exp2f(s[j][0] - m_lo), s[j][1] = exp2f(s[j][1] - m_lo);
+        s[j][2] = exp2f(s[j][2] - m_hi), s[j][3] = exp2f(s[j][3] - m_hi);
+        sum_lo += s[j][0] + s[j][1];
+        sum_hi += s[j][2] + s[j][3];
+      }
+      l_lo = l_lo * al_lo + sum_lo, l_hi = l_hi * al_hi + sum_hi;
+#pragma unroll
+      for (int j = 0; j < DV / 8; ++j) o[j][0] *= al_lo, o[j][1] *= al_lo, o[j][2] *= al_hi, o[j][3] *= al_hi;
+#pragma unroll
+      for (int kk = 0; kk < LP_BN / 16; ++kk) {
+        uint32_t ph[4], pl[4];
+        split_bf16(s[2 * kk][0], s[2 * kk][1], ph[0], pl[0]);
+        split_bf16(s[2 * kk][2], s[2 * kk][3], ph[1], pl[1]);
+        split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], ph[2], pl[2]);
+        split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], ph[3], pl[3]);
+#pragma unroll
+        for (int jd2 = 0; jd2 < DV / 16; ++jd2) {
+          const uint32_t row = kk * 16 + (mat & 1) * 8 + mr, col = jd2 * 16 + (mat >> 1) * 8;
+          uint32_t b0, b1, b2, b3;
+          ldsm_x4_trans(vt_u + (row * LV + col) * 2, b0, b1, b2, b3);
+          mma_bf16(o[2 * jd2], ph, b0, b1);
+          mma_bf16(o[2 * jd2 + 1], ph, b2, b3);
+          mma_bf16(o[2 * jd2], pl, b0, b1);
+          mma_bf16(o[2 * jd2 + 1], pl, b2, b3);
+        }
+      }
+    }
+    __syncthreads();  // the tile is free for the copy issued two turns from now
+  }
+
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 1);
+  l_lo += __shfl_xor_sync(0xffffffffu, l_lo, 2);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
+  l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
+  if (d.sink) l_lo += exp2f(sink - m_lo), l_hi += exp2f(sink - m_hi);
+  const float inv_lo = 1.0f / l_lo, inv_hi = 1.0f / l_hi;
+#pragma unroll
+  for (int j = 0; j < DV / 8; ++j) {
+    const uint32_t c = 8 * j + 2 * tg;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const uint32_t r = e < 2 ? row_lo : row_hi, cc = c + (e & 1);
+      if (r < ntok && cc < d.vdim)
+        store_out(d.out, d.out_dtype == CUTB_BF16, (size_t)(tok0 + r) * d.ldo + (size_t)h * d.vdim + cc, o[j][e] * (e < 2 ? inv_lo : inv_hi));
+    }
+  }
+}
+
+template <int DK, int DV> int lp_launch(const cutb_latent_attn_desc &d, cudaStream_t stream) {
+  constexpr size_t smem = ((size_t)(LP_BM + 2 * LP_BN) * (DK + LP_PAD) + (size_t)2 * LP_BN * (DV + LP_PAD)) * 2;
+  CUTB_CUDA_TRY(cudaFuncSetAttribute(latent_prefill_tc_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  CUTB_CUDA_TRY(launch_pdl(latent_prefill_tc_kernel<DK, DV>, dim3(d.n_heads, (d.n_tokens + LP_BM - 1) / LP_BM), dim3(LP_THREADS), smem, stream, d));
+  return CUTB_OK;
+}
+template <int DV> int lp_dispatch(const cutb_latent_attn_desc &d, cudaStream_t stream) {
+  const uint32_t width = d.dim + d.rot_dim;
+  if constexpr (DV <= 128) {
+    if (width <= 64) return lp_launch<64, DV>(d, stream);
+    if (width <= 128) return lp_launch<128, DV>(d, stream);
+    if (width <= 192) return lp_launch<192, DV>(d, stream);
+  }
+  return lp_launch<256, DV>(d, stream);
+}
+
 LatentSplit split_of(const cutb_latent_attn_desc &d) {
   LatentSplit s{};
   s.splits = latent_splits(d), s.ld = (d.rank + 3) / 4 * 4;
@@ -255,7 +460,14 @@ int latent_values_launch(const cutb_latent_attn_desc &d, cudaStream_t stream) {
   return head_matvec_launch(h, stream);
 }
 
-bool latent_prefill_supported(const cutb_latent_attn_desc &) { return false; }
-int latent_prefill_launch(const cutb_latent_attn_desc &, cudaStream_t) { return CUTB_ERR_UNSUPPORTED; }
+bool latent_prefill_supported(const cutb_latent_attn_desc &d) {
+  return d.kv_dtype == CUTB_BF16 && d.dim % 8 == 0 && d.rot_dim % 8 == 0 && d.vdim % 8 == 0 && d.vdim > 0 && d.dim + d.rot_dim > 0 &&
+         d.dim + d.rot_dim <= 256 && d.vdim <= 256 && d.n_heads <= 0x7fffffffu && (d.n_tokens + LP_BM - 1) / LP_BM <= 65535;
+}
+
+int latent_prefill_launch(const cutb_latent_attn_desc &d, cudaStream_t stream) {
+  if (d.vdim <= 64) return lp_dispatch<64>(d, stream);
+  return d.vdim <= 128 ? lp_dispatch<128>(d, stream) : lp_dispatch<256>(d, stream);
+}
 
 }  // namespace cutb

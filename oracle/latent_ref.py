@@ -77,6 +77,12 @@ def choose_experts(z, top):
     return ids, e / e.sum()
 
 
+def choice_margin(logits, top):
+    """How far the last chosen logit lies above the first one left out, in standard deviations of a token's logits."""
+    z = -np.sort(-logits, axis=-1)
+    return np.full(len(z), np.inf) if top == z.shape[1] else (z[:, top - 1] - z[:, top]) / z.std(axis=-1)
+
+
 def mixture(h, logits, gate, up, down, top, limit):
     """h [T, W]; logits [T, E]; gate / up / down: lists of matrices."""
     out = np.zeros_like(h)
@@ -98,6 +104,10 @@ class LatentReference:
     def reset(self):
         self.pos, self.c, self.r = 0, {}, {}
 
+    def forget(self, n):
+        """Back to the first n positions."""
+        self.pos, self.c, self.r = n, {i: a[:n] for i, a in self.c.items()}, {i: a[:n] for i, a in self.r.items()}
+
     def attention(self, i, m, h, positions):
         w, p, eps, T = self.w, f"l{i}.mix.", self.cfg["norm"]["eps"], len(h)
         H, dim, rank = m["heads"], m["dim"], m["kv_rank"]
@@ -117,10 +127,13 @@ class LatentReference:
         w, p, E = self.w, f"l{i}.mlp.", f["router"]["experts"]
         part = lambda n: [w[f"{p}e{e}.{n}"] for e in range(E)]
         logits = h @ w[p + "router"].T + w[p + "router.b"]
+        self.margin = np.minimum(self.margin, choice_margin(logits, f["router"]["top"]))
         return mixture(h, logits, part("gate"), part("up"), part("down"), f["router"]["top"], f["expert"]["limit"])
 
     def run(self, tokens, layers_out=None):
-        """Logits [T, vocab] of the next tokens; appends the residual after every layer to `layers_out`."""
+        """Logits [T, vocab] of the next tokens; appends the residual after every layer to `layers_out`.  `margin` [T] is left as the
+        closest call any router had on each token."""
+        self.margin = np.full(len(tokens), np.inf)
         cfg, w, eps = self.cfg, self.w, self.cfg["norm"]["eps"]
         positions = np.arange(self.pos, self.pos + len(tokens))
         x = w["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]

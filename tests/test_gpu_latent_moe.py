@@ -1,0 +1,649 @@
+"""Latent attention, mixtures of experts and parallel layers on the device: every mechanism alone against its oracle, then whole
+models in both element types -- prompts, token-by-token decoding, portions, places that are used again, sequences that
+alternate -- and greedy generation through the queue, the trace replay and the command line.
+
+Limits are relative to the rms of the wanted values: 32-bit mode 3e-5, bf16 mode 3e-2 for whole models."""
+import json
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+from cut_b200 import _lib as L
+from cut_b200 import layer_list, ops
+from cut_b200.decoding import RequestQueue
+from cut_b200.layer_list import Rotation, pad, rotation_tables
+from cut_b200.models import load_model
+from cut_b200.trace import replay
+from oracle import latent_ref as R
+from tests.layer_list_util import row_errors
+from tests.lenesun_util import (CONFIGS, SandwichReference, bf16, build_decoder, config, layer, random_weights, safe_tokens, sandwich_decoder,
+                                save_model)
+
+pytestmark = pytest.mark.gpu
+ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+LIMIT = {"float32": 3e-5, "bfloat16": 3e-2}
+
+
+def dev(a, dtype=torch.float32):
+    return torch.from_numpy(np.ascontiguousarray(a)).to(device="cuda", dtype=dtype)
+
+
+def ints(a):
+    return torch.tensor(np.asarray(a), dtype=torch.int32, device="cuda")
+
+
+def rel(got, want):
+    got, want = np.asarray(got.float().cpu() if torch.is_tensor(got) else got, np.float64), np.asarray(want, np.float64)
+    return float(np.linalg.norm(got - want) / np.linalg.norm(want))
+
+
+def padded(a, m=8):
+    out = np.zeros(a.shape[:-1] + (pad(a.shape[-1], m),), np.float32)
+    out[..., : a.shape[-1]] = a
+    return out
+
+
+def cuts_of(T, sizes):
+    cuts = [0]
+    while cuts[-1] < T:
+        cuts.append(min(T, cuts[-1] + sizes[(len(cuts) - 1) % len(sizes)]))
+    return cuts
+
+
+# ---- norms, residual, embedding ----------------------------------------------------------------------------------------
+@pytest.mark.parametrize("dim", [128, 96, 70, 35, 1280, 4096, 8192, 5000])
+@pytest.mark.parametrize("center", [True, False])
+def test_plain_residual_with_gathered_rows_and_centred_norm(dim, center):
+    rng = np.random.default_rng(dim)
+    rows, n, eps, scale = 5, 3, 1e-3, 0.37
+    x, y, m = rng.standard_normal((rows, dim)) + 30.0, rng.standard_normal((rows, dim)), rng.standard_normal((11, dim))  # (a mean far above the spread)
+    x = x.astype(np.float32).astype(np.float64)
+    w, wp = 1 + 0.3 * rng.standard_normal(dim), 1 + 0.3 * rng.standard_normal(dim)
+    at, pw = rng.integers(0, 11, (rows, n)), rng.uniform(0, 1, (rows, n))
+    norm = R.layer_norm if center else R.rms_norm
+    m16 = bf16(m)
+    ld, tx, ty = pad(dim, 8), dev(padded(x)), dev(padded(y))
+    for post in (None, wp):
+        for with_y, mt in ((True, None), (True, torch.float32), (False, torch.bfloat16), (False, None)):
+            add = (y if with_y else 0.0) + (0.0 if mt is None else np.einsum("rk,rkd->rd", pw, (m16 if mt == torch.bfloat16 else m)[at]))
+            if post is not None and not np.isscalar(add):
+                add = norm(add, post, eps)
+            nx = x + scale * add
+            want = norm(nx, w, eps)
+            parts = None if mt is None else (dev(padded(m), mt), ints(at), dev(pw))
+            kw = dict(dim=dim, y=ty if with_y else None, post_w=None if post is None else dev(post), center=center, y_scale=scale, parts=parts)
+            for dt, lim in ((torch.float32, 1e-5), (torch.bfloat16, 4e-3)):
+                keep, h = tx.clone(), torch.zeros((rows, ld), device="cuda", dtype=dt)
+                ops.residual_norm(keep, dev(w), 1, eps, x_out=keep, out=h, **kw)
+                assert rel(h[:, :dim], want) < lim and rel(keep[:, :dim], nx) < 1e-6
+            idx = ints([4, 0, 4])
+            h = ops.residual_norm(tx, dev(w), 1, eps, row_index=idx, **kw)
+            assert rel(h[:, :dim], want[[4, 0, 4]]) < 1e-5 and rel(tx[:, :dim], x) < 1e-7
+    # the mat-vec that makes its input the same way, and hands the normed row on
+    W, N = bf16(rng.standard_normal((24, dim)) / np.sqrt(dim)), 24
+    nx = x + scale * y
+    want = norm(nx, w, eps)
+    out, xo, ho = torch.zeros((1, N), device="cuda"), torch.zeros(ld, device="cuda"), torch.zeros(ld, device="cuda")
+    d = ops.dense_desc(None, dev(padded(W), torch.bfloat16), dim, out, N=N)
+    norm_w = dev(w)
+    ops.stage_input(d, tx[3], norm_w, 1, eps, ty[3], None, xo, center=center, y_scale=scale, norm_out=ho)
+    ops.dense_matmul(d)
+    assert rel(out[0], W.astype(np.float64) @ want[3]) < 2e-5 and rel(xo[:dim], nx[3]) < 1e-6 and rel(ho[:dim], want[3]) < 1e-5
+
+
+def test_scaled_embedding():
+    rng = np.random.default_rng(1)
+    for dim in (40, 30):
+        e, toks = bf16(rng.standard_normal((61, dim))), rng.integers(0, 61, 50)
+        got = ops.embedding_bigram(ints(toks), dev(e, torch.bfloat16), scale=2.75)
+        assert np.allclose(got.cpu().numpy(), e[toks] * 2.75, rtol=1e-6)
+
+
+# ---- a product per head --------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("heads,K,N,step", [(3, 24, 48, 40), (5, 9, 35, 15), (8, 128, 512, 192), (2, 512, 128, 512), (40, 72, 3, 80), (16, 1000, 64, 1000)])
+def test_product_per_head(heads, K, N, step):
+    rng = np.random.default_rng(K)
+    T = 37
+    A, W = rng.standard_normal((T, heads * step)).astype(np.float32), bf16(rng.standard_normal((heads, N, K)) / np.sqrt(K))
+    want = np.einsum("thk,hnk->thn", A.reshape(T, heads, step)[:, :, :K].astype(np.float64), W).reshape(T, -1)
+    w, a = dev(padded(W).reshape(heads * N, -1), torch.bfloat16), dev(padded(A))
+    for rows in (1, 2, T):
+        out = torch.full((rows, pad(heads * N, 8) + 8), 7.0, device="cuda")
+        ops.dense_matmul(ops.batch_desc(a[:rows], w, K, out, heads, step, N))
+        assert rel(out[:, : heads * N], want[:rows]) < 2e-6 and bool((out[:, heads * N:] == 7.0).all()), rows
+
+
+# ---- mixture of experts ----------------------------------------------------------------------------------------------------
+class Moe:
+    def __init__(self, T, E, top, width, ff, limit=1.0, seed=0):
+        rng = np.random.default_rng(seed + E)
+        self.T, self.E, self.top, self.width, self.ff, self.limit = T, E, top, width, ff, limit
+        self.h = bf16(rng.standard_normal((T, width)))
+        self.z = rng.standard_normal((T, E)).astype(np.float32)
+        self.gate, self.up = (bf16(rng.standard_normal((E, ff, width)) * 2 / np.sqrt(width)) for _ in range(2))
+        self.down = bf16(rng.standard_normal((E, width, ff)) / np.sqrt(ff))
+        self.gu = dev(padded(np.stack([self.gate, self.up], axis=2).reshape(E * 2 * ff, width)), torch.bfloat16)
+        self.dn = dev(padded(self.down.reshape(E * width, ff)), torch.bfloat16)
+        self.glu = dict(alpha=1.702, beta=1.0, limit=limit)
+
+    def want(self, t=None, **change):
+        rows = slice(None) if t is None else slice(t, t + 1)
+        f64 = lambda a: [m.astype(np.float64) for m in a]
+        k = {"top": self.top, "limit": self.limit, **change}
+        return R.mixture(self.h[rows].astype(np.float64), self.z[rows].astype(np.float64), f64(self.gate), f64(self.up), f64(self.down), k["top"], k["limit"])
+
+    def route(self):
+        e = lambda *s, t=torch.int32: torch.full(s, -7, dtype=t, device="cuda")
+        self.weights, self.ids, self.slots, self.offsets = e(self.T, self.top, t=torch.float32), e(self.T, self.top), e(self.T, self.top), e(self.E + 1)
+        z = dev(padded(self.z, 4))
+        ops.launch_layer_op("cutb_moe_route", ops.moe_route_desc(z, self.E, self.top, self.weights, self.ids, self.slots, self.offsets))
+        torch.cuda.synchronize()
+
+
+MOE = [(1, 4, 2, 40, 24), (2, 8, 3, 70, 13), (33, 6, 6, 64, 40), (300, 16, 4, 128, 96), (700, 5, 1, 96, 64), (40, 200, 7, 72, 16), (9, 1, 1, 24, 8),
+       (513, 64, 8, 256, 136), (20, 37, 2, 512, 300)]
+
+
+@pytest.mark.parametrize("T,E,top,width,ff", MOE)
+def test_routing_sorts_choices_by_expert_and_token(T, E, top, width, ff):
+    m = Moe(T, E, top, width, ff)
+    m.z[T // 2] = m.z[T // 2, 0]  # a token without preferences: the lower experts
+    m.route()
+    chosen = [R.choose_experts(z.astype(np.float64), top) for z in m.z]
+    ids = np.array([c[0] for c in chosen])
+    assert np.array_equal(m.ids.cpu().numpy(), ids)
+    assert np.allclose(m.weights.cpu().numpy(), [c[1] for c in chosen], rtol=1e-5)
+    flat = ids.reshape(-1)
+    assert np.array_equal(m.offsets.cpu().numpy(), [np.sum(flat < e) for e in range(E + 1)])
+    place = np.empty(T * top, int)
+    place[np.argsort(flat, kind="stable")] = np.arange(T * top)
+    assert np.array_equal(m.slots.cpu().numpy().reshape(-1), place)
+
+
+@pytest.mark.parametrize("T,E,top,width,ff", MOE)
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_grouped_products(T, E, top, width, ff, dtype):
+    m = Moe(T, E, top, width, ff, limit=0.8)
+    if E > 4:
+        m.z[:, 2] -= 50.0  # an expert that nobody chooses (unless all are chosen), and a crowded one
+        m.z[:, 3] += 3.0
+    m.route()
+    want = m.want()
+    if top < E:
+        assert rel(m.want(top=top + 1), want) > 0.01
+    assert rel(m.want(limit=50.0), want) > 0.01  # (the clamps matter)
+    x = dev(padded(m.h), dtype)
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
+    for variant in ([L.DENSE_SIMT] if dtype == torch.float32 else [L.DENSE_TC, L.DENSE_SIMT]):
+        for act_ld in (pad(ff, 8), pad(ff, 8) + 16):
+            rows = T * top
+            srt = torch.zeros((rows, x.shape[1]), device="cuda", dtype=dtype)
+            act = torch.full((rows, act_ld), 7.0, device="cuda", dtype=dtype)
+            out = torch.full((rows, x.shape[1]), 7.0, device="cuda", dtype=dtype)
+            ops.launch_layer_op("cutb_moe_scatter", ops.moe_scatter_desc(x, width, m.slots, E, srt))
+            group = dict(offsets=m.offsets, experts=E, tokens=T, top=top, variant=variant, status=status)
+            ops.launch_layer_op("cutb_moe_matmul", ops.moe_matmul_desc(srt, m.gu, width, out=act, glu=L.GLU_CLAMPED, **m.glu, **group))
+            ops.launch_layer_op("cutb_moe_matmul", ops.moe_matmul_desc(act, m.dn, ff, out=out, **group))
+            assert bool((act[:, ff:] == 7.0).all()) and bool((out[:, width:] == 7.0).all())
+            assert torch.equal(srt[m.slots.long().reshape(-1), :width], x[:, :width].repeat_interleave(top, 0))
+            got = (out[m.slots.long()][:, :, :width].float() * m.weights[:, :, None]).sum(1)
+            assert rel(got, want) < (3e-6 if dtype == torch.float32 else 8e-3), (variant, act_ld)
+    assert int(status.item()) == 0
+
+
+@pytest.mark.parametrize("T,E,top,width,ff", MOE)
+@pytest.mark.parametrize("dense", [False, True])
+def test_expert_matvecs(T, E, top, width, ff, dense):
+    m, rng = Moe(T, E, top, width, ff, limit=0.8), np.random.default_rng(7)
+    for Nd, Kd, normed in ((50, 24, False), (129, 256, True), (3, 21, True)) if dense else ((0, 0, False),):
+        for t in {0, T - 1}:
+            want = m.want(t)[0]
+            act, ids = torch.zeros(top * ff, device="cuda"), torch.full((top,), -1, dtype=torch.int32, device="cuda")
+            z, x = dev(m.z[t]), dev(m.h[t])
+            more, keep = {}, []
+            if dense:
+                Wd, xd, wn = bf16(rng.standard_normal((Nd, Kd)) / np.sqrt(Kd)), rng.standard_normal(Kd).astype(np.float32), 1 + 0.3 * rng.standard_normal(Kd)
+                q = torch.full((Nd + 1,), 7.0, device="cuda")
+                keep = [dev(padded(Wd), torch.bfloat16), dev(xd), dev(wn)]
+                more = dict(dense=keep[0], dense_K=Kd, xd=keep[1], xd_norm_w=keep[2] if normed else None, eps=1e-3, out=q)
+            ops.launch_layer_op("cutb_expert_up", ops.expert_desc(E, top, width, ff, m.gu, ids, act, logits=z, x=x, **m.glu, **more))
+            if dense:
+                xn = R.rms_norm(xd.astype(np.float64), wn, 1e-3) if normed else xd.astype(np.float64)
+                assert rel(q[:Nd], Wd @ xn) < 3e-6 and float(q[Nd]) == 7.0
+            assert ids.cpu().tolist() == R.choose_experts(m.z[t], top)[0].tolist()
+            y = torch.full((width + 1,), 7.0, device="cuda")
+            if dense:
+                Wo, a = bf16(rng.standard_normal((width, Kd)) / np.sqrt(Kd)), rng.standard_normal(Kd).astype(np.float32)
+                want = want + Wo.astype(np.float64) @ a
+                keep = [dev(padded(Wo), torch.bfloat16), dev(a)]
+                more = dict(dense=keep[0], dense_K=Kd, xd=keep[1])
+            ops.launch_layer_op("cutb_expert_down", ops.expert_desc(E, top, width, ff, m.dn, ids, act, **{**more, "out": y}))
+            assert rel(y[:width], want) < 3e-6 and float(y[width]) == 7.0
+
+
+# ---- latent attention ------------------------------------------------------------------------------------------------------
+class Latent:
+    """Random queries and latents of one layer, its oracle, and the device side over a cache."""
+
+    def __init__(self, H, dim, rot, vdim, rank, T, dtype, *, scale=None, sink=True, seed=0, base=1000.0, q_rank=40):
+        rng = np.random.default_rng(seed + H + rank)
+        self.p, self.T, self.dtype, self.base, self.eps = (H, dim, rot, vdim, rank), T, dtype, base, 1e-3
+        self.scale = 1.2 * (dim + rot) ** -0.5 if scale is None else scale
+        self.q = bf16(rng.standard_normal((T, H * (dim + rot))))
+        self.lat = bf16(rng.standard_normal((T, rank + rot)) * 3)
+        self.cq, self.cq_w = rng.standard_normal((T, q_rank)).astype(np.float32), 1 + 0.3 * rng.standard_normal(q_rank)
+        self.lat_w = bf16(1 + 0.3 * rng.standard_normal(rank))
+        self.uk, self.uv = (bf16(rng.standard_normal((H * n, rank)) * s / np.sqrt(rank)) for n, s in ((dim, 1.5), (vdim, 1.0)))
+        self.sink = bf16(rng.standard_normal(H) * 2 + 1.5) if sink else None
+        self.cos, self.sin = (torch.from_numpy(t).cuda() for t in rotation_tables(Rotation(base, rot), T))
+        self.status = torch.zeros(1, dtype=torch.int32, device="cuda")
+        self.cache = torch.zeros((pad(T, 64), pad(rank, 8) + pad(rot, 8)), device="cuda", dtype=dtype)
+        self.w_uv = dev(padded(self.uv), torch.bfloat16)
+        absorb = self.uk.reshape(H, dim, rank).transpose(0, 2, 1).reshape(H * rank, dim)
+        self.absorb = dev(padded(absorb), torch.bfloat16)
+        self.expand = dev(padded(np.concatenate([self.uk, self.uv])), torch.bfloat16)
+        self.keep = []
+
+    def parts(self):
+        H, dim, rot, vdim, rank = self.p
+        pos = np.arange(self.T)
+        q = self.q.astype(np.float64).reshape(self.T, H, dim + rot)
+        q = np.concatenate([q[:, :, :dim], R.turn_pairs(q[:, :, dim:], pos, self.base)], axis=2)
+        lat = self.lat.astype(np.float64)
+        return q, R.rms_norm(lat[:, :rank], self.lat_w, self.eps), R.turn_pairs(lat[:, rank:], pos, self.base)
+
+    def want(self, sink=True):
+        q, c, r = self.parts()
+        k, v = R.latent_keys_values(c, r, self.uk.astype(np.float64), self.uv.astype(np.float64), self.p[0])
+        return R.sink_attention(q, k, v, 0, self.scale, self.sink if sink else None)
+
+    def desc(self, a, b, **tensors):
+        H, dim, rot, vdim, rank = self.p
+        sink = dev(self.sink) if self.sink is not None else None
+        self.keep += [sink, tensors]  # (a descriptor holds addresses only)
+        return ops.latent_desc(self.cache, H, dim, rot, vdim, rank, scale=self.scale, eps=self.eps, max_pos=self.T, n_tokens=b - a, cos_t=self.cos,
+                               sin_t=self.sin, sink=sink, pos=a, status=self.status, **tensors)
+
+    def own(self, a, b):
+        return dict(lat=dev(padded(self.lat[a:b], 4)), lat_norm_w=dev(self.lat_w))
+
+    def write(self, a, b):
+        cq_out = torch.zeros((b - a, 48), device="cuda", dtype=self.dtype)
+        ops.launch_layer_op("cutb_latent_kv_write", self.desc(a, b, cq=dev(self.cq[a:b]), cq_norm_w=dev(self.cq_w), cq_out=cq_out, **self.own(a, b)))
+        return cq_out
+
+    def run(self, cuts, decode_from=None, expanded=False, own=True):
+        """Portions between the cuts (absorbed or expanded), then tokens alone; own: a token's launch makes its cache row."""
+        H, dim, rot, vdim, rank = self.p
+        out = torch.zeros((self.T, H * vdim), device="cuda")
+        for a, b in zip(cuts, cuts[1:]):
+            self.write(a, b)
+            if b - a == 1:
+                self.one(a, out, {})
+                continue
+            q = dev(self.q[a:b])
+            if expanded:
+                n = self.expand.shape[0]
+                exp = torch.full((pad(b, 64), pad(n, 8)), float("nan"), device="cuda", dtype=torch.bfloat16)
+                ops.dense_matmul(ops.dense_desc(self.cache[:b], self.expand, rank, exp, variant=L.DENSE_TC, N=n))
+                o = torch.full((b - a, pad(H * vdim, 8) + 8), 7.0, device="cuda")
+                ops.launch_layer_op("cutb_latent_prefill", self.desc(a, b, q=q, k_exp=exp, v_exp=exp[:, H * dim:], out=o))
+                assert bool((o[:, H * vdim:] == 7.0).all())
+                out[a:b] = o[:, : H * vdim]
+            else:
+                qa, lat = (torch.zeros((b - a, H * rank), device="cuda") for _ in range(2))
+                ops.dense_matmul(self.heads(q, self.absorb, dim, qa, dim + rot, rank))
+                ops.launch_layer_op("cutb_latent_attention", self.desc(a, b, q=q, qa=qa, out=lat))
+                ops.dense_matmul(self.heads(lat, self.w_uv, rank, out[a:b], rank, vdim))
+        for a in range(decode_from if decode_from is not None else self.T, self.T):
+            if not own:
+                self.write(a, a + 1)
+            self.one(a, out, self.own(a, a + 1) if own else {})
+        torch.cuda.synchronize()
+        assert int(self.status.item()) == 0
+        return out.cpu().numpy().astype(np.float64)
+
+    def heads(self, a, w, K, out, a_step, c_step):
+        if self.p[0] == 1:
+            return ops.dense_desc(a, w, K, out, variant=L.DENSE_SIMT, N=w.shape[0])
+        return ops.batch_desc(a, w, K, out, self.p[0], a_step, c_step)
+
+    def one(self, a, out, own):
+        H, dim, rot, vdim, rank = self.p
+        q, qa = dev(self.q[a:a + 1]), torch.zeros((1, H * rank), device="cuda")
+        ops.dense_matmul(self.heads(q, self.absorb, dim, qa, dim + rot, rank))
+        ws = torch.full((ops.latent_workspace_bytes(self.desc(a, a + 1)) // 4,), float("nan"), device="cuda")
+        ops.launch_layer_op("cutb_latent_attention", self.desc(a, a + 1, q=q, qa=qa, workspace=ws, **own))
+        ops.launch_layer_op("cutb_latent_values", self.desc(a, a + 1, out=out[a:a + 1], workspace=ws, w_uv=self.w_uv))
+
+
+LATENT = [(3, 24, 16, 40, 48, 150), (1, 10, 6, 7, 35, 70), (5, 8, 8, 8, 72, 300), (16, 128, 64, 128, 512, 200), (2, 192, 64, 200, 160, 140),
+          (33, 16, 0, 24, 64, 130), (4, 3, 2, 5, 9, 66), (2, 64, 32, 96, 1000, 90), (20, 64, 64, 64, 256, 260), (7, 40, 24, 16, 136, 129)]
+
+
+@pytest.mark.parametrize("H,dim,rot,vdim,rank,T", LATENT)
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_latent_cache_rows_and_query_norm(H, dim, rot, vdim, rank, T, dtype):
+    a = Latent(H, dim, rot, vdim, rank, T, dtype)
+    lim = 2e-6 if dtype == torch.float32 else 4e-3
+    cq = a.write(0, T // 2)
+    assert rel(cq[:, :40], R.rms_norm(a.cq[: T // 2].astype(np.float64), a.cq_w, a.eps)) < lim and not cq[:, 40:].any()
+    a.write(T // 2, T)
+    _, c, r = a.parts()
+    at = pad(rank, 8)
+    assert rel(a.cache[:T, :rank], c) < lim and not a.cache[:, rank:at].any() and not a.cache[T:].any()
+    if rot:
+        assert rel(a.cache[:T, at: at + rot], r) < lim and not a.cache[:, at + rot:].any()
+
+
+@pytest.mark.parametrize("H,dim,rot,vdim,rank,T", LATENT)
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_latent_attention_portions_and_decode(H, dim, rot, vdim, rank, T, dtype):
+    lim = 5e-6 if dtype == torch.float32 else 8e-3
+    for sink in (True, False):
+        make = lambda: Latent(H, dim, rot, vdim, rank, T, dtype, sink=sink)
+        want = make().want()
+        assert rel(make().run([0, T]), want) < lim
+        cuts = cuts_of(T, [2, 40, 1, 3, 17, 64, 2])
+        assert rel(make().run(cuts), want) < lim
+        start = [c for c in cuts if c < T // 3] + [T // 3]
+        assert rel(make().run(start, decode_from=T // 3), want) < lim
+        assert rel(make().run([0], decode_from=0, own=False), want) < lim  # rows already cached, as a layer that reads another's finds them
+        if dtype == torch.bfloat16 and dim % 8 == rot % 8 == vdim % 8 == 0:
+            assert rel(make().run([0, T], expanded=True), want) < lim
+            assert rel(make().run(cuts, expanded=True), want) < lim
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_one_key_that_stands_out_is_found_wherever_it_lies(dtype):
+    """One key whose score is far above all others at a time, around the borders of tiles, turns and shares of the context; every
+    later query must see it and no earlier one, in prompts, in portions and in decoding."""
+    H, dim, rot, vdim, rank, T = 4, 32, 16, 32, 64, 330
+    lim = 5e-6 if dtype == torch.float32 else 8e-3
+    for at in (0, 1, 31, 32, 63, 64, 65, 127, 128, 255, 256, 328):
+        def make(at=at):
+            a = Latent(H, dim, rot, vdim, rank, T, dtype, scale=0.25, sink=True, base=1e9)
+            a.q[:] = bf16(0.05 * a.q)
+            q = a.q.reshape(T, H, dim + rot)
+            q[:, :, dim:] = 0.0
+            q[:, :, dim + 14] = 8.0  # (the slowest pair: hardly turned)
+            a.lat[:, rank:] = 0.0
+            a.lat[at, rank + 14] = 8.0  # its score: 16
+            return a
+        want = make().want()
+        assert rel(make(at + 1 if at < 300 else at - 1).want()[at + 1:], want[at + 1:]) > 0.2  # (the neighbour's value is another)
+        assert rel(make().run([0, T]), want) < lim, at
+        assert rel(make().run([0, at - 1, at + 2, T] if 2 < at < T - 4 else [0, 2, T]), want) < lim, at
+        assert rel(make().run([0, 3], decode_from=3), want) < lim, at
+        if dtype == torch.bfloat16:
+            assert rel(make().run([0, T], expanded=True), want) < lim, at
+            assert rel(make().run([0, 40, 104, 129, T], expanded=True), want) < lim, at
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_learned_sinks_take_their_weight_head_by_head(dtype):
+    a = Latent(3, 16, 8, 16, 40, 80, dtype, scale=0.01)
+    a.sink = bf16(np.array([-30.0, 5.0, 60.0]))  # none of it, most of it, all of it
+    want = a.want()
+    heads = np.abs(want.reshape(80, 3, 16)).max(axis=(0, 2))
+    assert heads[2] < 1e-20 < 0.01 < heads[0] and rel(a.want(sink=False), want) > 0.1
+    lim = 5e-6 if dtype == torch.float32 else 8e-3
+    assert rel(a.run([0, 80]), want) < lim and rel(a.run([0, 5], decode_from=5), want) < lim
+    if dtype == torch.bfloat16:
+        assert rel(a.run([0, 80], expanded=True), want) < lim
+
+
+def test_positions_past_the_cache_are_reported_and_touch_nothing():
+    a = Latent(2, 16, 8, 16, 40, 60, torch.bfloat16)
+    d = a.desc(0, 4, **a.own(0, 4))
+    d.max_pos, d.pos = 50, 48
+    ops.launch_layer_op("cutb_latent_kv_write", d)
+    torch.cuda.synchronize()
+    assert int(a.status.item()) == L.ERR_INVALID
+    assert bool(a.cache[48:50].any()) and not a.cache[50:].any() and not a.cache[:48].any()
+    out, q = torch.zeros((4, 80), device="cuda"), torch.zeros((4, 80), device="cuda")
+    exp = torch.zeros((64, 64), device="cuda", dtype=torch.bfloat16)
+    for name, d in (("cutb_latent_attention", a.desc(0, 4, q=q, qa=q, out=out)), ("cutb_latent_prefill", a.desc(0, 4, q=q, k_exp=exp, v_exp=exp[:, 32:], out=out))):
+        a.status.zero_()
+        d.max_pos, d.pos = 50, 50
+        ops.launch_layer_op(name, d)
+        torch.cuda.synchronize()
+        assert int(a.status.item()) == L.ERR_INVALID and not out.any()
+    ws = torch.zeros(4096, device="cuda")
+    d = a.desc(0, 1, q=q, qa=q, workspace=ws, **a.own(0, 1))
+    d.max_pos, d.pos = 50, 50
+    a.status.zero_()
+    ops.launch_layer_op("cutb_latent_attention", d)
+    torch.cuda.synchronize()
+    assert int(a.status.item()) == L.ERR_INVALID and not ws.any() and not a.cache[50:].any()
+
+
+# ---- whole models ------------------------------------------------------------------------------------------------------------
+_MODELS = {}
+
+
+def reference(name, sandwich=False):
+    """(configuration, weights, tokens, logits, residuals) of a fixed sequence."""
+    key = (name, sandwich)
+    if key not in _MODELS:
+        cfg = CONFIGS[name]
+        w = random_weights(cfg, sum(map(ord, name)))
+        if sandwich:
+            rng = np.random.default_rng(5)
+            w["head"] = bf16(rng.standard_normal((cfg["vocab"], cfg["width"])) / np.sqrt(cfg["width"]))
+            for i in range(len(cfg["layers"])):
+                w.update({f"l{i}.{n}": bf16(1 + 0.2 * rng.standard_normal(cfg["width"])) for n in ("norm1b", "norm2", "norm2b")})
+        ref = (SandwichReference if sandwich else R.LatentReference)(cfg, w)
+        toks, trace = safe_tokens(ref, 230, 3), []
+        _MODELS[key] = (cfg, w, toks, ref.run(toks, trace), trace)
+    return _MODELS[key]
+
+
+def model(name, dtype, sandwich=False, **options):
+    cfg, w, toks, want, trace = reference(name, sandwich)
+    return toks, want, trace, (sandwich_decoder if sandwich else build_decoder)(cfg, w, dtype, **{"max_seq": 256, **options})
+
+
+def feed(dec, toks, cuts, seq=None, batched=False):
+    s = dec.open() if seq is None else seq
+    rows = []
+    for a, b in zip(cuts, cuts[1:]):
+        rows.append(dec.forward(s, toks[a:b], list(range(b - a)), batched=batched).cpu().numpy())
+    dec.check_status()
+    if seq is None:
+        dec.close(s)
+    return np.concatenate(rows)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name,sandwich", [(n, False) for n in CONFIGS] + [("mixed", True), ("odd", True)])
+def test_model_whole_portions_and_token_by_token(name, sandwich, dtype):
+    toks, want, trace, dec = model(name, dtype, sandwich)
+    T, lim = len(toks), LIMIT[dtype]
+    got = []
+    s = dec.open()
+    whole = dec.forward(s, toks, list(range(T)), trace=got).cpu().numpy()
+    dec.close(s)
+    assert len(got) == len(trace)
+    for i, (g, t) in enumerate(zip(got, trace)):
+        assert rel(g, t) < lim, f"residual after layer {i}"
+    assert row_errors(whole, want).max() < lim
+    assert row_errors(feed(dec, toks, list(range(T + 1))), want).max() < lim                  # the recorded step
+    assert row_errors(feed(dec, toks, list(range(21)), batched=True), want[:20]).max() < lim  # single tokens on the batch kernels
+    for sizes in ([2], [3, 2, 64, 1, 31], [100, 1, 1], [33]):
+        assert row_errors(feed(dec, toks, cuts_of(T, sizes)), want).max() < lim, sizes
+    # only some places wanted, none wanted, and the first token alone
+    s = dec.open()
+    assert dec.forward(s, toks[:1], []) is None
+    some = dec.forward(s, toks[1:200], [0, 5, 198]).cpu().numpy()
+    assert row_errors(some, want[[1, 6, 199]]).max() < lim
+    assert dec.forward(s, toks[200:210], []) is None and dec.forward(s, toks[210:211], []) is None
+    assert row_errors(dec.forward(s, toks[211:213], [1]).cpu().numpy(), want[[212]]).max() < lim
+    dec.close(s)
+    dec.check_status()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_long_portions_are_cut(dtype):
+    toks, want, _, dec = model("mixed", dtype, max_portion=48)
+    assert row_errors(feed(dec, toks, [0, len(toks)]), want).max() < LIMIT[dtype]
+    s = dec.open()
+    sparse = dec.forward(s, toks, [3, 47, 48, 229]).cpu().numpy()
+    assert row_errors(sparse, want[[3, 47, 48, 229]]).max() < LIMIT[dtype]
+    dec.close(s)
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_places_are_reused_and_sequences_do_not_mix(dtype):
+    toks, want, _, dec = model("mixed", dtype, slots=2)
+    cfg, w = reference("mixed")[:2]
+    lim = LIMIT[dtype]
+    ref = R.LatentReference(cfg, w)
+    other = safe_tokens(ref, 120, 8)
+    other_want = ref.run(other)
+    a, b = dec.open(), dec.open()
+    ga, gb = [], []
+    for i in range(0, 120, 10):  # alternate: portions of one, tokens of the other
+        ga.append(dec.forward(a, toks[i:i + 10], list(range(10))).cpu().numpy())
+        gb += [dec.forward(b, other[j:j + 1], [0]).cpu().numpy() for j in range(i, i + 10)]
+    assert row_errors(np.concatenate(ga), want[:120]).max() < lim and row_errors(np.concatenate(gb), other_want).max() < lim
+    dec.close(a)
+    c = dec.open()  # the place of `a`, with its old rows underneath
+    assert c is a
+    assert row_errors(feed(dec, other, [0, 1, 3, 60, 120], seq=c), other_want).max() < lim
+    dec.check_status()
+
+
+def test_same_tokens_give_the_same_bits_whatever_ran_before():
+    toks, _, _, dec = model("mixed", "bfloat16")
+    first = feed(dec, toks, [0, 100, 101, 102, 230])
+    feed(dec, toks[::-1], [0, 7, 90])
+    assert np.array_equal(first, feed(dec, toks, [0, 100, 101, 102, 230]))
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_a_far_token_shows_in_the_logits(dtype):
+    """Two sequences that differ in one early token only, whose latent every query looks for: the device follows the oracle at
+    every position, whether the token was read in a prompt, in an early portion or decoded."""
+    cfg = config(64, 50, [layer(2, 16, 8, 32, 32, 32, 4, 4, 24, scale=1.0), layer(2, 16, 8, 32, 32, 32, kv_from=0, scale=1.0)])  # (all experts: no close calls)
+    w = random_weights(cfg, 4)
+    rng = np.random.default_rng(4)
+    direction = rng.standard_normal(32) * 6
+    w["l0.mix.dkv"][:] = 0.2 * w["l0.mix.dkv"]
+    w["l0.mix.dkv"][:32, 0] = bf16(direction)  # feature 0 of a token drives its latent
+    for t in range(50):
+        w["embed"][t, 0] = 0.0
+    w["embed"][0, 0], w["embed"][1, 0] = 12.0, -12.0
+    ref = R.LatentReference(cfg, {k: bf16(v) for k, v in w.items()})
+    tail = rng.integers(4, 50, 200)
+    seqs, wants = [np.concatenate([[5, 9, t], tail]) for t in (0, 1)], []
+    for s in seqs:
+        ref.reset()
+        wants.append(ref.run(s))
+    assert np.median(row_errors(wants[0][100:], wants[1][100:])) > 3 * LIMIT["bfloat16"]
+    dec = build_decoder(cfg, {k: bf16(v) for k, v in w.items()}, dtype, max_seq=256)
+    for s, want in zip(seqs, wants):
+        for cuts in ([0, 203], [0, 2, 4, 100, 203], list(range(204))):
+            assert row_errors(feed(dec, s, cuts), want).max() < LIMIT[dtype], len(cuts)
+
+
+def test_refusals():
+    toks, _, _, dec = model("odd", "float32", max_seq=20)
+    s = dec.open()
+    for bad in ([], [99], [-1], list(range(21))):
+        with pytest.raises(ValueError):
+            dec.forward(s, bad, [])
+    dec.forward(s, [1, 2, 3], [2])
+    with pytest.raises(ValueError, match="further tokens fit"):
+        dec.decode_greedy(s, 30)
+    assert len(dec.decode_greedy(s, 18)) == 18 and s.pos == 20
+    dec.close(s)
+    assert dec.cache_bytes() > 0 and dec.weight_bytes_per_token() > 0 and dec.launches > 0
+
+
+# ---- generation ----------------------------------------------------------------------------------------------------------------
+def oracle_greedy(cfg, w, prompt, n):
+    """The oracle's continuation and the smallest margin between its first and second choice."""
+    ref, out, margin = R.LatentReference(cfg, w), [], np.inf
+    logits = ref.run(prompt)[-1]
+    for _ in range(n):
+        top = np.sort(logits)[-2:]
+        margin = min(margin, (top[1] - top[0]) / logits.std(), ref.margin.min())
+        out.append(int(np.argmax(logits)))
+        logits = ref.run([out[-1]])[-1]
+    return out, margin
+
+
+def test_greedy_generation_through_the_queue():
+    cfg = CONFIGS["mixed"]
+    w = random_weights(cfg, 77)
+    dec = build_decoder(cfg, w, "float32", max_seq=300)
+    rng = np.random.default_rng(2)
+    prompts = [rng.integers(0, cfg["vocab"], n).tolist() for n in (1, 2, 40, 90)]
+    compared = 0
+    for portion in (None, 7, 1):
+        q = RequestQueue(dec, portion)
+        reqs = [q.submit(p, 200 if len(p) == 40 else 30) for p in prompts]
+        q.run()
+        for r in reqs:
+            want, margin = oracle_greedy(cfg, w, r.prompt, r.n_new)
+            if margin > 1e-4:  # (a margin the 32-bit mode resolves)
+                assert r.tokens == want
+                compared += 1
+    assert compared >= 6
+    bf = build_decoder(cfg, w, "bfloat16", max_seq=300)
+    q = RequestQueue(bf, 16)
+    reqs = [q.submit(p, 20) for p in prompts]
+    q.run()
+    for r in reqs:  # every pick is the arg-max, to bf16 accuracy, of the oracle's logits after the same tokens
+        logits = R.LatentReference(cfg, w).run(r.prompt + r.tokens[:-1])[len(r.prompt) - 1:]
+        picked = logits[np.arange(20), r.tokens]
+        assert np.quantile(logits.max(axis=1) - picked, 0.9) < 0.15 * logits.std()
+
+
+def test_trace_replay_generate_and_runner_from_a_model_folder(tmp_path):
+    cfg, w, toks, want, _ = reference("wide")
+    folder = save_model(tmp_path / "model", cfg, w)
+    toks = [int(t) for t in toks[:60]]
+    steps = [{"step": 0, "entries": [{"id": "x", "tokens": toks[:50], "want": [49, 3]}], "end": []},
+             {"step": 1, "entries": [{"id": "x", "tokens": toks[50:52], "want": []}], "end": []}]
+    steps += [{"step": i - 50, "entries": [{"id": "x", "tokens": [toks[i]], "want": [0]}], "end": ["x"] if i == 59 else []} for i in range(52, 60)]
+    steps.append({"step": 10, "entries": [{"id": "y", "tokens": toks[:1], "want": [0]}], "end": ["y"]})
+    out = tmp_path / "out"
+    out.mkdir()
+    for dtype in ("float32", "bfloat16"):
+        lines = [json.dumps(s) for s in steps]
+        if dtype == "float32":
+            r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", folder, "--dtype", dtype, "--out", str(out), "--max-tokens", "64"],
+                               input="\n".join(lines), capture_output=True, text=True, timeout=600)
+            assert r.returncode == 0, r.stderr[-2000:]
+            said = r.stdout.splitlines()
+        else:
+            said = []
+            replay(load_model(folder, dtype, max_seq=64), lines, str(out), said.append)
+        assert [x for x in said if x.startswith("done")] == [f"done {i}" for i in range(11)]
+        got = np.concatenate([np.fromfile(out / f"{i}.f32", "<f4").reshape(-1, cfg["vocab"]) for i in [0, *range(2, 11)]])
+        assert row_errors(got, want[[49, 3, *range(52, 60), 0]]).max() < LIMIT[dtype] and not (out / "1.f32").exists()
+    r = subprocess.run([sys.executable, "-m", "cut_b200.generate", "--model", folder, "--tokens", "5,6,7;9", "--n", "6", "--dtype", "float32",
+                        "--portion", "2"], capture_output=True, text=True, timeout=600, cwd=ROOT)
+    assert r.returncode == 0, r.stderr[-2000:]
+    for line in (json.loads(x) for x in r.stdout.splitlines()):
+        picks, margin = oracle_greedy(cfg, w, line["prompt"], 6)
+        assert margin < 1e-4 or line["tokens"] == picks
+
+
+def test_short_and_long_portions_take_both_forms():
+    """The same prompt with every portion in latent space, and with every portion expanded."""
+    toks, want, _, dec = model("mixed", "bfloat16")
+    old = layer_list.EXPAND_TOKENS
+    try:
+        for least in (2, 10 ** 9):
+            layer_list.EXPAND_TOKENS = least
+            for sizes in ([230], [2], [65, 64, 2]):
+                assert row_errors(feed(dec, toks, cuts_of(230, sizes)), want).max() < LIMIT["bfloat16"]
+    finally:
+        layer_list.EXPAND_TOKENS = old
