@@ -1250,8 +1250,10 @@ def main() -> None:
     ap.add_argument("--exchange", choices=["fused", "nccl"], default="fused",
                     help="N > 1: slices meet through the mat-vec's own peer-store epilogue, or through an NCCL all-gather")
     ap.add_argument("--layer-list", action="store_true",
-                    help="measure the layer-list models (kernels against their rooflines and the llama path's like kernels, prefill "
-                         "and decode throughput at equal size) on one GPU and print that (not the contract line)")
+                    help="measure the layer-list models (kernels against their rooflines and the like kernels of another model path, "
+                         "prefill and decode throughput at equal size) on one GPU and print that (not the contract line)")
+    ap.add_argument("--layer-list-model", choices=["bigerax", "lenesun"], default="bigerax",
+                    help="with --layer-list: bigerax beside the llama path, or lenesun beside bigerax")
     ap.add_argument("--layer-list-sizes", default="2048,4096", help="with --layer-list: widths of the whole-model measurement")
     args = ap.parse_args()
     if args.layer_list:
@@ -1270,7 +1272,8 @@ def main() -> None:
                 tflops = float(json.load(f).get("bf16_tflops", tflops))
         clocks = ClockSampler(0)
         clocks.start()
-        res = layer_bench.measure(hbm, tflops, source, models=[x for x in args.layer_list_sizes.split(",") if x])
+        res = layer_bench.measure(hbm, tflops, source, models=[x for x in args.layer_list_sizes.split(",") if x],
+                                  design=args.layer_list_model)
         res["clocks"] = clocks.stop()
         print(json.dumps({"layer_list": res}), flush=True)
         return

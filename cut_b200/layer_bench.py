@@ -1,5 +1,6 @@
 """Measurements of the layer-list models (bench.py --layer-list): every kernel alone against its roofline, beside the like
-kernel of the llama path at equal shape, and prefill / decode throughput of whole models of equal size.
+kernel of another model path at equal shape, and prefill / decode throughput of whole models of equal size: Bigerax beside the
+llama path, Lenesun (--layer-list-model lenesun) beside Bigerax.
 
 Device time from CUDA events around replays of a graph of launches that walk through enough distinct operands (>= 400 MB)
 that L2 does not serve them.  Roofline time = max(bytes / copy bandwidth, FLOPs / bf16 GEMM rate); bytes count every operand
@@ -14,8 +15,8 @@ import torch
 
 from . import _lib as L
 from . import ops
-from .layer_list import (Bigram, FeedForward, GatedRecurrence, Layer, LayerListConfig, LayerListDecoder, Rotation, WindowAttention, pad,
-                         rotation_tables)
+from .layer_list import (Bigram, FeedForward, GatedRecurrence, LatentAttention, Layer, LayerListConfig, LayerListDecoder, MixtureOfExperts, Rotation,
+                         WindowAttention, pad, rotation_tables)
 
 
 def time_us(launches, reps: int = 5, warm: int = 3) -> float:
@@ -253,6 +254,233 @@ def model_config(hidden: int, ff: int, H: int, G: int, dim: int, window: int, n_
     return LayerListConfig(hidden, vocab, tuple(layers), 2, 1e-6, Bigram(65521, 36313, 27191))
 
 
+# ---- latent attention and mixtures of experts -----------------------------------------------------------------------------------
+def _graph_calls(name: str, ds, min_calls: int = 32):
+    return [lambda d=d: L.check(getattr(L.lib(), name)(C.byref(d), ops._stream_ptr())) for d in ds * max(1, min_calls // len(ds))]
+
+
+def head_matvec_us(H: int, N: int, K: int) -> float:
+    Ws, x, out = [_bf16(H * N, K) for _ in range(_copies(H * N * K * 2))], torch.randn((1, H * K), device="cuda"), torch.zeros((1, H * N), device="cuda")
+    return time_us(_graph_calls("cutb_dense_matmul", [ops.batch_desc(x, W, K, out, H, K, N) for W in Ws]))
+
+
+class _LatentShapes:
+    """Tensors of one latent-attention layer whose context is `ctx` tokens, the last T of them new."""
+
+    def __init__(self, H, dim, rot, vdim, rank, q_rank, T, ctx):
+        self.p, self.T, self.ctx = (H, dim, rot, vdim, rank), T, ctx
+        self.tables = tuple(torch.from_numpy(t).cuda() for t in rotation_tables(Rotation(10000.0, rot), ctx))
+        f = lambda *s: torch.randn(s, device="cuda")
+        self.cache = f(ctx, pad(rank, 8) + pad(rot, 8)).to(torch.bfloat16)
+        self.q, self.qa, self.lat, self.cq = f(T, H * (dim + rot)), f(1, H * rank), f(T, rank + rot), f(T, q_rank)
+        self.one, self.sink = torch.ones(max(rank, q_rank), device="cuda"), torch.zeros(H, device="cuda")
+        self.cq_out = torch.zeros((T, q_rank), device="cuda", dtype=torch.bfloat16)
+        self.out = torch.zeros((T, H * vdim), device="cuda", dtype=torch.bfloat16)
+
+    def desc(self, T=None, pos=None, **more):
+        H, dim, rot, vdim, rank = self.p
+        T = self.T if T is None else T
+        return ops.latent_desc(self.cache, H, dim, rot, vdim, rank, scale=(dim + rot) ** -0.5, eps=1e-6, max_pos=self.ctx, n_tokens=T, cos_t=self.tables[0],
+                               sin_t=self.tables[1], sink=self.sink, pos=self.ctx - T if pos is None else pos, **more)
+
+
+def latent_decode_us(H, dim, rot, vdim, rank, ctx):
+    """(attention over the cached latents, the values' mat-vec behind it) of one token, each launch timed alone."""
+    n = _copies(ctx * (rank + rot) * 2)
+    sets = [_LatentShapes(H, dim, rot, vdim, rank, 64, 1, ctx) for _ in range(n)]
+    ws = torch.zeros(ops.latent_workspace_bytes(sets[0].desc()) // 4, device="cuda")
+    att = [s.desc(q=s.q, qa=s.qa, workspace=ws, lat=s.lat, lat_norm_w=s.one) for s in sets]
+    a = time_us(_graph_calls("cutb_latent_attention", att))
+    Ws, out = [_bf16(H * vdim, rank) for _ in range(_copies(H * vdim * rank * 2))], torch.zeros((1, H * vdim), device="cuda")
+    v = time_us(_graph_calls("cutb_latent_values", [sets[0].desc(out=out, workspace=ws, w_uv=W) for W in Ws]))
+    return a, v
+
+
+def latent_prefill_us(H, dim, rot, vdim, rank, T) -> float:
+    n, keep, ds = _copies(T * H * (dim + vdim) * 2 + T * H * (dim + rot) * 4, hi=16), [], []
+    for _ in range(n):
+        s, exp = _LatentShapes(H, dim, rot, vdim, rank, 64, T, T), _bf16(T, H * (dim + vdim))
+        keep.append((s, exp))
+        ds.append(s.desc(q=s.q, k_exp=exp, v_exp=exp[:, H * dim:], out=s.out))
+    return time_us(_graph_calls("cutb_latent_prefill", ds, 1))
+
+
+def latent_write_us(H, dim, rot, vdim, rank, q_rank, T) -> float:
+    keep = [_LatentShapes(H, dim, rot, vdim, rank, q_rank, T, T) for _ in range(_copies(T * (rank + rot + q_rank) * 6, hi=32))]
+    return time_us(_graph_calls("cutb_latent_kv_write", [s.desc(lat=s.lat, lat_norm_w=s.one, cq=s.cq, cq_norm_w=s.one[:q_rank], cq_out=s.cq_out) for s in keep], 1))
+
+
+class _Experts:
+    def __init__(self, width, ff, E, top, T, sets):
+        self.p = (width, ff, E, top)
+        self.gu, self.dn = [_bf16(E * 2 * ff, width) for _ in range(sets)], [_bf16(E * width, ff) for _ in range(sets)]
+        z = torch.randn((T, E), device="cuda")
+        i32 = lambda *s: torch.zeros(s, dtype=torch.int32, device="cuda")
+        self.z, self.weights, self.ids, self.slots, self.offsets = z, torch.zeros((T, top), device="cuda"), i32(T, top), i32(T, top), i32(E + 1)
+        self.route = ops.moe_route_desc(z, E, top, self.weights, self.ids, self.slots, self.offsets)
+        ops.launch_layer_op("cutb_moe_route", self.route)
+        torch.cuda.synchronize()
+
+
+def expert_prefill_us(width, ff, E, top, T) -> dict:
+    n = _copies(E * 3 * ff * width * 2 + T * top * (width + ff) * 4, hi=8)
+    e, rows = _Experts(width, ff, E, top, T, n), T * top
+    bf = lambda r, c: torch.zeros((r, c), device="cuda", dtype=torch.bfloat16)
+    x, srt, act, out = [_bf16(T, width) for _ in range(4)], [_bf16(rows, width) for _ in range(n)], [_bf16(rows, ff) for _ in range(n)], bf(rows, width)
+    group = dict(offsets=e.offsets, experts=E, tokens=T, top=top, variant=L.DENSE_TC)
+    aout = bf(rows, ff)
+    up = [ops.moe_matmul_desc(a, W, width, out=aout, glu=L.GLU_CLAMPED, alpha=1.702, beta=1.0, limit=7.0, **group) for a, W in zip(srt, e.gu)]
+    down = [ops.moe_matmul_desc(a, W, ff, out=out, **group) for a, W in zip(act, e.dn)]
+    scatter = [ops.moe_scatter_desc(a, width, e.slots, E, b) for a, b in zip(x, srt)]
+    return {"route": time_us(_graph_calls("cutb_moe_route", [e.route], 16)), "scatter": time_us(_graph_calls("cutb_moe_scatter", scatter, 8)),
+            "up": time_us(_graph_calls("cutb_moe_matmul", up, 1)), "down": time_us(_graph_calls("cutb_moe_matmul", down, 1))}
+
+
+def expert_decode_us(width, ff, E, top, Nd, Kd, Ko):
+    """(up with the query projection beside it, down with the output projection beside it) of one token."""
+    active = top * 3 * ff * width * 2
+    n = _copies(active // 2, hi=16)
+    e = _Experts(width, ff, E, top, 1, n)
+    wd, wo = [_bf16(Nd, Kd) for _ in range(n)], [_bf16(width, Ko) for _ in range(n)]
+    f = lambda c: torch.randn(c, device="cuda")
+    x, xd, one, xo, act, q, y = f(width), f(Kd), torch.ones(Kd, device="cuda"), f(Ko), f(top * ff), f(Nd), f(width)
+    ids = torch.zeros(top, dtype=torch.int32, device="cuda")
+    up = [ops.expert_desc(E, top, width, ff, W, ids, act, logits=e.z, x=x, alpha=1.702, beta=1.0, limit=7.0, dense=D, dense_K=Kd, xd=xd, xd_norm_w=one,
+                          eps=1e-6, out=q) for W, D in zip(e.gu, wd)]
+    down = [ops.expert_desc(E, top, width, ff, W, ids, act, dense=D, dense_K=Ko, xd=xo, out=y) for W, D in zip(e.dn, wo)]
+    return time_us(_graph_calls("cutb_expert_up", up)), time_us(_graph_calls("cutb_expert_down", down))
+
+
+def parallel_norm_us(T: int, dim: int, top: int) -> float:
+    keep, launches, w = [], [], torch.ones(dim, device="cuda")
+    for _ in range(_copies(T * dim * (14 + 2 * top), hi=32)):
+        x, y, m = torch.randn((T, dim), device="cuda"), torch.randn((T, dim), device="cuda"), _bf16(T * top, dim)
+        h, rows = torch.zeros((T, dim), device="cuda", dtype=torch.bfloat16), torch.randperm(T * top, device="cuda").to(torch.int32).view(T, top)
+        pw = torch.rand((T, top), device="cuda")
+        keep.append((x, y, m, h, rows, pw))
+        launches.append(lambda a=keep[-1]: ops.residual_norm(a[0], w, 1, 1e-6, y=a[1], x_out=a[0], out=a[3], center=True, y_scale=0.3, parts=(a[2], a[4], a[5])))
+    return time_us(launches)
+
+
+def latent_table(roof: Roofline, hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, context, T, vocab, kv_heads) -> dict:
+    """Every kernel of a Lenesun decode step and of a T-token prefill at one layer size, with Bigerax's like kernel."""
+    out, mv_bytes = {}, lambda N, K: N * K * 2 + 4 * (N + K)
+    n_in, n_uq, wide = q_rank + rank + rot + E, H * (dim + rot), dim + rot
+
+    def put(name, us, nbytes, flops=0.0, like=None):
+        out[name] = {"ours": roof.entry(us, nbytes, flops), **({"bigerax": roof.entry(*like)} if like else {})}
+
+    dense_like = lambda N, K, **kw: (matvec_us(N, K, **kw), mv_bytes(N, K))
+    put(f"decode input mat-vec (layer norm fused) {n_in}x{hidden}", matvec_us(n_in, hidden, norm=True), mv_bytes(n_in, hidden), like=dense_like(n_in, hidden, norm=True))
+    up, down = expert_decode_us(hidden, ff, E, top, n_uq, q_rank, H * vdim)
+    ub = mv_bytes(n_uq, q_rank) + mv_bytes(top * 2 * ff, hidden)
+    db = mv_bytes(hidden, H * vdim + top * ff)
+    put(f"decode experts up {top}x{2 * ff}x{hidden} + queries {n_uq}x{q_rank}", up, ub, like=dense_like(ub // (2 * hidden), hidden, norm=True))
+    put(f"decode experts down {hidden}x{top}x{ff} + output {hidden}x{H * vdim}", down, db, like=dense_like(hidden, H * vdim + top * ff))
+    put(f"decode queries into latent space {H}x{rank}x{dim}", head_matvec_us(H, rank, dim), mv_bytes(H * rank, dim), like=dense_like(H * dim, rank))
+    att, val = latent_decode_us(H, dim, rot, vdim, rank, context)
+    put(f"decode latent attention, context {context}", att, context * (rank + rot) * 2 + 4 * H * (rank + wide),
+        4.0 * H * context * (2 * rank + rot) / 2, like=(window_us(1, H, kv_heads, dim, context, True, context), context * kv_heads * dim * 4 + 8 * H * dim))
+    put(f"decode values out of latent space {H}x{vdim}x{rank}", val, mv_bytes(H * vdim, rank), like=dense_like(H * vdim, rank))
+    put(f"decode head mat-vec (layer norm fused) {vocab}x{hidden}", matvec_us(vocab, hidden, norm=True), mv_bytes(vocab, hidden), like=dense_like(vocab, hidden, norm=True))
+
+    gemm_bytes = lambda M, N, K, o: N * K * 2 + M * K * 2 + M * N * o
+    for M in sorted({128, 512, T}):
+        rows = M * top
+        e = expert_prefill_us(hidden, ff, E, top, M)
+        used = min(E, rows)
+        for k, N, K, o in (("up", 2 * ff, hidden, 1), ("down", hidden, ff, 2)):
+            like = (gemm_us(rows, N, K, out_t=torch.bfloat16), gemm_bytes(rows, N, K, 2), 2.0 * rows * N * K)
+            put(f"prefill experts {k}, {M} tokens, {E} x {N}x{K}", e[k], used * N * K * 2 + rows * K * 2 + rows * N * o, 2.0 * rows * N * K, like=like)
+    e = expert_prefill_us(hidden, ff, E, top, T)
+    put(f"prefill routing (choice, sort), {T} tokens", e["route"], T * E * 4 + T * top * 16)
+    put(f"prefill expert order (row copies), {T} x {top} x {hidden}", e["scatter"], T * hidden * 2 + T * top * hidden * 2)
+    for name, N, K in (("input", n_in, hidden), ("queries", n_uq, q_rank), ("expansion", H * (dim + vdim), rank), ("output", hidden, H * vdim)):
+        us = gemm_us(T, N, K)
+        put(f"prefill {name} GEMM {T}x{N}x{K}", us, gemm_bytes(T, N, K, 4), 2.0 * T * N * K)
+    pairs = T * (T + 1) / 2
+    put(f"prefill latent attention (expanded), {T} tokens", latent_prefill_us(H, dim, rot, vdim, rank, T), T * H * (wide * 4 + (dim + vdim) * 2 + vdim * 2) + T * rot * 2,
+        2.0 * pairs * H * (wide + vdim), like=(window_us(T, H, kv_heads, dim, T, False, 0), T * (H * dim * 6 + 2 * kv_heads * dim * 2), 4.0 * pairs * H * dim))
+    put(f"prefill cache write and query norm, {T} tokens", latent_write_us(H, dim, rot, vdim, rank, q_rank, T), T * (rank + rot + q_rank) * 6,
+        like=(kv_write_us(T, H, kv_heads, dim), T * 2 * kv_heads * dim * 6))
+    put(f"prefill residual + gathered experts + layer norm, {T} x {hidden}", parallel_norm_us(T, hidden, top), T * hidden * (14.0 + 2 * top),
+        like=(norm_us(T, hidden), T * hidden * 14.0))
+    put(f"prefill embedding, {T} x {hidden}", embed_us(T, hidden, vocab), T * hidden * 8.0)
+    return out
+
+
+def latent_model_config(hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, n_layers, vocab) -> LayerListConfig:
+    """Every other layer reads the latents of the one before it."""
+    att = lambda j: LatentAttention(H, dim, vdim, q_rank, rank, (dim + rot) ** -0.5, Rotation(10000.0, rot), True, j)
+    layers = tuple(Layer(att(None if i % 2 == 0 else i - 1), MixtureOfExperts(E, top, ff, 7.0, 1.702, 1.0)) for i in range(n_layers))
+    return LayerListConfig(hidden, vocab, layers, 1, 1e-6, norm_center=True, parallel=True, residual_mult=0.3, embed_scale=2.0, tied_head=True)
+
+
+def latent_random_weights(cfg: LayerListConfig) -> dict:
+    layers = []
+    for l in cfg.layers:
+        m, f, one = l.mixer, l.mlp, lambda n: torch.ones(n, device="cuda")
+        mix = {"dq": _bf16(m.q_rank, cfg.width), "dq.norm": one(m.q_rank), "uq": _bf16(m.q_rows, m.q_rank), "uk": _bf16(m.heads * m.dim, m.kv_rank),
+               "uv": _bf16(m.heads * m.vdim, m.kv_rank), "o": _bf16(cfg.width, m.heads * m.vdim), "sink": torch.zeros(m.heads, device="cuda")}
+        if m.kv_from is None:
+            mix.update({"dkv": _bf16(m.kv_rows, cfg.width), "dkv.norm": one(m.kv_rank)})
+        layers.append({"norm1": one(cfg.width), "mix": mix, "mlp": {
+            "gate": _bf16(f.experts, f.ff, cfg.width), "up": _bf16(f.experts, f.ff, cfg.width), "down": _bf16(f.experts, cfg.width, f.ff),
+            "router": _bf16(f.experts, cfg.width), "router.b": torch.zeros(f.experts, device="cuda")}})
+    return {"embed": _bf16(cfg.vocab, cfg.width), "final_norm": torch.ones(cfg.width, device="cuda"), "layers": layers}
+
+
+def decoder_throughput(roof: Roofline, dec: LayerListDecoder, vocab: int, T: int, steps: int, matmul_flops: float) -> dict:
+    """Prefill of T tokens (best of 4) and the following `steps` tokens."""
+    prompt = np.random.default_rng(1).integers(0, vocab, T)
+    ev = lambda: torch.cuda.Event(enable_timing=True)
+    best = float("inf")
+    for turn in range(4):
+        s = dec.open()
+        torch.cuda.synchronize()
+        a, b = ev(), ev()
+        a.record()
+        dec.forward(s, prompt, [T - 1])
+        b.record()
+        torch.cuda.synchronize()
+        best = min(best, a.elapsed_time(b))
+        if turn < 3:
+            dec.close(s)
+    dec.decode_greedy(s, 4)
+    torch.cuda.synchronize()
+    a, b = ev(), ev()
+    a.record()
+    for _ in range(steps):
+        dec._one_token(s)
+    b.record()
+    torch.cuda.synchronize()
+    dec.check_status()
+    ms = a.elapsed_time(b) / steps
+    return {"prefill_tokens": T, "prefill_ms": round(best, 3), "prefill_tok/s": round(T / best * 1e3),
+            "prefill_GEMM_roofline_fraction": round(matmul_flops / roof.tf / 1e9 / best, 3), "decode_ms": round(ms, 4), "decode_tok/s": round(1e3 / ms, 1),
+            "weight_GB_per_token": round(dec.weight_bytes_per_token() / 1e9, 3),
+            "decode_roofline_fraction": round(dec.weight_bytes_per_token() / roof.hbm / 1e6 / ms, 3), "launches_per_token": s.step.launches}
+
+
+def latent_throughput(roof: Roofline, hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, n_layers, vocab, T, kv_heads, steps: int = 128) -> dict:
+    cfg = latent_model_config(hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, n_layers, vocab)
+    dec = LayerListDecoder(cfg, latent_random_weights(cfg), max_seq=T + steps + 16)
+    per_token = sum(d["in"].K * d["in"].N + d["uq"].K * d["uq"].N + d["expand"].K * d["expand"].N + d["out"].K * d["out"].N + top * 3 * ff * hidden for d in dec.layers)
+    res = {"lenesun": decoder_throughput(roof, dec, vocab, T, steps, 2.0 * T * per_token)}
+    del dec
+    torch.cuda.empty_cache()
+    # Bigerax with as many layers, all of them attention with a window over the whole context, and as much feed-forward per token
+    ff_like = top * ff * 3 // 2
+    att = WindowAttention(H, kv_heads, dim, dim, T + steps + 16, dim ** -0.5, Rotation(10000.0, dim), True, True)
+    like = LayerListConfig(hidden, vocab, tuple(Layer(att, FeedForward(ff_like)) for _ in range(n_layers)), 2, 1e-6, Bigram(65521, 36313, 27191))
+    dec = LayerListDecoder(like, random_weights(like), max_seq=T + steps + 16)
+    per_token = (dec.weight_bytes_per_token() - dec.head.nbytes) / 2
+    res["bigerax"] = decoder_throughput(roof, dec, vocab, T, steps, 2.0 * T * per_token)
+    del dec
+    torch.cuda.empty_cache()
+    return res
+
+
 def random_weights(cfg: LayerListConfig) -> dict:
     lin = lambda d, names, rows, cols, bias: {**{n: _bf16(r, cols) for n, r in zip(names, rows)},
                                               **({n + ".b": torch.zeros(r, device="cuda") for n, r in zip(names, rows)} if bias else {})}
@@ -278,41 +506,15 @@ def model_throughput(roof: Roofline, hidden: int, ff: int, H: int, G: int, dim: 
     cfg = model_config(hidden, ff, H, G, dim, window, n_layers, vocab)
     dec = LayerListDecoder(cfg, random_weights(cfg), max_seq=T + steps + 16)
     prompt = np.random.default_rng(1).integers(0, vocab, T)
-    ev = lambda: torch.cuda.Event(enable_timing=True)
-    best = float("inf")
-    for _ in range(4):
-        s = dec.open()
-        torch.cuda.synchronize()
-        a, b = ev(), ev()
-        a.record()
-        dec.forward(s, prompt, [T - 1])
-        b.record()
-        torch.cuda.synchronize()
-        best = min(best, a.elapsed_time(b))
-        if _ < 3:
-            dec.close(s)
-    dec.decode_greedy(s, 4)
-    torch.cuda.synchronize()
-    a, b = ev(), ev()
-    a.record()
-    for _ in range(steps):
-        dec._one_token(s)
-    b.record()
-    torch.cuda.synchronize()
-    dec.check_status()
-    ms = a.elapsed_time(b) / steps
-    n_lin = (dec.weight_bytes_per_token() - dec.head.nbytes) / 2
-    pre_roof = 2.0 * T * n_lin / roof.tf / 1e9
-    ours = {"prefill_tokens": T, "prefill_ms": round(best, 3), "prefill_tok/s": round(T / best * 1e3), "prefill_GEMM_roofline_fraction": round(pre_roof / best, 3),
-            "decode_ms": round(ms, 4), "decode_tok/s": round(1e3 / ms, 1), "weight_GB_per_token": round(dec.weight_bytes_per_token() / 1e9, 3),
-            "decode_roofline_fraction": round(dec.weight_bytes_per_token() / roof.hbm / 1e6 / ms, 3), "launches_per_token": s.step.launches}
-    del dec, s
+    ours = decoder_throughput(roof, dec, vocab, T, steps, 2.0 * T * (dec.weight_bytes_per_token() - dec.head.nbytes) / 2)
+    del dec
     torch.cuda.empty_cache()
 
     from .llama_decode import LlamaConfig, LlamaDecoder, synthetic_weights
 
     lc = LlamaConfig(n_layers=n_layers, hidden=hidden, n_heads=H, n_kv_heads=G, head_dim=dim, ffn=ff, vocab=vocab, max_seq=T + steps + 16)
     ll = LlamaDecoder(lc, synthetic_weights(lc, seed=41, distinct_layers=False, scale_shift=7))
+    ev = lambda: torch.cuda.Event(enable_timing=True)
     best = float("inf")
     for _ in range(4):
         torch.cuda.synchronize()
@@ -348,15 +550,26 @@ SIZES = {  # hidden, ff, query heads, KV heads, head, window, layers, vocabulary
 }
 
 
-def measure(hbm_gbs: float, tflops: float, source: str, tables=("4096",), models=("2048", "4096"), T: int = 2048) -> dict:
+LATENT_SIZES = {  # hidden, heads, unrotated, rotated and value parts, query and latent ranks, experts, top, ff, layers, vocabulary, KV heads beside it
+    "2048": (2048, 16, 128, 64, 128, 768, 512, 32, 4, 1024, 16, 32000, 4),
+    "4096": (4096, 32, 128, 64, 128, 1536, 512, 16, 4, 2048, 8, 32000, 8),
+}
+
+
+def measure(hbm_gbs: float, tflops: float, source: str, tables=("4096",), models=("2048", "4096"), T: int = 2048, design: str = "bigerax") -> dict:
     roof = Roofline(hbm_gbs, tflops)
     res = {"roofline": {"hbm_GB/s": hbm_gbs, "bf16_TFLOP/s": tflops, "source": source},
            "timing": "CUDA-graph chains over >= 400 MB of distinct operands, best of 5", "kernels": {}, "models": {}}
     for s in tables:
-        hidden, ff, H, G, dim, window, _, vocab = SIZES[s]
-        res["kernels"][s] = kernel_table(roof, hidden, ff, H, G, dim, window, 2048, T, vocab)
+        if design == "lenesun":
+            hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, _, vocab, kv = LATENT_SIZES[s]
+            res["kernels"][s] = latent_table(roof, hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, 2048, T, vocab, kv)
+        else:
+            hidden, ff, H, G, dim, window, _, vocab = SIZES[s]
+            res["kernels"][s] = kernel_table(roof, hidden, ff, H, G, dim, window, 2048, T, vocab)
         torch.cuda.empty_cache()
     for s in models:
-        res["models"][s] = model_throughput(roof, *SIZES[s], T=T)
+        res["models"][s] = (latent_throughput(roof, *LATENT_SIZES[s][:-1], T, LATENT_SIZES[s][-1]) if design == "lenesun"
+                            else model_throughput(roof, *SIZES[s], T=T))
         torch.cuda.empty_cache()
     return res
