@@ -205,6 +205,7 @@ constexpr int HV_THREADS = 256;
 
 template <int LPR> __global__ void __launch_bounds__(HV_THREADS) head_matvec_kernel(const HeadMvParams p, uint32_t rows_per_block) {
   extern __shared__ __align__(16) float hv_smem[];
+  __shared__ float share[64];
   constexpr uint32_t RPW = 32 / LPR, PASS = HV_THREADS / 32 * RPW;  // rows of a warp and of the block at a time
   constexpr int U = 4;
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, sub = lane % LPR;
@@ -227,18 +228,25 @@ template <int LPR> __global__ void __launch_bounds__(HV_THREADS) head_matvec_ker
     if (p.splits) {
       const float2 *ml = p.ml + (size_t)(h0 + h) * p.splits;
       const float *part = p.part + (size_t)(h0 + h) * p.splits * p.ld_part;
-      float m = -1e30f, l = 0.f;
-      for (uint32_t s = 0; s < p.splits; ++s) m = fmaxf(m, ml[s].x);
-      for (uint32_t s = 0; s < p.splits; ++s) l = fmaf(exp2f(ml[s].x - m), ml[s].y, l);
-      const float inv = 1.0f / l;
+      if (warp == 0) {  // a partial sum's share: exp2(its maximum - the largest) / the whole weight sum
+        const float2 a = lane < p.splits ? ml[lane] : make_float2(-1e30f, 0.f), b = lane + 32 < p.splits ? ml[lane + 32] : make_float2(-1e30f, 0.f);
+        float m = fmaxf(a.x, b.x);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        const float wa = exp2f(a.x - m), wb = exp2f(b.x - m);
+        const float inv = 1.0f / warp_sum(wa * a.y + wb * b.y);
+        share[lane] = wa * inv, share[lane + 32] = wb * inv;
+      }
+      __syncthreads();
       for (uint32_t k = tid; k < 8 * K8; k += HV_THREADS) {
         float v = 0.f;
         if (k < p.K) {
 #pragma unroll 8
-          for (uint32_t s = 0; s < p.splits; ++s) v = fmaf(exp2f(ml[s].x - m), part[(size_t)s * p.ld_part + k], v);
+          for (uint32_t s = 0; s < p.splits; ++s) v = fmaf(share[s], part[(size_t)s * p.ld_part + k], v);
         }
-        put(h, k, v * inv);
+        put(h, k, v);
       }
+      __syncthreads();
     } else {
       const float *x = p.x + (size_t)(h0 + h) * p.x_batch;
       for (uint32_t k = tid; k < 8 * K8; k += HV_THREADS) put(h, k, k < p.K ? x[k] : 0.f);

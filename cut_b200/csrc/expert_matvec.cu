@@ -8,7 +8,7 @@
 // DOWN  a tile is one output row: the dense matrix's row and the same row of every chosen expert, one running sum.
 //
 // A tile belongs to one warp, tiles are dealt over the SMs first; a lane takes every 32nd 16-byte piece, two steps of loads are
-// in flight.  The first dense rows start towards L2 before the wait for the previous kernel; the experts are not known then.
+// in flight.  The first steps of the dense rows are issued before the wait for the previous kernel.
 #include <cuda_bf16.h>
 
 #include "common.cuh"
@@ -47,9 +47,60 @@ template <bool UP> __global__ void __launch_bounds__(EX_MAX_THREADS, 1) expert_m
   const uint32_t tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5;
   const uint32_t tstep = gridDim.x * (nt >> 5), first = warp * gridDim.x + blockIdx.x;
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-  if (p.Kd8 && lane < R) {
-    const uint32_t row = first * R + lane;
-    if (row < p.Nd) asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(p.Wd + (size_t)row * p.ldwd8), "r"(p.Kd8 * 16u) : "memory");
+
+  // a tile is a sequence of segments (one in UP): consecutive pieces of R rows against a stretch of the staged input
+  struct Segment {
+    const uint4 *w;
+    uint32_t step, k8;  // distance of the rows (0: there is no second one), pieces
+  };
+  auto is_dense = [&](uint32_t tile, uint32_t s) { return UP ? tile < p.dense_tiles : p.Kd8 && s == 0; };
+  auto segment = [&](uint32_t tile, uint32_t s) {
+    Segment g;
+    if constexpr (UP) {
+      if (tile < p.dense_tiles) {
+        g.w = p.Wd + (size_t)tile * R * p.ldwd8, g.step = tile * R + 1 < p.Nd ? p.ldwd8 : 0, g.k8 = p.Kd8;
+      } else {
+        const uint32_t t = tile - p.dense_tiles, k = t / p.ff;
+        g.w = p.W + ((size_t)ids[k] * 2 * p.ff + 2 * (t - k * p.ff)) * p.ldw8, g.step = p.ldw8, g.k8 = p.K8;
+      }
+    } else {
+      const uint32_t k = s - (p.Kd8 ? 1 : 0);
+      if (p.Kd8 && s == 0) g.w = p.Wd + (size_t)tile * p.ldwd8, g.k8 = p.Kd8;
+      else g.w = p.W + ((size_t)ids[k] * p.width + tile) * p.ldw8, g.k8 = p.K8;
+      g.step = 0;
+    }
+    return g;
+  };
+  const uint32_t nseg = UP ? 1 : p.top + (p.Kd8 ? 1 : 0);
+  uint32_t l_tile = first, l_s = 0, l_k = lane;
+  bool l_new = true;  // the segment under the load cursor has not been looked up (that of an expert needs its number)
+  Segment lg{};
+  auto load = [&](uint4 (&w)[UNR][R]) {
+    if (l_tile >= p.ntiles) return;
+    if (l_new) lg = segment(l_tile, l_s), l_new = false;
+#pragma unroll
+    for (int u = 0; u < UNR; ++u)
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const uint32_t k = l_k + 32 * u;
+        w[u][r] = k < lg.k8 && (r == 0 || lg.step) ? ld_stream(lg.w + (size_t)r * lg.step + k) : make_uint4(0, 0, 0, 0);
+      }
+    l_k += 32 * UNR;
+    if (l_k >= lg.k8 + lane) {  // (the same step in every lane)
+      l_k = lane, l_new = true;
+      if (++l_s == nseg) l_s = 0, l_tile += tstep;
+    }
+  };
+  // loads of the dense matrix are on their way before the wait for the previous kernel; the experts are not known then
+  uint4 wa[UNR][R], wb[UNR][R];
+  uint32_t early = 0;
+  if (l_tile < p.ntiles && is_dense(l_tile, l_s)) {
+    load(wa);
+    early = 1;
+    if (l_tile < p.ntiles && is_dense(l_tile, l_s)) {
+      load(wb);
+      early = 2;
+    }
   }
   asm volatile("griddepcontrol.wait;" ::: "memory");
 
@@ -90,48 +141,6 @@ template <bool UP> __global__ void __launch_bounds__(EX_MAX_THREADS, 1) expert_m
   }
   __syncthreads();
 
-  // a tile is a sequence of segments (one in UP): consecutive pieces of R rows against a stretch of the staged input
-  struct Segment {
-    const uint4 *w;
-    uint32_t step, k8, x8;  // distance of the rows (0: there is no second one), pieces, first piece of the input
-  };
-  auto segment = [&](uint32_t tile, uint32_t s) {
-    Segment g;
-    if constexpr (UP) {
-      if (tile < p.dense_tiles) {
-        g.w = p.Wd + (size_t)tile * R * p.ldwd8, g.step = tile * R + 1 < p.Nd ? p.ldwd8 : 0, g.k8 = p.Kd8, g.x8 = 0;
-      } else {
-        const uint32_t t = tile - p.dense_tiles, k = t / p.ff;
-        g.w = p.W + ((size_t)ids[k] * 2 * p.ff + 2 * (t - k * p.ff)) * p.ldw8, g.step = p.ldw8, g.k8 = p.K8, g.x8 = p.Kd8;
-      }
-    } else {
-      const uint32_t k = s - (p.Kd8 ? 1 : 0);
-      if (p.Kd8 && s == 0) g.w = p.Wd + (size_t)tile * p.ldwd8, g.k8 = p.Kd8, g.x8 = 0;
-      else g.w = p.W + ((size_t)ids[k] * p.width + tile) * p.ldw8, g.k8 = p.K8, g.x8 = p.Kd8 + k * p.K8;
-      g.step = 0;
-    }
-    return g;
-  };
-  const uint32_t nseg = UP ? 1 : p.top + (p.Kd8 ? 1 : 0);
-  uint32_t l_tile = first, l_s = 0, l_k = lane;
-  Segment lg{};
-  if (l_tile < p.ntiles) lg = segment(l_tile, 0);
-  auto load = [&](uint4 (&w)[UNR][R]) {
-    if (l_tile >= p.ntiles) return;
-#pragma unroll
-    for (int u = 0; u < UNR; ++u)
-#pragma unroll
-      for (int r = 0; r < R; ++r) {
-        const uint32_t k = l_k + 32 * u;
-        w[u][r] = k < lg.k8 && (r == 0 || lg.step) ? ld_stream(lg.w + (size_t)r * lg.step + k) : make_uint4(0, 0, 0, 0);
-      }
-    l_k += 32 * UNR;
-    if (l_k >= lg.k8 + lane) {  // (the same step in every lane)
-      l_k = lane;
-      if (++l_s == nseg) l_s = 0, l_tile += tstep;
-      if (l_tile < p.ntiles) lg = segment(l_tile, l_s);
-    }
-  };
   uint32_t tile = first, seg = 0, k = lane, c_k8 = 0, c_x8 = 0;
   auto at = [&]() {
     if constexpr (UP) c_k8 = tile < p.dense_tiles ? p.Kd8 : p.K8, c_x8 = tile < p.dense_tiles ? 0 : p.Kd8;
@@ -176,9 +185,8 @@ template <bool UP> __global__ void __launch_bounds__(EX_MAX_THREADS, 1) expert_m
     tile += tstep;
     at();
   };
-  uint4 wa[UNR][R], wb[UNR][R];
-  load(wa);
-  load(wb);
+  if (early < 1) load(wa);
+  if (early < 2) load(wb);
   while (tile < p.ntiles) {
     use(wa);
     load(wa);

@@ -2,19 +2,26 @@
 // rotated key part that all heads share.  Beside window_attention.cu, whose caches hold keys and values per head.
 //
 //  * latent_kv_write_kernel: a batch of tokens into the cache, and the norm of the latent queries;
-//  * latent_attention_simt_kernel: the absorbed form (every head's query against the cache row itself) in fp32 arithmetic, for
-//    any size, either cache type, and any number of tokens.  For one token the keys are shared out over blocks, which leave
-//    partial sums; the values' mat-vec behind it merges them while it stages its input (head_matvec_kernel);
+//  * latent_decode_tc_kernel: the absorbed form (every head's query against the cache row itself) over a bf16 cache: one token
+//    or a few.  A block takes 16 heads of a token and a share of its keys; the eight blocks of a cluster take neighbouring
+//    shares and merge their sums through distributed shared memory.  Products are m16n8k16 warp MMAs; queries and weights enter
+//    as the sum of two bf16 terms, so they keep 16 significant bits;
+//  * latent_attention_simt_kernel: the same in fp32 arithmetic, for any size and either cache type.
+//    For one token the partial sums of the clusters (or blocks) go to memory; the values' mat-vec behind them merges them
+//    while it stages its input (head_matvec_kernel);
 //  * latent_prefill_tc_kernel: many tokens over expanded keys and values (a GEMM over the cache makes them), bf16.  A block of
 //    eight warps owns 128 consecutive tokens of one head; tiles of 64 keys -- the head's own part, and the shared rotated part
 //    straight from the cache -- stream through a two-deep cp.async ring, products are m16n8k16 warp MMAs with fp32
 //    accumulators, the softmax runs online.  The weights enter the value product as the sum of two bf16 terms.
+#include <cooperative_groups.h>
 #include <cuda_bf16.h>
 
 #include "attn_common.cuh"
 #include "common.cuh"
 #include "dense_common.cuh"
 #include "kernels.h"
+
+namespace cg = cooperative_groups;
 
 namespace cutb {
 namespace {
@@ -207,6 +214,237 @@ template <typename KV> __global__ void __launch_bounds__(LA_THREADS) latent_atte
     }
   }
   if (sp.part && tid < nh) sp.ml[(size_t)(h0 + tid) * sp.splits + split] = make_float2(head_m[tid], head_l[tid]);
+}
+
+// ---- absorbed form on the tensor cores ---------------------------------------------------------------------------------
+constexpr int LD_THREADS = 256, LD_WARPS = 8, LD_HEADS = 16, LD_KEYS = 32, LD_CLUSTER = 8, LD_PAD = 8;
+
+// shared memory: queries (high and low parts), two key tiles (afterwards the block's sums), the new row
+__host__ __device__ inline uint32_t ld_stride(uint32_t row_len) { return (row_len + 15) / 16 * 16 + LD_PAD; }
+uint32_t ld_smem_bytes(const cutb_latent_attn_desc &d) {
+  const uint32_t st = ld_stride(d.rot_at + (d.rot_dim + 7) / 8 * 8), tiles = 2 * LD_KEYS * st * 2, sums = LD_HEADS * ((d.rank + 3) / 4 * 4) * 4;
+  return 2 * LD_HEADS * st * 2 + (tiles > sums ? tiles : sums) + st * 2;
+}
+bool ld_applies(const cutb_latent_attn_desc &d) { return d.kv_dtype == CUTB_BF16 && d.rank <= 1024 && ld_smem_bytes(d) <= 220 * 1024; }
+
+// NC: 16-column pieces of the latent per warp.  grid = (head groups, shares, tokens), cluster (1, 8, 1).
+template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc_kernel(const cutb_latent_attn_desc d, const LatentSplit sp, uint32_t row_len) {
+  extern __shared__ __align__(16) uint8_t ld_smem[];
+  __shared__ float sc[2][LD_HEADS][LD_KEYS + 1];                   // scores, a half of the row each
+  __shared__ __align__(16) __nv_bfloat16 ps[2][LD_HEADS][LD_KEYS + 8];  // weights, high and low parts
+  __shared__ float head_m[LD_HEADS], head_l[LD_HEADS], fac[LD_HEADS], part[LD_WARPS];
+  cg::cluster_group cluster = cg::this_cluster();
+  const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h0 = blockIdx.x * LD_HEADS, split = blockIdx.y, shares = gridDim.y, tok = blockIdx.z;
+  const uint32_t nh = min((uint32_t)LD_HEADS, d.n_heads - h0), width = d.dim + d.rot_dim, st = ld_stride(row_len), steps = (st - LD_PAD) / 16;
+  __nv_bfloat16 *qh = reinterpret_cast<__nv_bfloat16 *>(ld_smem), *ql = qh + LD_HEADS * st, *tiles = ql + LD_HEADS * st;
+  float *sums = reinterpret_cast<float *>(tiles);
+  const uint32_t tile_bytes = LD_KEYS * st * 2, tiles_len = 2 * tile_bytes, sums_ld = (d.rank + 3) / 4 * 4, sums_len = LD_HEADS * sums_ld * 4;
+  __nv_bfloat16 *fresh = reinterpret_cast<__nv_bfloat16 *>(reinterpret_cast<uint8_t *>(tiles) + (tiles_len > sums_len ? tiles_len : sums_len));
+  const uint32_t qh_u = smem_u32(qh), ql_u = smem_u32(ql), tile_u = smem_u32(tiles), ps_u = smem_u32(ps);
+  asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  pdl_enter();
+  const uint32_t pos = (d.pos_ptr ? *d.pos_ptr : d.pos) + tok;
+  if (pos >= d.max_pos) {  // (the same in every block of the cluster)
+    if (d.status && tid == 0) atomicExch(d.status, (int)CUTB_ERR_INVALID);
+    return;
+  }
+  const uint32_t n = pos + 1, per = (n + shares - 1) / shares, k_lo = min(split * per, n), k_hi = min(k_lo + per, n);
+  const __nv_bfloat16 *cache = reinterpret_cast<const __nv_bfloat16 *>(d.cache);
+  const bool make = d.lat && k_hi == n && k_lo < n;  // this block's keys end with the token's own
+  const uint32_t pieces = (st - LD_PAD) / 8;
+  auto load_tile = [&](uint32_t k0, uint32_t buf) {
+    for (uint32_t r = warp; r < LD_KEYS; r += LD_WARPS) {
+      const uint32_t key = k0 + r;
+      const bool in = key < k_hi && !(make && key == pos);
+      const __nv_bfloat16 *src = cache + (size_t)key * d.ld_cache;
+      const uint32_t dst = tile_u + buf * tile_bytes + r * st * 2;
+      for (uint32_t c = lane; c < pieces; c += 32) {
+        if (in && c * 8 < row_len) cp_async16(dst + c * 16, src + c * 8);
+        else *reinterpret_cast<uint4 *>(reinterpret_cast<uint8_t *>(tiles) + buf * tile_bytes + r * st * 2 + c * 16) = make_uint4(0, 0, 0, 0);
+      }
+    }
+    cp_async_commit();
+  };
+  if (k_lo < k_hi) load_tile(k_lo, 0);
+
+  // queries laid out as a cache row, scaled to log2 units, zeros in its gaps and past the last head
+  const float scale = d.scale * LA_LOG2E;
+  const uint32_t half = d.rot_dim / 2;
+  for (uint32_t r = warp; r < LD_HEADS; r += LD_WARPS) {
+    const float *qa = d.qa + tok * d.ld_qa + (size_t)(h0 + r) * d.rank, *q = d.q + tok * d.ldq + (size_t)(h0 + r) * width + d.dim;
+#pragma unroll 4
+    for (uint32_t e = lane * 2; e < st - LD_PAD; e += 64) {
+      float u = 0.f, v = 0.f;
+      if (r < nh) {
+        if (e < d.rank) {
+          u = qa[e] * scale;
+          if (e + 1 < d.rank) v = qa[e + 1] * scale;
+        } else if (e >= d.rot_at && e < d.rot_at + d.rot_dim) {
+          const uint32_t i = (e - d.rot_at) / 2;
+          const float c = __ldg(d.cos_table + (size_t)pos * half + i), s = __ldg(d.sin_table + (size_t)pos * half + i);
+          const float a = q[2 * i], b = q[2 * i + 1];
+          u = (a * c - b * s) * scale, v = (b * c + a * s) * scale;
+        }
+      }
+      uint32_t hi, lo;
+      split_bf16(u, v, hi, lo);
+      *reinterpret_cast<uint32_t *>(qh + r * st + e) = hi;
+      *reinterpret_cast<uint32_t *>(ql + r * st + e) = lo;
+    }
+  }
+  if (make) {
+    __nv_bfloat16 *row = reinterpret_cast<__nv_bfloat16 *>(d.cache) + pos * d.ld_cache;
+    for (uint32_t i = tid; i < st; i += LD_THREADS) fresh[i] = __float2bfloat16_rn(0.f);
+    __syncthreads();
+    make_cache_row(d, tok, pos, part, [&](uint32_t i, float v) {
+      fresh[i] = __float2bfloat16_rn(v);
+      if (blockIdx.x == 0) row[i] = fresh[i];
+    });
+  }
+  if (tid < LD_HEADS) {
+    const bool sink = d.sink && split == 0 && tid < nh;
+    head_m[tid] = sink ? d.sink[h0 + tid] * LA_LOG2E : LA_NEG, head_l[tid] = sink ? 1.f : 0.f;
+  }
+  const uint32_t g = lane >> 2, tg = lane & 3, mat = lane >> 3, mr = lane & 7;
+  float o[2 * NC][4];
+#pragma unroll
+  for (int j = 0; j < 2 * NC; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+  const uint32_t col0 = warp * NC * 16;  // this warp's columns of the latent
+  const uint32_t s_half = warp >> 2, s_n = warp & 3;  // and its part of the scores: half the row, eight keys
+  const uint32_t s_first = s_half ? (steps + 1) / 2 : 0, s_last = s_half ? steps : (steps + 1) / 2;
+
+  for (uint32_t k0 = k_lo, turn = 0; k0 < k_hi; k0 += LD_KEYS, ++turn) {
+    const uint32_t buf = turn & 1, cnt = min((uint32_t)LD_KEYS, k_hi - k0);
+    if (k0 + LD_KEYS < k_hi) {
+      load_tile(k0 + LD_KEYS, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    if (make && pos - k0 < cnt) {  // the row made here
+      for (uint32_t c = tid; c < pieces; c += LD_THREADS)
+        *reinterpret_cast<uint4 *>(reinterpret_cast<uint8_t *>(tiles) + buf * tile_bytes + (pos - k0) * st * 2 + c * 16) = reinterpret_cast<const uint4 *>(fresh)[c];
+      __syncthreads();
+    }
+    const uint32_t t_u = tile_u + buf * tile_bytes;
+    {  // scores of 16 heads x 8 keys over half the row; high and low query parts in sums of their own
+      float s0[4] = {}, s1[4] = {};
+      const uint32_t a_off = ((mat & 1) * 8 + mr) * st + (mat >> 1) * 8, b_off = (s_n * 8 + mr) * st + mat * 8;
+      uint32_t k = s_first;
+      for (; k + 1 < s_last; k += 2) {
+        uint32_t ah[4], al[4], b0, b1, b2, b3;
+        ldsm_x4(t_u + (b_off + k * 16) * 2, b0, b1, b2, b3);
+        ldsm_x4(qh_u + (a_off + k * 16) * 2, ah[0], ah[1], ah[2], ah[3]);
+        ldsm_x4(ql_u + (a_off + k * 16) * 2, al[0], al[1], al[2], al[3]);
+        mma_bf16(s0, ah, b0, b1);
+        mma_bf16(s1, al, b0, b1);
+        ldsm_x4(qh_u + (a_off + k * 16 + 16) * 2, ah[0], ah[1], ah[2], ah[3]);
+        ldsm_x4(ql_u + (a_off + k * 16 + 16) * 2, al[0], al[1], al[2], al[3]);
+        mma_bf16(s0, ah, b2, b3);
+        mma_bf16(s1, al, b2, b3);
+      }
+      if (k < s_last) {
+        uint32_t ah[4], al[4], b0, b1, b2, b3;
+        // (lanes 16 and up would address past the last step: they repeat the first half's rows)
+        ldsm_x4(t_u + ((s_n * 8 + mr) * st + (mat & 1) * 8 + k * 16) * 2, b0, b1, b2, b3);
+        ldsm_x4(qh_u + (a_off + k * 16) * 2, ah[0], ah[1], ah[2], ah[3]);
+        ldsm_x4(ql_u + (a_off + k * 16) * 2, al[0], al[1], al[2], al[3]);
+        mma_bf16(s0, ah, b0, b1);
+        mma_bf16(s1, al, b0, b1);
+      }
+      const uint32_t c = s_n * 8 + 2 * tg;
+      sc[s_half][g][c] = s0[0] + s1[0], sc[s_half][g][c + 1] = s0[1] + s1[1];
+      sc[s_half][g + 8][c] = s0[2] + s1[2], sc[s_half][g + 8][c + 1] = s0[3] + s1[3];
+    }
+    __syncthreads();
+#pragma unroll
+    for (uint32_t i = 0; i < LD_HEADS / LD_WARPS; ++i) {  // softmax: a warp per head, a lane per key
+      const uint32_t r = warp + i * LD_WARPS;
+      const float v = lane < cnt ? sc[0][r][lane] + sc[1][r][lane] : -INFINITY, before = head_m[r];
+      float m = fmaxf(v, before);
+#pragma unroll
+      for (int w = 16; w > 0; w >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, w));
+      const float e = exp2f(v - m);
+      float l = e;
+#pragma unroll
+      for (int w = 16; w > 0; w >>= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
+      const __nv_bfloat16 hi = __float2bfloat16_rn(e);
+      ps[0][r][lane] = hi;
+      ps[1][r][lane] = __float2bfloat16_rn(e - __bfloat162float(hi));
+      if (lane == 0) {
+        const float f = exp2f(before - m);
+        head_l[r] = fmaf(head_l[r], f, l), head_m[r] = m, fac[r] = f;
+      }
+    }
+    __syncthreads();
+    if (col0 < d.rank) {
+      const float f_lo = fac[g], f_hi = fac[g + 8];
+#pragma unroll
+      for (int j = 0; j < 2 * NC; ++j) o[j][0] *= f_lo, o[j][1] *= f_lo, o[j][2] *= f_hi, o[j][3] *= f_hi;
+#pragma unroll
+      for (int kk = 0; kk < LD_KEYS / 16; ++kk) {
+        uint32_t ph[4], pl[4];
+        const uint32_t a_off = ((mat & 1) * 8 + mr) * (LD_KEYS + 8) + kk * 16 + (mat >> 1) * 8;
+        ldsm_x4(ps_u + a_off * 2, ph[0], ph[1], ph[2], ph[3]);
+        ldsm_x4(ps_u + (LD_HEADS * (LD_KEYS + 8) + a_off) * 2, pl[0], pl[1], pl[2], pl[3]);
+#pragma unroll
+        for (int j2 = 0; j2 < NC; ++j2) {
+          const uint32_t row = kk * 16 + (mat & 1) * 8 + mr, col = col0 + j2 * 16 + (mat >> 1) * 8;
+          if (col0 + j2 * 16 < d.rank) {
+            uint32_t b0, b1, b2, b3;
+            ldsm_x4_trans(t_u + (row * st + col) * 2, b0, b1, b2, b3);
+            mma_bf16(o[2 * j2], ph, b0, b1);
+            mma_bf16(o[2 * j2 + 1], ph, b2, b3);
+            mma_bf16(o[2 * j2], pl, b0, b1);
+            mma_bf16(o[2 * j2 + 1], pl, b2, b3);
+          }
+        }
+      }
+    }
+    __syncthreads();  // the tile is free for the copy issued next turn
+  }
+
+  // the block's sums, then the cluster's
+#pragma unroll
+  for (int j = 0; j < 2 * NC; ++j) {
+    const uint32_t c = col0 + j * 8 + 2 * tg;
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (c + (e & 1) < d.rank) sums[(e < 2 ? g : g + 8) * sums_ld + c + (e & 1)] = o[j][e];
+  }
+  cluster.sync();
+  const uint32_t me = cluster.block_rank(), out_split = split / LD_CLUSTER, out_splits = shares / LD_CLUSTER;
+  const uint32_t quads = sums_ld / 4;
+  for (uint32_t i = me * LD_THREADS + tid; i < nh * quads; i += LD_CLUSTER * LD_THREADS) {
+    const uint32_t r = i / quads, c = i % quads * 4;
+    float mk[LD_CLUSTER], lk[LD_CLUSTER], m = LA_NEG, l = 0.f;
+    float4 ak[LD_CLUSTER], s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (uint32_t k = 0; k < LD_CLUSTER; ++k) {  // every remote read in flight at once
+      mk[k] = *cluster.map_shared_rank(&head_m[r], k);
+      lk[k] = *cluster.map_shared_rank(&head_l[r], k);
+      ak[k] = *reinterpret_cast<const float4 *>(cluster.map_shared_rank(&sums[r * sums_ld + c], k));
+    }
+#pragma unroll
+    for (uint32_t k = 0; k < LD_CLUSTER; ++k) m = fmaxf(m, mk[k]);
+#pragma unroll
+    for (uint32_t k = 0; k < LD_CLUSTER; ++k) {
+      const float w = exp2f(mk[k] - m);
+      l = fmaf(w, lk[k], l);
+      s.x = fmaf(w, ak[k].x, s.x), s.y = fmaf(w, ak[k].y, s.y), s.z = fmaf(w, ak[k].z, s.z), s.w = fmaf(w, ak[k].w, s.w);
+    }
+    if (sp.part) {
+      *reinterpret_cast<float4 *>(sp.part + ((size_t)(h0 + r) * out_splits + out_split) * sp.ld + c) = s;
+      if (c == 0) sp.ml[(size_t)(h0 + r) * out_splits + out_split] = make_float2(m, l);
+    } else {
+      const float inv = 1.0f / l, v[4] = {s.x * inv, s.y * inv, s.z * inv, s.w * inv};
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (c + e < d.rank) store_out(d.out, d.out_dtype == CUTB_BF16, tok * d.ldo + (size_t)(h0 + r) * d.rank + c + e, v[e]);
+    }
+  }
+  cluster.sync();  // nobody leaves while its shared memory may still be read
 }
 
 // ---- expanded form on the tensor cores ---------------------------------------------------------------------------------
@@ -420,12 +658,41 @@ LatentSplit split_of(const cutb_latent_attn_desc &d) {
   return s;
 }
 
+template <int NC> int ld_launch(const cutb_latent_attn_desc &d, const LatentSplit &sp, uint32_t row_len, cudaStream_t stream) {
+  const uint32_t smem = ld_smem_bytes(d);
+  CUTB_CUDA_TRY(cudaFuncSetAttribute(latent_decode_tc_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((d.n_heads + LD_HEADS - 1) / LD_HEADS, sp.splits * LD_CLUSTER, d.n_tokens);
+  cfg.blockDim = dim3(LD_THREADS);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = 1;
+  attr[0].val.clusterDim.y = LD_CLUSTER;
+  attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = 2;
+  CUTB_CUDA_TRY(cudaLaunchKernelEx(&cfg, latent_decode_tc_kernel<NC>, d, sp, row_len));
+  return CUTB_OK;
+}
+
 }  // namespace
 
 uint32_t latent_splits(const cutb_latent_attn_desc &d) {
   if (d.n_tokens != 1) return 1;
   DeviceInfo di;
-  const uint32_t sms = get_device_info(&di) == CUTB_OK ? (uint32_t)di.sm_count : 148u, groups = (d.n_heads + LS_HEADS - 1) / LS_HEADS;
+  const uint32_t sms = get_device_info(&di) == CUTB_OK ? (uint32_t)di.sm_count : 148u;
+  if (ld_applies(d)) {  // clusters per head group: as many as run at once, at least 16 keys per block at the full context
+    const uint32_t groups = (d.n_heads + LD_HEADS - 1) / LD_HEADS;
+    uint32_t s = sms / (groups * LD_CLUSTER), most = (d.max_pos + 16 * LD_CLUSTER - 1) / (16 * LD_CLUSTER);
+    if (s > most) s = most;
+    if (s > 16) s = 16;
+    return s < 1 ? 1 : s;
+  }
+  const uint32_t groups = (d.n_heads + LS_HEADS - 1) / LS_HEADS;
   uint32_t s = 2 * sms / groups, most = (d.max_pos + 31) / 32;
   if (s > most) s = most;
   if (s > 64) s = 64;
@@ -442,6 +709,11 @@ int latent_kv_write_launch(const cutb_latent_attn_desc &d, cudaStream_t stream) 
 int latent_attention_launch(const cutb_latent_attn_desc &d, cudaStream_t stream) {
   const LatentSplit sp = split_of(d);
   const uint32_t row_len = d.rot_at + (d.rot_dim + 7) / 8 * 8, smem = 4 * row_len * (LS_HEADS + 1);
+  if (ld_applies(d)) {
+    if (d.rank <= 128) return ld_launch<1>(d, sp, row_len, stream);
+    if (d.rank <= 256) return ld_launch<2>(d, sp, row_len, stream);
+    return d.rank <= 512 ? ld_launch<4>(d, sp, row_len, stream) : ld_launch<8>(d, sp, row_len, stream);
+  }
   const dim3 grid((d.n_heads + LS_HEADS - 1) / LS_HEADS, sp.splits, d.n_tokens);
   auto go = [&](auto kernel) -> int {
     if (smem > 48 * 1024) CUTB_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));

@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(32 * MR_WARPS) moe_route_kernel(const cutb_moe
   }
 }
 
-constexpr int MS_THREADS = 256;
+constexpr int MS_THREADS = 1024;
 
 // Thread i owns the i-th stretch of the choices; two passes over it: count, then number.
 __global__ void __launch_bounds__(MS_THREADS) moe_sort_kernel(const uint32_t *ids, uint32_t n, uint32_t experts, uint32_t *slots, uint32_t *offsets) {
