@@ -228,6 +228,14 @@ template <int LPR> __global__ void __launch_bounds__(HV_THREADS) head_matvec_ker
     if (p.splits) {
       const float2 *ml = p.ml + (size_t)(h0 + h) * p.splits;
       const float *part = p.part + (size_t)(h0 + h) * p.splits * p.ld_part;
+      float a[2][16];  // the first ones are on their way while their shares are worked out
+#pragma unroll
+      for (uint32_t i = 0; i < 2; ++i)
+#pragma unroll
+        for (uint32_t s = 0; s < 16; ++s) {
+          const uint32_t k = tid + i * HV_THREADS;
+          a[i][s] = k < p.K && s < p.splits ? part[(size_t)s * p.ld_part + k] : 0.f;
+        }
       if (warp == 0) {  // a partial sum's share: exp2(its maximum - the largest) / the whole weight sum
         const float2 a = lane < p.splits ? ml[lane] : make_float2(-1e30f, 0.f), b = lane + 32 < p.splits ? ml[lane + 32] : make_float2(-1e30f, 0.f);
         float m = fmaxf(a.x, b.x);
@@ -238,12 +246,18 @@ template <int LPR> __global__ void __launch_bounds__(HV_THREADS) head_matvec_ker
         share[lane] = wa * inv, share[lane + 32] = wb * inv;
       }
       __syncthreads();
-      for (uint32_t k = tid; k < 8 * K8; k += HV_THREADS) {
+#pragma unroll
+      for (uint32_t i = 0; i < 2; ++i) {
+        const uint32_t k = tid + i * HV_THREADS;
         float v = 0.f;
-        if (k < p.K) {
-#pragma unroll 8
-          for (uint32_t s = 0; s < p.splits; ++s) v = fmaf(share[s], part[(size_t)s * p.ld_part + k], v);
-        }
+#pragma unroll
+        for (uint32_t s = 0; s < 16; ++s) v = fmaf(share[s], a[i][s], v);
+        for (uint32_t s = 16; s < p.splits && k < p.K; ++s) v = fmaf(share[s], part[(size_t)s * p.ld_part + k], v);
+        if (k < 8 * K8) put(h, k, v);
+      }
+      for (uint32_t k = tid + 2 * HV_THREADS; k < 8 * K8; k += HV_THREADS) {
+        float v = 0.f;
+        for (uint32_t s = 0; s < p.splits && k < p.K; ++s) v = fmaf(share[s], part[(size_t)s * p.ld_part + k], v);
         put(h, k, v);
       }
       __syncthreads();

@@ -20,7 +20,8 @@
 namespace cutb {
 namespace {
 
-constexpr int EX_MIN_WARPS = 16, EX_MAX_WARPS = 24, EX_MAX_THREADS = 32 * EX_MAX_WARPS;
+constexpr int EX_MIN_WARPS = 16;
+constexpr int ex_max_warps(bool up) { return up ? 24 : 28; }
 constexpr uint32_t EX_MAX_TOP = 64;
 
 struct ExParams {
@@ -36,7 +37,7 @@ struct ExParams {
   GluParams glu;
 };
 
-template <bool UP> __global__ void __launch_bounds__(EX_MAX_THREADS, 1) expert_matvec_kernel(const ExParams p) {
+template <bool UP> __global__ void __launch_bounds__(32 * ex_max_warps(UP), 1) expert_matvec_kernel(const ExParams p) {
   constexpr int R = UP ? 2 : 1, UNR = UP ? 2 : 4;
   extern __shared__ __align__(16) float ex_smem[];
   __shared__ uint32_t ids[EX_MAX_TOP];
@@ -219,7 +220,7 @@ template <bool UP> int ex_launch(const cutb_expert_desc &d, cudaStream_t stream)
     CUTB_CUDA_TRY(cudaFuncSetAttribute(expert_matvec_kernel<UP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)di.smem_optin - 2048));
     if (dev >= 0 && dev < 64) configured[dev] = true;
   }
-  const uint32_t sms = (uint32_t)di.sm_count, per_sm = (p.ntiles + sms - 1) / sms, turns = (per_sm + EX_MAX_WARPS - 1) / EX_MAX_WARPS;
+  const uint32_t sms = (uint32_t)di.sm_count, per_sm = (p.ntiles + sms - 1) / sms, most = ex_max_warps(UP), turns = (per_sm + most - 1) / most;
   uint32_t warps = (per_sm + turns - 1) / turns;
   if (warps < EX_MIN_WARPS) warps = EX_MIN_WARPS;
   const dim3 grid(p.ntiles < sms ? p.ntiles : sms), block(32 * warps);

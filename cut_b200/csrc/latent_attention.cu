@@ -217,12 +217,13 @@ template <typename KV> __global__ void __launch_bounds__(LA_THREADS) latent_atte
 }
 
 // ---- absorbed form on the tensor cores ---------------------------------------------------------------------------------
-constexpr int LD_THREADS = 256, LD_WARPS = 8, LD_HEADS = 16, LD_KEYS = 32, LD_CLUSTER = 8, LD_PAD = 8;
+constexpr int LD_THREADS = 256, LD_WARPS = 8, LD_HEADS = 16, LD_KEYS = 16, LD_STAGES = 3, LD_CLUSTER = 8, LD_PAD = 8;
 
-// shared memory: queries (high and low parts), two key tiles (afterwards the block's sums), the new row
+// shared memory: queries (high and low parts), a ring of key tiles (afterwards the block's sums), the new row.  Below 112 KB two
+// blocks share an SM, so that 32 clusters run at once.
 __host__ __device__ inline uint32_t ld_stride(uint32_t row_len) { return (row_len + 15) / 16 * 16 + LD_PAD; }
 uint32_t ld_smem_bytes(const cutb_latent_attn_desc &d) {
-  const uint32_t st = ld_stride(d.rot_at + (d.rot_dim + 7) / 8 * 8), tiles = 2 * LD_KEYS * st * 2, sums = LD_HEADS * ((d.rank + 3) / 4 * 4) * 4;
+  const uint32_t st = ld_stride(d.rot_at + (d.rot_dim + 7) / 8 * 8), tiles = LD_STAGES * LD_KEYS * st * 2, sums = LD_HEADS * ((d.rank + 3) / 4 * 4) * 4;
   return 2 * LD_HEADS * st * 2 + (tiles > sums ? tiles : sums) + st * 2;
 }
 bool ld_applies(const cutb_latent_attn_desc &d) { return d.kv_dtype == CUTB_BF16 && d.rank <= 1024 && ld_smem_bytes(d) <= 220 * 1024; }
@@ -230,7 +231,7 @@ bool ld_applies(const cutb_latent_attn_desc &d) { return d.kv_dtype == CUTB_BF16
 // NC: 16-column pieces of the latent per warp.  grid = (head groups, shares, tokens), cluster (1, 8, 1).
 template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc_kernel(const cutb_latent_attn_desc d, const LatentSplit sp, uint32_t row_len) {
   extern __shared__ __align__(16) uint8_t ld_smem[];
-  __shared__ float sc[2][LD_HEADS][LD_KEYS + 1];                   // scores, a half of the row each
+  __shared__ float sc[4][LD_HEADS][LD_KEYS + 1];                        // scores, a quarter of the row each
   __shared__ __align__(16) __nv_bfloat16 ps[2][LD_HEADS][LD_KEYS + 8];  // weights, high and low parts
   __shared__ float head_m[LD_HEADS], head_l[LD_HEADS], fac[LD_HEADS], part[LD_WARPS];
   cg::cluster_group cluster = cg::this_cluster();
@@ -238,11 +239,26 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
   const uint32_t nh = min((uint32_t)LD_HEADS, d.n_heads - h0), width = d.dim + d.rot_dim, st = ld_stride(row_len), steps = (st - LD_PAD) / 16;
   __nv_bfloat16 *qh = reinterpret_cast<__nv_bfloat16 *>(ld_smem), *ql = qh + LD_HEADS * st, *tiles = ql + LD_HEADS * st;
   float *sums = reinterpret_cast<float *>(tiles);
-  const uint32_t tile_bytes = LD_KEYS * st * 2, tiles_len = 2 * tile_bytes, sums_ld = (d.rank + 3) / 4 * 4, sums_len = LD_HEADS * sums_ld * 4;
+  const uint32_t tile_bytes = LD_KEYS * st * 2, tiles_len = LD_STAGES * tile_bytes, sums_ld = (d.rank + 3) / 4 * 4, sums_len = LD_HEADS * sums_ld * 4;
   __nv_bfloat16 *fresh = reinterpret_cast<__nv_bfloat16 *>(reinterpret_cast<uint8_t *>(tiles) + (tiles_len > sums_len ? tiles_len : sums_len));
   const uint32_t qh_u = smem_u32(qh), ql_u = smem_u32(ql), tile_u = smem_u32(tiles), ps_u = smem_u32(ps);
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
   pdl_enter();
+  // the first latent parts of the queries (a warp per two heads, eight pairs per lane) are on their way before anything else
+  const float *qa0 = d.qa + tok * d.ld_qa + (size_t)h0 * d.rank, *q0 = d.q + tok * d.ldq + (size_t)h0 * width + d.dim;
+  constexpr uint32_t QH = LD_HEADS / LD_WARPS;
+  float u[QH][4], v[QH][4];
+  auto load_q = [&](uint32_t e0) {
+#pragma unroll
+    for (uint32_t i = 0; i < QH; ++i)
+#pragma unroll
+      for (uint32_t j = 0; j < 4; ++j) {
+        const uint32_t r = warp + i * LD_WARPS, e = e0 + j * 64 + lane * 2;
+        const float *qa = qa0 + (size_t)r * d.rank + e;
+        u[i][j] = r < nh && e < d.rank ? qa[0] : 0.f, v[i][j] = r < nh && e + 1 < d.rank ? qa[1] : 0.f;
+      }
+  };
+  load_q(0);
   const uint32_t pos = (d.pos_ptr ? *d.pos_ptr : d.pos) + tok;
   if (pos >= d.max_pos) {  // (the same in every block of the cluster)
     if (d.status && tid == 0) atomicExch(d.status, (int)CUTB_ERR_INVALID);
@@ -263,34 +279,52 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
         else *reinterpret_cast<uint4 *>(reinterpret_cast<uint8_t *>(tiles) + buf * tile_bytes + r * st * 2 + c * 16) = make_uint4(0, 0, 0, 0);
       }
     }
-    cp_async_commit();
   };
-  if (k_lo < k_hi) load_tile(k_lo, 0);
+#pragma unroll
+  for (uint32_t i = 0; i + 1 < LD_STAGES; ++i) {
+    if (k_lo + i * LD_KEYS < k_hi) load_tile(k_lo + i * LD_KEYS, i);
+    cp_async_commit();
+  }
 
   // queries laid out as a cache row, scaled to log2 units, zeros in its gaps and past the last head
   const float scale = d.scale * LA_LOG2E;
   const uint32_t half = d.rot_dim / 2;
-  for (uint32_t r = warp; r < LD_HEADS; r += LD_WARPS) {
-    const float *qa = d.qa + tok * d.ld_qa + (size_t)(h0 + r) * d.rank, *q = d.q + tok * d.ldq + (size_t)(h0 + r) * width + d.dim;
-#pragma unroll 4
-    for (uint32_t e = lane * 2; e < st - LD_PAD; e += 64) {
-      float u = 0.f, v = 0.f;
-      if (r < nh) {
-        if (e < d.rank) {
-          u = qa[e] * scale;
-          if (e + 1 < d.rank) v = qa[e + 1] * scale;
-        } else if (e >= d.rot_at && e < d.rot_at + d.rot_dim) {
-          const uint32_t i = (e - d.rot_at) / 2;
-          const float c = __ldg(d.cos_table + (size_t)pos * half + i), s = __ldg(d.sin_table + (size_t)pos * half + i);
-          const float a = q[2 * i], b = q[2 * i + 1];
-          u = (a * c - b * s) * scale, v = (b * c + a * s) * scale;
-        }
+  auto put_q = [&](uint32_t r, uint32_t e, float u, float v) {
+    uint32_t hi, lo;
+    split_bf16(u, v, hi, lo);
+    *reinterpret_cast<uint32_t *>(qh + r * st + e) = hi;
+    *reinterpret_cast<uint32_t *>(ql + r * st + e) = lo;
+  };
+  constexpr int RU = 2;
+  float ra[RU], rb[RU], rc[RU], rs[RU];
+#pragma unroll
+  for (int u = 0; u < RU; ++u) {
+    const uint32_t i = tid + u * LD_THREADS, r = half ? i / half : 0, e = half ? i - r * half : 0;
+    const bool in = half && r < nh;
+    ra[u] = in ? q0[(size_t)r * width + 2 * e] : 0.f, rb[u] = in ? q0[(size_t)r * width + 2 * e + 1] : 0.f;
+    rc[u] = in ? __ldg(d.cos_table + (size_t)pos * half + e) : 0.f, rs[u] = in ? __ldg(d.sin_table + (size_t)pos * half + e) : 0.f;
+  }
+  for (uint32_t e0 = 0; e0 < st - LD_PAD; e0 += 256) {
+    if (e0) load_q(e0);
+#pragma unroll
+    for (uint32_t i = 0; i < QH; ++i)
+#pragma unroll
+      for (uint32_t j = 0; j < 4; ++j) {
+        const uint32_t e = e0 + j * 64 + lane * 2;
+        if (e < st - LD_PAD) put_q(warp + i * LD_WARPS, e, u[i][j] * scale, v[i][j] * scale);
       }
-      uint32_t hi, lo;
-      split_bf16(u, v, hi, lo);
-      *reinterpret_cast<uint32_t *>(qh + r * st + e) = hi;
-      *reinterpret_cast<uint32_t *>(ql + r * st + e) = lo;
-    }
+  }
+  __syncthreads();  // (the turned part overwrites zeros)
+#pragma unroll
+  for (int u = 0; u < RU; ++u) {
+    const uint32_t i = tid + u * LD_THREADS, r = half ? i / half : 0, e = half ? i - r * half : 0;
+    if (half && r < nh) put_q(r, d.rot_at + 2 * e, (ra[u] * rc[u] - rb[u] * rs[u]) * scale, (rb[u] * rc[u] + ra[u] * rs[u]) * scale);
+  }
+  for (uint32_t i = tid + RU * LD_THREADS; i < nh * half; i += LD_THREADS) {
+    const uint32_t r = i / half, e = i - r * half;
+    const float c = __ldg(d.cos_table + (size_t)pos * half + e), s = __ldg(d.sin_table + (size_t)pos * half + e);
+    const float a = q0[(size_t)r * width + 2 * e], b = q0[(size_t)r * width + 2 * e + 1];
+    put_q(r, d.rot_at + 2 * e, (a * c - b * s) * scale, (b * c + a * s) * scale);
   }
   if (make) {
     __nv_bfloat16 *row = reinterpret_cast<__nv_bfloat16 *>(d.cache) + pos * d.ld_cache;
@@ -310,17 +344,14 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
 #pragma unroll
   for (int j = 0; j < 2 * NC; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
   const uint32_t col0 = warp * NC * 16;  // this warp's columns of the latent
-  const uint32_t s_half = warp >> 2, s_n = warp & 3;  // and its part of the scores: half the row, eight keys
-  const uint32_t s_first = s_half ? (steps + 1) / 2 : 0, s_last = s_half ? steps : (steps + 1) / 2;
+  const uint32_t s_part = warp >> 1, s_n = warp & 1;  // and its part of the scores: a quarter of the row, eight keys
+  const uint32_t s_first = steps * s_part / 4, s_last = steps * (s_part + 1) / 4;
 
   for (uint32_t k0 = k_lo, turn = 0; k0 < k_hi; k0 += LD_KEYS, ++turn) {
-    const uint32_t buf = turn & 1, cnt = min((uint32_t)LD_KEYS, k_hi - k0);
-    if (k0 + LD_KEYS < k_hi) {
-      load_tile(k0 + LD_KEYS, buf ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
+    const uint32_t buf = turn % LD_STAGES, cnt = min((uint32_t)LD_KEYS, k_hi - k0);
+    if (k0 + (LD_STAGES - 1) * LD_KEYS < k_hi) load_tile(k0 + (LD_STAGES - 1) * LD_KEYS, (turn + LD_STAGES - 1) % LD_STAGES);
+    cp_async_commit();
+    cp_async_wait<LD_STAGES - 1>();
     __syncthreads();
     if (make && pos - k0 < cnt) {  // the row made here
       for (uint32_t c = tid; c < pieces; c += LD_THREADS)
@@ -328,7 +359,7 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
       __syncthreads();
     }
     const uint32_t t_u = tile_u + buf * tile_bytes;
-    {  // scores of 16 heads x 8 keys over half the row; high and low query parts in sums of their own
+    {  // scores of 16 heads x 8 keys over a quarter of the row; high and low query parts in sums of their own
       float s0[4] = {}, s1[4] = {};
       const uint32_t a_off = ((mat & 1) * 8 + mr) * st + (mat >> 1) * 8, b_off = (s_n * 8 + mr) * st + mat * 8;
       uint32_t k = s_first;
@@ -354,25 +385,26 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
         mma_bf16(s1, al, b0, b1);
       }
       const uint32_t c = s_n * 8 + 2 * tg;
-      sc[s_half][g][c] = s0[0] + s1[0], sc[s_half][g][c + 1] = s0[1] + s1[1];
-      sc[s_half][g + 8][c] = s0[2] + s1[2], sc[s_half][g + 8][c + 1] = s0[3] + s1[3];
+      sc[s_part][g][c] = s0[0] + s1[0], sc[s_part][g][c + 1] = s0[1] + s1[1];
+      sc[s_part][g + 8][c] = s0[2] + s1[2], sc[s_part][g + 8][c + 1] = s0[3] + s1[3];
     }
     __syncthreads();
+    {  // softmax: half a warp per head, a lane per key
+      static_assert(LD_KEYS == 16 && LD_HEADS == 2 * LD_WARPS, "a head per 16 lanes");
+      const uint32_t r = warp * 2 + (lane >> 4), key = lane & 15;
+      const float x = key < cnt ? (sc[0][r][key] + sc[1][r][key]) + (sc[2][r][key] + sc[3][r][key]) : -INFINITY, before = head_m[r];
+      float m = fmaxf(x, before);
 #pragma unroll
-    for (uint32_t i = 0; i < LD_HEADS / LD_WARPS; ++i) {  // softmax: a warp per head, a lane per key
-      const uint32_t r = warp + i * LD_WARPS;
-      const float v = lane < cnt ? sc[0][r][lane] + sc[1][r][lane] : -INFINITY, before = head_m[r];
-      float m = fmaxf(v, before);
-#pragma unroll
-      for (int w = 16; w > 0; w >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, w));
-      const float e = exp2f(v - m);
+      for (int w = 8; w > 0; w >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, w));
+      const float e = exp2f(x - m);
       float l = e;
 #pragma unroll
-      for (int w = 16; w > 0; w >>= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
+      for (int w = 8; w > 0; w >>= 1) l += __shfl_xor_sync(0xffffffffu, l, w);
       const __nv_bfloat16 hi = __float2bfloat16_rn(e);
-      ps[0][r][lane] = hi;
-      ps[1][r][lane] = __float2bfloat16_rn(e - __bfloat162float(hi));
-      if (lane == 0) {
+      ps[0][r][key] = hi;
+      ps[1][r][key] = __float2bfloat16_rn(e - __bfloat162float(hi));
+      __syncwarp();
+      if (key == 0) {
         const float f = exp2f(before - m);
         head_l[r] = fmaf(head_l[r], f, l), head_m[r] = m, fac[r] = f;
       }
@@ -687,7 +719,7 @@ uint32_t latent_splits(const cutb_latent_attn_desc &d) {
   const uint32_t sms = get_device_info(&di) == CUTB_OK ? (uint32_t)di.sm_count : 148u;
   if (ld_applies(d)) {  // clusters per head group: as many as run at once, at least 16 keys per block at the full context
     const uint32_t groups = (d.n_heads + LD_HEADS - 1) / LD_HEADS;
-    uint32_t s = sms / (groups * LD_CLUSTER), most = (d.max_pos + 16 * LD_CLUSTER - 1) / (16 * LD_CLUSTER);
+    uint32_t s = (2 * sms > 40 ? 2 * sms - 40 : 1) / (groups * LD_CLUSTER), most = (d.max_pos + 16 * LD_CLUSTER - 1) / (16 * LD_CLUSTER);
     if (s > most) s = most;
     if (s > 16) s = 16;
     return s < 1 ? 1 : s;
