@@ -39,7 +39,7 @@ EXPORTS = [
     "cutb_variant_name",
     "cutb_dense_select_variant", "cutb_dense_workspace_bytes", "cutb_dense_matmul", "cutb_residual_norm", "cutb_embedding_bigram",
     "cutb_mingru_scan", "cutb_sequence_advance", "cutb_window_kv_write", "cutb_window_attention", "cutb_window_attention_decode",
-    "cutb_latent_kv_write", "cutb_latent_attention", "cutb_latent_splits", "cutb_latent_workspace_bytes", "cutb_latent_values",
+    "cutb_latent_kv_write", "cutb_latent_attention", "cutb_latent_takes_split_queries", "cutb_latent_splits", "cutb_latent_workspace_bytes", "cutb_latent_values",
     "cutb_latent_prefill_supported", "cutb_latent_prefill", "cutb_moe_route", "cutb_moe_scatter", "cutb_moe_matmul", "cutb_expert_up",
     "cutb_expert_down",
 ]
@@ -79,6 +79,7 @@ class DenseDesc(C.Structure):
         ("gru_state", C.c_void_p),
         ("norm_center", C.c_int32), ("res_scale", C.c_float), ("norm_out", C.c_void_p),
         ("batch", C.c_uint32), ("a_batch", C.c_uint32), ("c_batch", C.c_uint32),
+        ("c_low", C.c_void_p), ("c_scale", C.c_float),
     ]
 
 
@@ -141,6 +142,7 @@ class LatentAttnDesc(C.Structure):
         ("workspace", C.c_void_p), ("workspace_bytes", C.c_uint64),
         ("status", C.c_void_p),
         ("w_uv", C.c_void_p), ("ld_uv", C.c_uint64),
+        ("qa_high", C.c_void_p), ("qa_low", C.c_void_p), ("ld_qa_split", C.c_uint64),
     ]
 
 
@@ -215,7 +217,8 @@ def _bind_layers(l: C.CDLL) -> None:
                        ("cutb_expert_down", ExpertDesc)):
         getattr(l, name).restype = C.c_int
         getattr(l, name).argtypes = [C.POINTER(desc), C.c_void_p]
-    for name, kind in (("cutb_latent_splits", C.c_uint32), ("cutb_latent_workspace_bytes", C.c_uint64), ("cutb_latent_prefill_supported", C.c_int)):
+    for name, kind in (("cutb_latent_splits", C.c_uint32), ("cutb_latent_workspace_bytes", C.c_uint64), ("cutb_latent_prefill_supported", C.c_int),
+                       ("cutb_latent_takes_split_queries", C.c_int)):
         getattr(l, name).restype = kind
         getattr(l, name).argtypes = [C.POINTER(LatentAttnDesc)]
     l.cutb_dense_select_variant.restype = C.c_int

@@ -58,6 +58,10 @@ int check_dense(const cutb_dense_desc *d) {
     set_last_error("dense_matmul: a batch of products has no bias, no elementwise op and no fused steps, and its columns lie within the rows");
     return CUTB_ERR_INVALID;
   }
+  if (d->c_low && (d->M != 1 || d->c_dtype != CUTB_BF16 || d->batch < 2)) {
+    set_last_error("dense_matmul: results in two terms are those of a batch for one row, in bf16");
+    return CUTB_ERR_INVALID;
+  }
   if (d->gru_state && (d->M != 1 || d->N % 3)) {
     set_last_error("dense_matmul: the recurrence step needs one row and three stacked matrices");
     return CUTB_ERR_INVALID;
@@ -373,6 +377,10 @@ int cutb_latent_kv_write(const cutb_latent_attn_desc *d, void *stream) {
 
 uint32_t cutb_latent_splits(const cutb_latent_attn_desc *d) { return check_latent(d, "latent_splits", false) == CUTB_OK ? latent_splits(*d) : 0; }
 
+int cutb_latent_takes_split_queries(const cutb_latent_attn_desc *d) {
+  return check_latent(d, "latent_takes_split_queries", false) == CUTB_OK && latent_takes_split_queries(*d) ? 1 : 0;
+}
+
 uint64_t cutb_latent_workspace_bytes(const cutb_latent_attn_desc *d) {
   if (check_latent(d, "latent_workspace", false) != CUTB_OK || d->n_tokens != 1) return 0;
   const uint64_t n = (uint64_t)d->n_heads * latent_splits(*d);
@@ -381,7 +389,12 @@ uint64_t cutb_latent_workspace_bytes(const cutb_latent_attn_desc *d) {
 
 int cutb_latent_attention(const cutb_latent_attn_desc *d, void *stream) {
   if (int rc = check_latent(d, "latent_attention", true)) return rc;
-  if (!d->q || !d->qa || (d->lat && d->n_tokens != 1) || (d->n_tokens != 1 && (!d->out || d->ldo < (uint64_t)d->n_heads * d->rank)) ||
+  if (d->qa_high && (!d->qa_low || !latent_takes_split_queries(*d) || d->ld_qa_split % 8 || d->ld_qa_split < d->rank ||
+                     (reinterpret_cast<uintptr_t>(d->qa_high) | reinterpret_cast<uintptr_t>(d->qa_low)) % 16)) {
+    set_last_error("latent_attention: queries in two terms need one token, a bf16 cache and 16-byte aligned rows");
+    return CUTB_ERR_INVALID;
+  }
+  if (!d->q || (!d->qa && !d->qa_high) || (d->lat && d->n_tokens != 1) || (d->n_tokens != 1 && (!d->out || d->ldo < (uint64_t)d->n_heads * d->rank)) ||
       (d->n_tokens > 1 && (d->ldq < (uint64_t)d->n_heads * (d->dim + d->rot_dim) || d->ld_qa < (uint64_t)d->n_heads * d->rank))) {
     set_last_error("latent_attention: null pointer, short rows, or a cache row to make for more than one token");
     return CUTB_ERR_INVALID;

@@ -279,7 +279,17 @@ template <int LPR> __global__ void __launch_bounds__(HV_THREADS) head_matvec_ker
     }
 #pragma unroll
     for (int o = LPR / 2; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-    if (sub == 0 && row < r1) store_out(p.C, p.c_bf16, (size_t)(row / p.N) * p.c_batch + row % p.N, acc);
+    if (sub == 0 && row < r1) {
+      const size_t at = (size_t)(row / p.N) * p.c_batch + row % p.N;
+      if (p.c_low) {
+        acc *= p.scale;
+        const __nv_bfloat16 high = __float2bfloat16_rn(acc);
+        reinterpret_cast<__nv_bfloat16 *>(p.C)[at] = high;
+        reinterpret_cast<__nv_bfloat16 *>(p.c_low)[at] = __float2bfloat16_rn(acc - __bfloat162float(high));
+      } else {
+        store_out(p.C, p.c_bf16, at, acc);
+      }
+    }
   }
 }
 
@@ -329,6 +339,7 @@ int dense_matvec_launch(const cutb_dense_desc &d, cudaStream_t stream) {
   if (d.batch > 1) {
     HeadMvParams h{};
     h.x = reinterpret_cast<const float *>(d.A), h.x_batch = d.a_batch, h.W = d.W, h.C = d.C, h.c_bf16 = d.c_dtype == CUTB_BF16;
+    h.c_low = d.c_low, h.scale = d.c_scale;
     h.batch = d.batch, h.K = d.K, h.K8 = (d.K + 7) / 8, h.N = d.N, h.ldw8 = d.ldw / 8, h.c_batch = d.c_batch;
     return head_matvec_launch(h, stream);
   }

@@ -95,6 +95,8 @@ struct HeadMvParams {
   const float2 *ml;
   const float *part;
   uint32_t splits, ld_part;
+  void *c_low;  // with it: C (bf16) + c_low (bf16) = scale * the product
+  float scale;
 };
 int head_matvec_launch(const HeadMvParams &p, cudaStream_t stream);
 int moe_gemm_tc_launch(const cutb_moe_desc &d, cudaStream_t stream);
@@ -105,6 +107,7 @@ bool expert_matvec_supported(const cutb_expert_desc &d, bool up);
 int expert_up_launch(const cutb_expert_desc &d, cudaStream_t stream);
 int expert_down_launch(const cutb_expert_desc &d, cudaStream_t stream);
 uint32_t latent_splits(const cutb_latent_attn_desc &d);
+bool latent_takes_split_queries(const cutb_latent_attn_desc &d);
 int latent_kv_write_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);
 int latent_attention_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);
 int latent_values_launch(const cutb_latent_attn_desc &d, cudaStream_t stream);

@@ -222,8 +222,9 @@ constexpr int LD_THREADS = 256, LD_WARPS = 8, LD_HEADS = 16, LD_KEYS = 16, LD_ST
 // shared memory: queries (high and low parts), a ring of key tiles (afterwards the block's sums), the new row.  Below 112 KB two
 // blocks share an SM, so that 32 clusters run at once.
 __host__ __device__ inline uint32_t ld_stride(uint32_t row_len) { return (row_len + 15) / 16 * 16 + LD_PAD; }
+__host__ __device__ inline uint32_t ld_sums_stride(uint32_t rank) { return (rank + 31) / 32 * 32 + 8; }  // (rows eight banks apart)
 uint32_t ld_smem_bytes(const cutb_latent_attn_desc &d) {
-  const uint32_t st = ld_stride(d.rot_at + (d.rot_dim + 7) / 8 * 8), tiles = LD_STAGES * LD_KEYS * st * 2, sums = LD_HEADS * ((d.rank + 3) / 4 * 4) * 4;
+  const uint32_t st = ld_stride(d.rot_at + (d.rot_dim + 7) / 8 * 8), tiles = LD_STAGES * LD_KEYS * st * 2, sums = LD_HEADS * ld_sums_stride(d.rank) * 4;
   return 2 * LD_HEADS * st * 2 + (tiles > sums ? tiles : sums) + st * 2;
 }
 bool ld_applies(const cutb_latent_attn_desc &d) { return d.kv_dtype == CUTB_BF16 && d.rank <= 1024 && ld_smem_bytes(d) <= 220 * 1024; }
@@ -234,16 +235,32 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
   __shared__ float sc[4][LD_HEADS][LD_KEYS + 1];                        // scores, a quarter of the row each
   __shared__ __align__(16) __nv_bfloat16 ps[2][LD_HEADS][LD_KEYS + 8];  // weights, high and low parts
   __shared__ float head_m[LD_HEADS], head_l[LD_HEADS], fac[LD_HEADS], part[LD_WARPS];
+  __shared__ float2 all_ml[LD_CLUSTER][LD_HEADS];  // every block's maxima and weight sums
   cg::cluster_group cluster = cg::this_cluster();
   const uint32_t tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h0 = blockIdx.x * LD_HEADS, split = blockIdx.y, shares = gridDim.y, tok = blockIdx.z;
   const uint32_t nh = min((uint32_t)LD_HEADS, d.n_heads - h0), width = d.dim + d.rot_dim, st = ld_stride(row_len), steps = (st - LD_PAD) / 16;
   __nv_bfloat16 *qh = reinterpret_cast<__nv_bfloat16 *>(ld_smem), *ql = qh + LD_HEADS * st, *tiles = ql + LD_HEADS * st;
   float *sums = reinterpret_cast<float *>(tiles);
-  const uint32_t tile_bytes = LD_KEYS * st * 2, tiles_len = LD_STAGES * tile_bytes, sums_ld = (d.rank + 3) / 4 * 4, sums_len = LD_HEADS * sums_ld * 4;
+  const uint32_t tile_bytes = LD_KEYS * st * 2, tiles_len = LD_STAGES * tile_bytes, sums_ld = ld_sums_stride(d.rank), sums_len = LD_HEADS * sums_ld * 4;
   __nv_bfloat16 *fresh = reinterpret_cast<__nv_bfloat16 *>(reinterpret_cast<uint8_t *>(tiles) + (tiles_len > sums_len ? tiles_len : sums_len));
   const uint32_t qh_u = smem_u32(qh), ql_u = smem_u32(ql), tile_u = smem_u32(tiles), ps_u = smem_u32(ps);
   asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+  asm volatile("barrier.cluster.arrive.aligned;" ::: "memory");  // (waited for before the first access to another block)
   pdl_enter();
+  const bool split_q = d.qa_high != nullptr;
+  if (split_q) {  // the latent parts as they are, asynchronously
+    const __nv_bfloat16 *gh = reinterpret_cast<const __nv_bfloat16 *>(d.qa_high) + h0 * d.ld_qa_split, *gl = reinterpret_cast<const __nv_bfloat16 *>(d.qa_low) + h0 * d.ld_qa_split;
+    for (uint32_t r = warp; r < LD_HEADS; r += LD_WARPS)
+      for (uint32_t c = lane * 8; c < st - LD_PAD; c += 256) {
+        const uint32_t at = r * st + c;
+        if (r < nh && c < d.rot_at) {
+          cp_async16(qh_u + at * 2, gh + r * d.ld_qa_split + c);
+          cp_async16(ql_u + at * 2, gl + r * d.ld_qa_split + c);
+        } else {
+          *reinterpret_cast<uint4 *>(qh + at) = *reinterpret_cast<uint4 *>(ql + at) = make_uint4(0, 0, 0, 0);
+        }
+      }
+  }
   // the first latent parts of the queries (a warp per two heads, eight pairs per lane) are on their way before anything else
   const float *qa0 = d.qa + tok * d.ld_qa + (size_t)h0 * d.rank, *q0 = d.q + tok * d.ldq + (size_t)h0 * width + d.dim;
   constexpr uint32_t QH = LD_HEADS / LD_WARPS;
@@ -258,10 +275,12 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
         u[i][j] = r < nh && e < d.rank ? qa[0] : 0.f, v[i][j] = r < nh && e + 1 < d.rank ? qa[1] : 0.f;
       }
   };
-  load_q(0);
+  if (!split_q) load_q(0);
   const uint32_t pos = (d.pos_ptr ? *d.pos_ptr : d.pos) + tok;
   if (pos >= d.max_pos) {  // (the same in every block of the cluster)
     if (d.status && tid == 0) atomicExch(d.status, (int)CUTB_ERR_INVALID);
+    cp_async_wait<0>();
+    asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
     return;
   }
   const uint32_t n = pos + 1, per = (n + shares - 1) / shares, k_lo = min(split * per, n), k_hi = min(k_lo + per, n);
@@ -304,7 +323,7 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
     ra[u] = in ? q0[(size_t)r * width + 2 * e] : 0.f, rb[u] = in ? q0[(size_t)r * width + 2 * e + 1] : 0.f;
     rc[u] = in ? __ldg(d.cos_table + (size_t)pos * half + e) : 0.f, rs[u] = in ? __ldg(d.sin_table + (size_t)pos * half + e) : 0.f;
   }
-  for (uint32_t e0 = 0; e0 < st - LD_PAD; e0 += 256) {
+  for (uint32_t e0 = 0; e0 < st - LD_PAD && !split_q; e0 += 256) {
     if (e0) load_q(e0);
 #pragma unroll
     for (uint32_t i = 0; i < QH; ++i)
@@ -437,33 +456,38 @@ template <int NC> __global__ void __launch_bounds__(LD_THREADS) latent_decode_tc
     __syncthreads();  // the tile is free for the copy issued next turn
   }
 
-  // the block's sums, then the cluster's
+  // the block's sums, then the cluster's; maxima and weight sums go to every block
+  cp_async_wait<0>();
+  __syncthreads();
 #pragma unroll
   for (int j = 0; j < 2 * NC; ++j) {
     const uint32_t c = col0 + j * 8 + 2 * tg;
-#pragma unroll
-    for (int e = 0; e < 4; ++e)
-      if (c + (e & 1) < d.rank) sums[(e < 2 ? g : g + 8) * sums_ld + c + (e & 1)] = o[j][e];
+    if (c < d.rank) {
+      *reinterpret_cast<float2 *>(sums + g * sums_ld + c) = make_float2(o[j][0], o[j][1]);
+      *reinterpret_cast<float2 *>(sums + (g + 8) * sums_ld + c) = make_float2(o[j][2], o[j][3]);
+    }
+  }
+  asm volatile("barrier.cluster.wait.aligned;" ::: "memory");
+  if (tid < LD_CLUSTER * LD_HEADS) {
+    const uint32_t r = tid % LD_HEADS;
+    *cluster.map_shared_rank(&all_ml[cluster.block_rank()][r], tid / LD_HEADS) = make_float2(head_m[r], head_l[r]);
   }
   cluster.sync();
   const uint32_t me = cluster.block_rank(), out_split = split / LD_CLUSTER, out_splits = shares / LD_CLUSTER;
-  const uint32_t quads = sums_ld / 4;
+  const uint32_t quads = (d.rank + 3) / 4;
   for (uint32_t i = me * LD_THREADS + tid; i < nh * quads; i += LD_CLUSTER * LD_THREADS) {
     const uint32_t r = i / quads, c = i % quads * 4;
-    float mk[LD_CLUSTER], lk[LD_CLUSTER], m = LA_NEG, l = 0.f;
+    float m = LA_NEG, l = 0.f;
     float4 ak[LD_CLUSTER], s = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-    for (uint32_t k = 0; k < LD_CLUSTER; ++k) {  // every remote read in flight at once
-      mk[k] = *cluster.map_shared_rank(&head_m[r], k);
-      lk[k] = *cluster.map_shared_rank(&head_l[r], k);
+    for (uint32_t k = 0; k < LD_CLUSTER; ++k)  // every remote read in flight at once
       ak[k] = *reinterpret_cast<const float4 *>(cluster.map_shared_rank(&sums[r * sums_ld + c], k));
-    }
 #pragma unroll
-    for (uint32_t k = 0; k < LD_CLUSTER; ++k) m = fmaxf(m, mk[k]);
+    for (uint32_t k = 0; k < LD_CLUSTER; ++k) m = fmaxf(m, all_ml[k][r].x);
 #pragma unroll
     for (uint32_t k = 0; k < LD_CLUSTER; ++k) {
-      const float w = exp2f(mk[k] - m);
-      l = fmaf(w, lk[k], l);
+      const float w = exp2f(all_ml[k][r].x - m);
+      l = fmaf(w, all_ml[k][r].y, l);
       s.x = fmaf(w, ak[k].x, s.x), s.y = fmaf(w, ak[k].y, s.y), s.z = fmaf(w, ak[k].z, s.z), s.w = fmaf(w, ak[k].w, s.w);
     }
     if (sp.part) {
@@ -712,6 +736,8 @@ template <int NC> int ld_launch(const cutb_latent_attn_desc &d, const LatentSpli
 }
 
 }  // namespace
+
+bool latent_takes_split_queries(const cutb_latent_attn_desc &d) { return d.n_tokens == 1 && ld_applies(d); }
 
 uint32_t latent_splits(const cutb_latent_attn_desc &d) {
   if (d.n_tokens != 1) return 1;

@@ -272,7 +272,7 @@ class _LatentShapes:
         self.tables = tuple(torch.from_numpy(t).cuda() for t in rotation_tables(Rotation(10000.0, rot), ctx))
         f = lambda *s: torch.randn(s, device="cuda")
         self.cache = f(ctx, pad(rank, 8) + pad(rot, 8)).to(torch.bfloat16)
-        self.q, self.qa, self.lat, self.cq = f(T, H * (dim + rot)), f(1, H * rank), f(T, rank + rot), f(T, q_rank)
+        self.q, self.qa, self.lat, self.cq = f(T, H * (dim + rot)), _bf16(2, H, pad(rank, 8)), f(T, rank + rot), f(T, q_rank)
         self.one, self.sink = torch.ones(max(rank, q_rank), device="cuda"), torch.zeros(H, device="cuda")
         self.cq_out = torch.zeros((T, q_rank), device="cuda", dtype=torch.bfloat16)
         self.out = torch.zeros((T, H * vdim), device="cuda", dtype=torch.bfloat16)
@@ -289,7 +289,7 @@ def latent_decode_us(H, dim, rot, vdim, rank, ctx):
     n = _copies(ctx * (rank + rot) * 2)
     sets = [_LatentShapes(H, dim, rot, vdim, rank, 64, 1, ctx) for _ in range(n)]
     ws = torch.zeros(ops.latent_workspace_bytes(sets[0].desc()) // 4, device="cuda")
-    att = [s.desc(q=s.q, qa=s.qa, workspace=ws, lat=s.lat, lat_norm_w=s.one) for s in sets]
+    att = [s.desc(q=s.q, qa_split=(s.qa[0], s.qa[1]), workspace=ws, lat=s.lat, lat_norm_w=s.one) for s in sets]
     a = time_us(_graph_calls("cutb_latent_attention", att))
     Ws, out = [_bf16(H * vdim, rank) for _ in range(_copies(H * vdim * rank * 2))], torch.zeros((1, H * vdim), device="cuda")
     v = time_us(_graph_calls("cutb_latent_values", [sets[0].desc(out=out, workspace=ws, w_uv=W) for W in Ws]))

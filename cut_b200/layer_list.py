@@ -242,6 +242,8 @@ class Addend:
     parts: tuple | None = None
 
 
+LOG2_E = 1.4426950408889634
+
 # Portions of at least this many tokens expand the cached latents into every head's keys and values; fewer stay in latent space.
 EXPAND_TOKENS = 32
 
@@ -472,7 +474,7 @@ class LayerListDecoder:
     # -- a portion of a prompt ----------------------------------------------------------------------------------------
     def _sizes(self) -> dict:
         """Columns of the activation buffers: what any layer needs of each."""
-        cfg, n = self.cfg, dict.fromkeys(("pre", "mid", "first", "q", "lat", "cq", "logits", "top", "experts", "act", "workspace"), 0)
+        cfg, n = self.cfg, dict.fromkeys(("pre", "mid", "first", "q", "lat", "lat_split", "cq", "logits", "top", "experts", "act", "workspace"), 0)
 
         def need(**sizes):
             for k, v in sizes.items():
@@ -482,7 +484,7 @@ class LayerListDecoder:
             need(pre=d["in"].N, mid=max(d["out"].K, d["up"].N if "up" in d else 0))  # pre-activations of a mixer, fp32; its output
             if isinstance(l.mixer, LatentAttention):
                 m = l.mixer
-                need(q=m.q_rows, lat=m.heads * m.kv_rank, cq=m.q_rank)
+                need(q=m.q_rows, lat=m.heads * m.kv_rank, lat_split=m.heads * pad(m.kv_rank, 8), cq=m.q_rank)
                 cos_t, sin_t = self._tables[m.rot]
                 need(workspace=ops.latent_workspace_bytes(ops.latent_desc(
                     torch.empty((1, m.cache_row)), m.heads, m.dim, m.rot.dims, m.vdim, m.kv_rank, scale=m.scale, eps=cfg.norm_eps,
@@ -628,7 +630,7 @@ class LayerListDecoder:
         n = self._sizes()
         e = lambda cols: torch.zeros((1, cols), dtype=torch.float32, device=self.dev) if cols else None
         return {"x": [e(self.ldx), e(self.ldx)], "y": e(self.ldx), "h": e(self.ldx), "pre": e(n["pre"]), "mid": e(n["mid"]), "first": e(n["first"]),
-                "q": e(n["q"]), "lat": e(n["lat"]), "router": e(n["logits"]), "act": e(n["act"]),
+                "q": e(n["q"]), "lat": e(n["lat"]), "lat_split": torch.zeros(2 * n["lat_split"], dtype=torch.bfloat16, device=self.dev), "router": e(n["logits"]), "act": e(n["act"]),
                 "ids": torch.zeros(max(1, n["top"]), dtype=torch.int32, device=self.dev),
                 "workspace": torch.zeros(max(4, n["workspace"] // 4), dtype=torch.float32, device=self.dev),
                 "logits": e(pad(self.cfg.vocab, 8)), "next": torch.zeros(1, dtype=torch.float32, device=self.dev)}
@@ -671,9 +673,17 @@ class LayerListDecoder:
                         eps=cfg.norm_eps, out=b["q"])
             else:
                 call("cutb_dense_matmul", ops.stage_input(self._dense_desc(d["uq"], 1, None, b["q"]), pre, d["cq_norm"], 1, cfg.norm_eps))
-            call("cutb_dense_matmul", ops.batch_desc(b["q"], d["absorb"].w, m.dim, b["lat"], m.heads, m.dim + m.rot.dims, m.kv_rank, status=self.status))
             own = {"lat": pre[:, m.q_rank:], "lat_norm_w": d["c_norm"]} if m.kv_from is None else {}
-            call("cutb_latent_attention", self._latent_desc(i, seq, 1, q=b["q"], qa=b["lat"], workspace=b["workspace"], **own))
+            attention = self._latent_desc(i, seq, 1, q=b["q"], qa=b["lat"], workspace=b["workspace"], **own)
+            if m.heads > 1 and ops.latent_takes_split_queries(attention):  # the absorbed queries as the tensor cores read them
+                row = pad(m.kv_rank, 8)
+                high, low = b["lat_split"][: 2 * m.heads * row].view(2, m.heads, row)
+                attention = self._latent_desc(i, seq, 1, q=b["q"], qa_split=(high, low), workspace=b["workspace"], **own)
+                call("cutb_dense_matmul", ops.batch_desc(b["q"], d["absorb"].w, m.dim, high, m.heads, m.dim + m.rot.dims, row, status=self.status,
+                                                         low=low, scale=m.scale * LOG2_E))
+            else:
+                call("cutb_dense_matmul", ops.batch_desc(b["q"], d["absorb"].w, m.dim, b["lat"], m.heads, m.dim + m.rot.dims, m.kv_rank, status=self.status))
+            call("cutb_latent_attention", attention)
             call("cutb_latent_values", self._latent_desc(i, seq, 1, out=b["mid"], workspace=b["workspace"], w_uv=d["uv"].w))
             if f is not None:
                 experts(f, d, "cutb_expert_down", dense=d["out"].w, dense_K=d["out"].K, xd=b["mid"], out=b["y"])

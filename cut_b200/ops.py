@@ -335,10 +335,12 @@ def stage_input(d, x: torch.Tensor, norm_w: torch.Tensor, groups: int, eps: floa
     return d
 
 
-def batch_desc(A: torch.Tensor, W: torch.Tensor, K: int, out: torch.Tensor, heads: int, a_step: int, c_step: int, *, status=None):
-    """cutb_dense_desc of `heads` products: number b maps columns b * a_step .. + K of A by rows b N .. of W to columns b * c_step .. of out."""
+def batch_desc(A: torch.Tensor, W: torch.Tensor, K: int, out: torch.Tensor, heads: int, a_step: int, c_step: int, *, status=None, low=None,
+               scale: float = 1.0):
+    """cutb_dense_desc of `heads` products: number b maps columns b * a_step .. + K of A by rows b N .. of W to columns b * c_step .. of out.
+    low (one row, bf16 out): the results times scale as the sum of out and low."""
     d = dense_desc(A, W, K, out, status=status, N=W.shape[0] // heads)
-    d.batch, d.a_batch, d.c_batch = heads, a_step, c_step
+    d.batch, d.a_batch, d.c_batch, d.c_low, d.c_scale = heads, a_step, c_step, _ptr(low), scale
     return d
 
 
@@ -437,7 +439,7 @@ def window_attention_decode(d) -> None:
 # ---- latent attention, mixtures of experts ----
 def latent_desc(cache: torch.Tensor, n_heads: int, dim: int, rot_dim: int, vdim: int, rank: int, *, scale: float, eps: float, max_pos: int,
                 n_tokens: int, cos_t=None, sin_t=None, sink=None, pos: int = 0, pos_ptr: int | None = None, lat=None, lat_norm_w=None, cq=None,
-                cq_norm_w=None, cq_out=None, q=None, qa=None, k_exp=None, v_exp=None, out=None, workspace=None, w_uv=None, status=None):
+                cq_norm_w=None, cq_out=None, q=None, qa=None, qa_split=None, k_exp=None, v_exp=None, out=None, workspace=None, w_uv=None, status=None):
     """cutb_latent_attn_desc over a cache [rows, pad8(rank) + pad8(rot_dim)]; what a call does not use may be missing."""
     d = L.LatentAttnDesc()
     shape = out if out is not None else cq_out
@@ -454,9 +456,15 @@ def latent_desc(cache: torch.Tensor, n_heads: int, dim: int, rot_dim: int, vdim:
         if t is not None:
             setattr(d, name, t.data_ptr())
             setattr(d, {"q": "ldq", "qa": "ld_qa", "k_exp": "ld_k", "v_exp": "ld_v", "out": "ldo", "w_uv": "ld_uv"}[name], t.stride(0))
+    if qa_split is not None:  # (high, low) [heads, pad8(rank)] bf16
+        d.qa_high, d.qa_low, d.ld_qa_split = qa_split[0].data_ptr(), qa_split[1].data_ptr(), qa_split[0].stride(0)
     if workspace is not None:
         d.workspace, d.workspace_bytes = workspace.data_ptr(), workspace.numel() * workspace.element_size()
     return d
+
+
+def latent_takes_split_queries(d) -> bool:
+    return bool(L.lib().cutb_latent_takes_split_queries(C.byref(d)))
 
 
 def latent_workspace_bytes(d) -> int:

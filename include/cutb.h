@@ -451,7 +451,8 @@ enum { CUTB_DENSE_AUTO = -1, CUTB_DENSE_MATVEC = 0, CUTB_DENSE_TC = 1, CUTB_DENS
  *   CUTB_DENSE_SIMT    fp32 fused multiply-adds, A fp32 or bf16: the true 32-bit path of a prefill.
  * CUTB_DENSE_AUTO: one row -> mat-vec, more bf16 rows -> tensor cores, fp32 rows -> SIMT.
  * batch > 1 (mat-vec and SIMT; no fused steps): `batch` products of these sizes, number b over the columns b * a_batch on of A,
- * the rows b * N on of W and the columns b * c_batch on of C (a matrix per head).
+ * the rows b * N on of W and the columns b * c_batch on of C (a matrix per head).  One row with c_low set (c_dtype bf16): the
+ * results times c_scale as the sum of two bf16 terms, the high part in C and the low part in c_low.
  */
 typedef struct cutb_dense_desc {
   int32_t a_dtype, c_dtype;
@@ -478,6 +479,8 @@ typedef struct cutb_dense_desc {
   float res_scale;
   float *norm_out;
   uint32_t batch, a_batch, c_batch;
+  void *c_low;
+  float c_scale;
 } cutb_dense_desc;
 CUTB_API int cutb_dense_select_variant(const cutb_dense_desc *desc);
 CUTB_API uint64_t cutb_dense_workspace_bytes(const cutb_dense_desc *desc);
@@ -588,7 +591,8 @@ CUTB_API int cutb_window_attention_decode(const cutb_window_attn_desc *desc, voi
  *       pre-activations (lat null: nothing is cached); and the latent queries cq_out = N(cq; cq_norm_w), q_rank elements (cq
  *       null: none).  N = RMS norm.
  *   cutb_latent_attention   absorbed form: q [T][ldq] holds each head's dim + rot_dim elements (the turned part is read), qa
- *       [T][ld_qa] each head's W_uk,h^T q_h (rank elements); out [T][ldo] = each head's weighted sum of latents.  With lat
+ *       [T][ld_qa] each head's W_uk,h^T q_h (rank elements); or, for one token, qa_high + qa_low (bf16, rows of ld_qa_split elements
+ *       per head, a multiple of 8, zero past rank) hold them times scale * log2(e) (cutb_latent_takes_split_queries); out [T][ldo] = each head's weighted sum of latents.  With lat
  *       set (one token only) the call also makes, uses and stores that token's cache row.  For one token the keys are shared
  *       out over cutb_latent_splits() blocks per head group: their partial sums go to `workspace`, and the product over W_uv
  *       that follows reads them there (cutb_latent_values).
@@ -620,9 +624,12 @@ typedef struct cutb_latent_attn_desc {
   int *status;
   const void *w_uv; /* cutb_latent_values: bf16 [n_heads * vdim][ld_uv] */
   uint64_t ld_uv;
+  const void *qa_high, *qa_low;
+  uint64_t ld_qa_split;
 } cutb_latent_attn_desc;
 CUTB_API int cutb_latent_kv_write(const cutb_latent_attn_desc *desc, void *stream);
 CUTB_API int cutb_latent_attention(const cutb_latent_attn_desc *desc, void *stream);
+CUTB_API int cutb_latent_takes_split_queries(const cutb_latent_attn_desc *desc);
 CUTB_API uint32_t cutb_latent_splits(const cutb_latent_attn_desc *desc);
 CUTB_API uint64_t cutb_latent_workspace_bytes(const cutb_latent_attn_desc *desc);
 CUTB_API int cutb_latent_values(const cutb_latent_attn_desc *desc, void *stream);

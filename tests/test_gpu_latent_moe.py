@@ -115,6 +115,10 @@ def test_product_per_head(heads, K, N, step):
         out = torch.full((rows, pad(heads * N, 8) + 8), 7.0, device="cuda")
         ops.dense_matmul(ops.batch_desc(a[:rows], w, K, out, heads, step, N))
         assert rel(out[:, : heads * N], want[:rows]) < 2e-6 and bool((out[:, heads * N:] == 7.0).all()), rows
+    two = torch.zeros((2, 1, heads * (N + 3)), device="cuda", dtype=torch.bfloat16)  # one row, scaled, as the sum of two bf16 terms
+    ops.dense_matmul(ops.batch_desc(a[:1], w, K, two[0], heads, step, N + 3, low=two[1], scale=0.3))
+    got = (two[0].double() + two[1].double()).view(heads, N + 3)
+    assert rel(got[:, :N].reshape(-1), 0.3 * want[0]) < 2e-5 and not got[:, N:].any()
 
 
 # ---- mixture of experts ----------------------------------------------------------------------------------------------------
@@ -315,9 +319,15 @@ class Latent:
     def one(self, a, out, own):
         H, dim, rot, vdim, rank = self.p
         q, qa = dev(self.q[a:a + 1]), torch.zeros((1, H * rank), device="cuda")
-        ops.dense_matmul(self.heads(q, self.absorb, dim, qa, dim + rot, rank))
         ws = torch.full((ops.latent_workspace_bytes(self.desc(a, a + 1)) // 4,), float("nan"), device="cuda")
-        ops.launch_layer_op("cutb_latent_attention", self.desc(a, a + 1, q=q, qa=qa, workspace=ws, **own))
+        if a % 2 and H > 1 and ops.latent_takes_split_queries(self.desc(a, a + 1)):  # every other token: the queries in two bf16 terms
+            two = torch.zeros((2, H, pad(rank, 8)), device="cuda", dtype=torch.bfloat16)
+            ops.dense_matmul(ops.batch_desc(q, self.absorb, dim, two[0], H, dim + rot, pad(rank, 8), low=two[1], scale=self.scale * layer_list.LOG2_E))
+            queries = {"qa_split": (two[0], two[1])}
+        else:
+            ops.dense_matmul(self.heads(q, self.absorb, dim, qa, dim + rot, rank))
+            queries = {"qa": qa}
+        ops.launch_layer_op("cutb_latent_attention", self.desc(a, a + 1, q=q, workspace=ws, **queries, **own))
         ops.launch_layer_op("cutb_latent_values", self.desc(a, a + 1, out=out[a:a + 1], workspace=ws, w_uv=self.w_uv))
 
 
