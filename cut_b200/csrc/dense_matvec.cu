@@ -49,7 +49,7 @@ struct MvParams {
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void *src) {
   asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
-template <int R, int UNR, bool GRU>
+template <int R, int UNR, bool GRU, bool PLAIN>
 __global__ void __launch_bounds__(MV_MAX_THREADS, 1) dense_matvec_kernel(const MvParams p) {
   extern __shared__ __align__(16) float mv_smem[];
   float4 *lo = reinterpret_cast<float4 *>(mv_smem), *hi = lo + p.K8;  // activation planes
@@ -94,18 +94,18 @@ __global__ void __launch_bounds__(MV_MAX_THREADS, 1) dense_matvec_kernel(const M
   // ---- the activation row -> two planes, zero past K ----
   auto put1 = [&](uint32_t i, float v) { mv_smem[(i & 4 ? 4 * p.K8 : 0) + (i >> 3) * 4 + (i & 3)] = v; };
   auto put4 = [&](uint32_t i, float4 v) { (i & 4 ? hi : lo)[i >> 3] = v; };
-  float *keep = blockIdx.x == 0 ? p.norm_out : nullptr;
+  float *keep = !GRU && blockIdx.x == 0 ? p.norm_out : nullptr;
   auto norm1 = [&](uint32_t i, float v) {
     put1(i, v);
-    if (keep) keep[i] = v;
+    if (!GRU && keep) keep[i] = v;
   };
   auto norm4 = [&](uint32_t i, float4 v) {
     put4(i, v);
-    if (keep) *reinterpret_cast<float4 *>(keep + i) = v;
+    if (!GRU && keep) *reinterpret_cast<float4 *>(keep + i) = v;
   };
   for (uint32_t i = p.K + tid; i < 8 * p.K8; i += nt) put1(i, 0.f);
   if (fast_norm) {
-    stage_norm_regs<2>(p.norm, stage + 2 * p.K, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, norm4);
+    stage_norm_regs<2, PLAIN>(p.norm, stage + 2 * p.K, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, norm4);
   } else if (p.norm.pre_w) {
     stage_norm(p.norm, stage, blockIdx.x == 0 && p.norm.x_out != nullptr, norm4, norm1);
   } else if (p.a_bf16) {
@@ -177,14 +177,14 @@ __global__ void __launch_bounds__(MV_MAX_THREADS, 1) dense_matvec_kernel(const M
   }
 }
 
-template <int R, int UNR, bool GRU> int mv_launch(MvParams &p, uint32_t smem, uint32_t sms, bool overlap, cudaStream_t stream) {
+template <int R, int UNR, bool GRU, bool PLAIN> int mv_launch(MvParams &p, uint32_t smem, uint32_t sms, bool overlap, cudaStream_t stream) {
   static bool configured[64] = {};
   int dev = 0;
   CUTB_CUDA_TRY(cudaGetDevice(&dev));
   if (dev < 0 || dev >= 64 || !configured[dev]) {
     DeviceInfo di;
     if (int rc = get_device_info(&di)) return rc;
-    CUTB_CUDA_TRY(cudaFuncSetAttribute(dense_matvec_kernel<R, UNR, GRU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)di.smem_optin - 2048));
+    CUTB_CUDA_TRY(cudaFuncSetAttribute(dense_matvec_kernel<R, UNR, GRU, PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)di.smem_optin - 2048));
     if (dev >= 0 && dev < 64) configured[dev] = true;
   }
   const uint32_t per_sm = (p.ntiles + sms - 1) / sms, turns = (per_sm + MV_MAX_WARPS - 1) / MV_MAX_WARPS;
@@ -192,9 +192,9 @@ template <int R, int UNR, bool GRU> int mv_launch(MvParams &p, uint32_t smem, ui
   if (warps < MV_MIN_WARPS) warps = MV_MIN_WARPS;  // (the staging of the input wants threads too)
   const dim3 grid(p.ntiles < sms ? p.ntiles : sms), block(32 * warps);
   if (overlap) {
-    CUTB_CUDA_TRY(launch_pdl(dense_matvec_kernel<R, UNR, GRU>, grid, block, smem, stream, p));
+    CUTB_CUDA_TRY(launch_pdl(dense_matvec_kernel<R, UNR, GRU, PLAIN>, grid, block, smem, stream, p));
   } else {
-    dense_matvec_kernel<R, UNR, GRU><<<grid, block, smem, stream>>>(p);
+    dense_matvec_kernel<R, UNR, GRU, PLAIN><<<grid, block, smem, stream>>>(p);
     CUTB_CUDA_TRY(cudaGetLastError());
   }
   return CUTB_OK;
@@ -357,8 +357,14 @@ int dense_matvec_launch(const cutb_dense_desc &d, cudaStream_t stream) {
   p.ntiles = gru ? d.N / 3 : (two ? (d.N + 1) / 2 : d.N);
   const uint32_t smem = mv_smem_bytes(d);
   const bool overlap = !(d.flags & CUTB_FLAG_NO_OVERLAP);
-  if (gru) return mv_launch<3, 1, true>(p, smem, sms, overlap, stream);
-  return two ? mv_launch<2, 2, false>(p, smem, sms, overlap, stream) : mv_launch<1, 4, false>(p, smem, sms, overlap, stream);
+  if (gru && (!norm_stage_plain(p.norm) || p.norm_out)) {
+    set_last_error("dense_matvec: the recurrence step behind a layer norm or a plain residual, or with the normed row kept, is not built");
+    return CUTB_ERR_UNSUPPORTED;
+  }
+  if (!norm_stage_plain(p.norm))
+    return two ? mv_launch<2, 2, false, false>(p, smem, sms, overlap, stream) : mv_launch<1, 4, false, false>(p, smem, sms, overlap, stream);
+  if (gru) return mv_launch<3, 1, true, true>(p, smem, sms, overlap, stream);
+  return two ? mv_launch<2, 2, false, true>(p, smem, sms, overlap, stream) : mv_launch<1, 4, false, true>(p, smem, sms, overlap, stream);
 }
 
 }  // namespace cutb

@@ -122,7 +122,7 @@ template <bool UP> __global__ void __launch_bounds__(32 * ex_max_warps(UP), 1) e
         n.x = p.xd, n.pre_w = p.xd_norm_w, n.dim = p.Kd, n.groups = 1, n.eps = p.eps;
         auto n1 = [&](uint32_t i, float v) { put1(0, i, v); };
         auto n4 = [&](uint32_t i, float4 v) { (i & 4 ? hi : lo)[i >> 3] = v; };
-        if (norm_stage_fits(p.Kd, 1, nt, 2)) stage_norm_regs<2>(n, z + epad, nullptr, false, n4);
+        if (norm_stage_fits(p.Kd, 1, nt, 2)) stage_norm_regs<2, true>(n, z + epad, nullptr, false, n4);
         else stage_norm(n, z + epad, false, n4, n1);
       } else {
         put_row(0, p.xd, p.Kd, p.Kd8);

@@ -45,7 +45,7 @@ __global__ void __launch_bounds__(256) embedding_bigram_kernel(const cutb_embed_
 }
 
 // One block per row: x' = x + y_scale P(y + gathered parts), h = N(x') (norm_stage.cuh), h in bf16 or fp32.
-template <int IT>  // 16-byte pieces per thread of the register path; 0: any row
+template <int IT, bool PLAIN>  // 16-byte pieces per thread of the register path; 0: any row
 __global__ void __launch_bounds__(512) residual_norm_kernel(NormStage n, uint64_t ldx, uint64_t ldy, const uint32_t *row_index, void *h,
                                                             uint64_t ldh, int h_bf16) {
   extern __shared__ __align__(16) float rn_smem[];
@@ -61,7 +61,7 @@ __global__ void __launch_bounds__(512) residual_norm_kernel(NormStage n, uint64_
     else *reinterpret_cast<float4 *>(reinterpret_cast<float *>(h) + base + i) = v;
   };
   auto put1 = [&](uint32_t i, float v) { store_out(h, h_bf16, base + i, v); };
-  if constexpr (IT > 0) stage_norm_regs<IT>(n, rn_smem, nullptr, n.x_out != nullptr, put4);
+  if constexpr (IT > 0) stage_norm_regs<IT, PLAIN>(n, rn_smem, nullptr, n.x_out != nullptr, put4);
   else stage_norm(n, rn_smem, n.x_out != nullptr, put4, put1);
 }
 
@@ -159,10 +159,10 @@ int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) 
     auto go = [&](auto kernel, uint32_t threads) -> cudaError_t {
       return launch_pdl(kernel, dim3(d.rows), dim3(threads), small, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16);
     };
-    if (d.dim <= 1024) CUTB_CUDA_TRY(go(residual_norm_kernel<2>, 128));
-    else if (d.dim <= 2048) CUTB_CUDA_TRY(go(residual_norm_kernel<2>, 256));
-    else if (d.dim <= 4096) CUTB_CUDA_TRY(go(residual_norm_kernel<2>, 512));
-    else CUTB_CUDA_TRY(go(residual_norm_kernel<4>, 512));
+    const bool plain = norm_stage_plain(n);
+    const uint32_t threads = d.dim <= 1024 ? 128 : d.dim <= 2048 ? 256 : 512;
+    if (d.dim <= 4096) CUTB_CUDA_TRY(plain ? go(residual_norm_kernel<2, true>, threads) : go(residual_norm_kernel<2, false>, threads));
+    else CUTB_CUDA_TRY(plain ? go(residual_norm_kernel<4, true>, threads) : go(residual_norm_kernel<4, false>, threads));
     return CUTB_OK;
   }
   const uint32_t smem = 4 * norm_stage_floats(d.dim, d.groups);
@@ -173,9 +173,9 @@ int residual_norm_launch(const cutb_residual_norm_desc &d, cudaStream_t stream) 
       set_last_error("residual_norm: rows of %u elements do not fit in shared memory", d.dim);
       return CUTB_ERR_UNSUPPORTED;
     }
-    CUTB_CUDA_TRY(cudaFuncSetAttribute(residual_norm_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    CUTB_CUDA_TRY(cudaFuncSetAttribute(residual_norm_kernel<0, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
   }
-  CUTB_CUDA_TRY(launch_pdl(residual_norm_kernel<0>, dim3(d.rows), dim3(256), smem, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16));
+  CUTB_CUDA_TRY(launch_pdl(residual_norm_kernel<0, false>, dim3(d.rows), dim3(256), smem, stream, n, d.ldx, d.ldy, d.row_index, d.h, d.ldh, bf16));
   return CUTB_OK;
 }
 

@@ -110,8 +110,8 @@ __device__ __forceinline__ void group_factors(const float *row, const NormStage 
 // Fast path for rows whose groups are whole multiples of 128 elements and which the block holds in registers (IT 16-byte pieces
 // per thread): a warp's piece of 128 elements lies in one group, its moments are entries of `part`, and every warp merges its
 // own group's entries.  Two barriers in all.  `norms` (optional): post_w then pre_w in shared memory, copied there by this
-// block's own cp.async.
-template <int IT, class Store4>
+// block's own cp.async.  PLAIN: RMS norms before and after, nothing gathered, y_scale 1 (norm_stage_plain), known at compile time.
+template <int IT, bool PLAIN, class Store4>
 __device__ __forceinline__ void stage_norm_regs(const NormStage &n, float *part, const float *norms, bool write_x, Store4 store4) {
   const uint32_t tid = threadIdx.x, lane = tid & 31, nt = blockDim.x, d4 = n.dim / 4, chunks = n.dim / 128, per = chunks / n.groups;
   const float inv_gs = 1.0f / (float)(n.dim / n.groups);
@@ -120,15 +120,17 @@ __device__ __forceinline__ void stage_norm_regs(const NormStage &n, float *part,
   for (int it = 0; it < IT; ++it) {
     const uint32_t i = tid + it * nt;
     x[it] = i < d4 ? reinterpret_cast<const float4 *>(n.x)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
-    y[it] = i < d4 ? stage_y4(n, i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if constexpr (PLAIN) y[it] = n.y && i < d4 ? reinterpret_cast<const float4 *>(n.y)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+    else y[it] = i < d4 ? stage_y4(n, i) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
+  const bool center = !PLAIN && n.center;
   if (norms) asm volatile("cp.async.wait_all;" ::: "memory");  // (this thread's pieces; a barrier lies before their use)
   auto factors = [&](float4 (&v)[IT], float *buf, float (&f)[IT]) {  // centred: v loses its mean here
     float *dev = buf + chunks;
 #pragma unroll
     for (int it = 0; it < IT; ++it) {
       const uint32_t c = (tid + it * nt) / 32;
-      if (n.center) {
+      if (center) {
         const float m = warp_sum((v[it].x + v[it].y) + (v[it].z + v[it].w)) * (1.0f / 128.0f);
         const float a = v[it].x - m, b = v[it].y - m, e = v[it].z - m, g = v[it].w - m;
         const float s = warp_sum(fmaf(a, a, fmaf(b, b, fmaf(e, e, g * g))));
@@ -146,7 +148,7 @@ __device__ __forceinline__ void stage_norm_regs(const NormStage &n, float *part,
       if (c < chunks)
         for (uint32_t k = lane; k < per; k += 32) s += buf[g0 + k];
       s = warp_sum(s);
-      if (n.center) {
+      if (center) {
         const float m = s / (float)per;
         s = 0.f;
         if (c < chunks)
@@ -161,7 +163,21 @@ __device__ __forceinline__ void stage_norm_regs(const NormStage &n, float *part,
     }
   };
   float f[IT];
-  if (stage_has_y(n)) {
+  if (PLAIN && n.y) {
+    factors(y, part, f);
+    const float4 *w4 = reinterpret_cast<const float4 *>(norms ? norms : n.post_w);
+#pragma unroll
+    for (int it = 0; it < IT; ++it) {
+      const uint32_t i = tid + it * nt;
+      if (i < d4) {
+        const float4 w = w4[i];
+        x[it].x = fmaf(y[it].x * f[it], w.x, x[it].x), x[it].y = fmaf(y[it].y * f[it], w.y, x[it].y);
+        x[it].z = fmaf(y[it].z * f[it], w.z, x[it].z), x[it].w = fmaf(y[it].w * f[it], w.w, x[it].w);
+        if (write_x) reinterpret_cast<float4 *>(n.x_out)[i] = x[it];
+      }
+    }
+  }
+  if (!PLAIN && stage_has_y(n)) {
     if (n.post_w) {
       factors(y, part, f);
       const float4 *w4 = reinterpret_cast<const float4 *>(norms ? norms : n.post_w);
@@ -192,6 +208,9 @@ __device__ __forceinline__ void stage_norm_regs(const NormStage &n, float *part,
       store4(4 * i, make_float4(x[it].x * f[it] * w.x, x[it].y * f[it] * w.y, x[it].z * f[it] * w.z, x[it].w * f[it] * w.w));
     }
   }
+}
+__host__ __device__ inline bool norm_stage_plain(const NormStage &n) {
+  return !n.center && n.n_parts == 0 && (!n.y || (n.post_w && n.y_scale == 1.0f));
 }
 __host__ __device__ inline bool norm_stage_fits(uint32_t dim, uint32_t groups, uint32_t threads, int it) {
   return dim % groups == 0 && dim / groups % 128 == 0 && dim <= threads * 4 * (uint32_t)it;
