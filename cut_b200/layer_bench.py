@@ -378,9 +378,10 @@ def latent_table(roof: Roofline, hidden, H, dim, rot, vdim, q_rank, rank, E, top
     put(f"decode experts up {top}x{2 * ff}x{hidden} + queries {n_uq}x{q_rank}", up, ub, like=dense_like(ub // (2 * hidden), hidden, norm=True))
     put(f"decode experts down {hidden}x{top}x{ff} + output {hidden}x{H * vdim}", down, db, like=dense_like(hidden, H * vdim + top * ff))
     put(f"decode queries into latent space {H}x{rank}x{dim}", head_matvec_us(H, rank, dim), mv_bytes(H * rank, dim), like=dense_like(H * dim, rank))
-    att, val = latent_decode_us(H, dim, rot, vdim, rank, context)
-    put(f"decode latent attention, context {context}", att, context * (rank + rot) * 2 + 4 * H * (rank + wide),
-        4.0 * H * context * (2 * rank + rot) / 2, like=(window_us(1, H, kv_heads, dim, context, True, context), context * kv_heads * dim * 4 + 8 * H * dim))
+    for c in (context, 8 * context):
+        att, val = latent_decode_us(H, dim, rot, vdim, rank, c)
+        put(f"decode latent attention, context {c}", att, c * (rank + rot) * 2 + 4 * H * (rank + wide), 2.0 * H * c * (2 * rank + rot),
+            like=(window_us(1, H, kv_heads, dim, c, True, c), c * kv_heads * dim * 4 + 8 * H * dim))
     put(f"decode values out of latent space {H}x{vdim}x{rank}", val, mv_bytes(H * vdim, rank), like=dense_like(H * vdim, rank))
     put(f"decode head mat-vec (layer norm fused) {vocab}x{hidden}", matvec_us(vocab, hidden, norm=True), mv_bytes(vocab, hidden), like=dense_like(vocab, hidden, norm=True))
 
