@@ -358,7 +358,7 @@ def parallel_norm_us(T: int, dim: int, top: int) -> float:
         h, rows = torch.zeros((T, dim), device="cuda", dtype=torch.bfloat16), torch.randperm(T * top, device="cuda").to(torch.int32).view(T, top)
         pw = torch.rand((T, top), device="cuda")
         keep.append((x, y, m, h, rows, pw))
-        launches.append(lambda a=keep[-1]: ops.residual_norm(a[0], w, 1, 1e-6, y=a[1], x_out=a[0], out=a[3], center=True, y_scale=0.3, parts=(a[2], a[4], a[5])))
+        launches.append(lambda a=keep[-1]: ops.residual_norm(a[0], w, 1, 1e-6, y=a[1], x_out=a[0], out=a[3], center=True, y_scale=0.4, parts=(a[2], a[4], a[5])))
     return time_us(launches)
 
 
@@ -414,7 +414,7 @@ def latent_model_config(hidden, H, dim, rot, vdim, q_rank, rank, E, top, ff, n_l
     """Every other layer reads the latents of the one before it."""
     att = lambda j: LatentAttention(H, dim, vdim, q_rank, rank, (dim + rot) ** -0.5, Rotation(10000.0, rot), True, j)
     layers = tuple(Layer(att(None if i % 2 == 0 else i - 1), MixtureOfExperts(E, top, ff, 7.0, 1.702, 1.0)) for i in range(n_layers))
-    return LayerListConfig(hidden, vocab, layers, 1, 1e-6, norm_center=True, parallel=True, residual_mult=0.3, embed_scale=2.0, tied_head=True)
+    return LayerListConfig(hidden, vocab, layers, 1, 1e-6, norm_center=True, parallel=True, residual_mult=0.4, embed_scale=2.0, tied_head=True)
 
 
 def latent_random_weights(cfg: LayerListConfig) -> dict:

@@ -148,7 +148,7 @@ class Moe:
         torch.cuda.synchronize()
 
 
-MOE = [(1, 4, 2, 40, 24), (2, 8, 3, 70, 13), (33, 6, 6, 64, 40), (300, 16, 4, 128, 96), (700, 5, 1, 96, 64), (40, 200, 7, 72, 16), (9, 1, 1, 24, 8),
+MOE = [(1, 4, 2, 40, 24), (2, 8, 3, 70, 13), (33, 6, 6, 64, 40), (300, 12, 3, 128, 104), (700, 5, 1, 96, 64), (40, 200, 7, 72, 16), (9, 1, 1, 24, 8),
        (513, 64, 8, 256, 136), (20, 37, 2, 512, 300)]
 
 
